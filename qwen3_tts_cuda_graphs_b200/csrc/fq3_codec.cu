@@ -317,7 +317,7 @@ __device__ __forceinline__ uint64_t umma_desc_sw128(uint32_t smem_addr) {
 // Split-K (splits > 1, short-and-wide problems that would leave most SMs idle): blockIdx.z takes a contiguous range of
 // k-blocks and stores its raw fp32 tile into the workspace [split][M][Nw]; fq3c_splitk_reduce_kernel adds the splits in
 // order and applies the fused epilogue.
-// TMA = true: the operand tiles arrive by cp.async.bulk.tensor (SASS UTMALDG) — one elected thread asks for the A box (128 rows x 64
+// TMA = true: the operand tiles arrive by cp.async.bulk.tensor — one elected thread asks for the A box (128 rows x 64
 // columns at row m0 + tap offset: rows outside the tensor, i.e. the causal padding, come back as zeros) and the B box (BN x 64) of a
 // k-block and both count their bytes on the stage's `full` mbarrier; SWIZZLE_128B writes exactly the layout described above.  Used
 // whenever a k-block cannot straddle two taps (one tap, or c_in a multiple of 64); the cp.async loaders stay for the rest.

@@ -4,8 +4,8 @@
 // attention / sampling).  One CTA per SM runs the whole program.  Every GEMV weight matrix is kept in HBM as a
 // *fragment image*: groups of 8 consecutive rows, each group a run of 512-byte blocks (8 rows x 32 columns) laid out
 // so that one 16-byte shared-memory load per lane yields the mma.m16n8k16 B fragments of two k-steps.  A producer
-// warp streams a CTA's groups through a shared-memory ring of 16 KB stages with cp.async.bulk (TMA bulk copy, SASS
-// UBLKCP) — one contiguous copy per stage — and runs ahead of the consumers across phases and frames, so HBM stays
+// warp streams a CTA's groups through a shared-memory ring of 16 KB stages with cp.async.bulk (TMA bulk copy)
+// — one contiguous copy per stage — and runs ahead of the consumers across phases and frames, so HBM stays
 // busy while the CTAs wait for each other.  The activations are the A operand (one stream per A row), so after the
 // k loop every lane holds the dot products of one (stream, output word).  See DESIGN.md §3.
 #pragma once
