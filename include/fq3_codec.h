@@ -172,6 +172,26 @@ enum fq3c_kind {
    *     taps 1-3, M >= 512: when ws has room behind the per-row coefficients (rounded up to four floats) for P pieces' states and
    *     decay products, P * i0 * i2 * (cin + 1) floats with 2 <= P <= 16, the rows are cut into P pieces that are walked side by
    *     side, twice (own contribution from zero; start states by a carry pass; outputs): same sums in another order.              */
+  /* ABI 10 adds to existing kinds:
+   *   FQ3C_EMBED: C2, when given: the row also in the table's type, at pitch ldr, i1 times side by side (columns 0, N, ..): the operand of
+   *     a product that reads the embedding.
+   *   FQ3C_GNORM: bias (f32 [M, cin], one divisor per row and group), when given: the group is divided by it first; FQ3C_SIGMOID: the gate
+   *     p1 is a sigmoid instead of a silu.
+   *   FQ3C_SUM_NORM: norm_out without norm_w: the finished row itself.
+   *   FQ3C_ROT_APPEND: FQ3C_UNIT: heads are divided by their root mean square over i2 entries (eps f0), no weights (a rotation keeps it).
+   *     m_begin = P > 0: every block of P positions bP .. bP + P - 1 that the step completes leaves the mean of its P rows of the caches
+   *     as row b of norm_out (keys, pitch ldc) and ws (values, pitch ldr), in the caches' type.
+   *   FQ3C_CACHE_ATTN: tap_off[1] = P > 0 (with a window K): C2 / norm_out = those pooled rows; beside its tokens, position i sees the
+   *     blocks that lie wholly before its window (bP + P - 1 <= i - K), in the same softmax.
+   *   FQ3C_MSTATE_SCAN: taps = 4 (forget gates that also decide what is written): queries of head h at column h * i2, gate logits at
+   *     col_mod + h * i2, values at a_rows + h * cin of the rows A; l = scale f32 [i0 * i2];  f = l + (1 - l) sigmoid(z);
+   *     S <- diag(f) S + (1 - f) v^T;  o = f0 S^T silu(q);  ws = f32 [M, round_up(3 * i0 * i2, 4)].
+   *     taps = 5 (exponential gates under a running maximum): queries at h * i2, keys at K + h * i2, values at a_rows + h * cin; gate logits
+   *     per head in the rows res at columns col_mod (input) and m_begin (forget);  li = f1 tanh(zi / f1), lf = log sigmoid(f1 tanh(zf / f1));
+   *     m' = max(lf + m, li);  S <- e^(lf + m - m') S + e^(li - m') k v^T;  n likewise with k alone;  C = f0 S^T q, and
+   *     norm_out[row, h] (f32, pitch norm_ld) = max(|f0 n . q|, e^(-m')) + norm_eps, what the read-out is to be divided by.  The state p0 / C2
+   *     is f32 [i0, i2, cin + 1] (column cin = n), the maxima are read from scale (f32 [i0]) and written to p1;
+   *     ws = f32 [M, round_up(3 * i0, 4)].  Both: no workspace up to 16 rows; pieces as above, with states of cin + 1 columns for taps = 5.   */
 };
 
 enum fq3c_flags {
@@ -192,7 +212,9 @@ enum fq3c_flags {
   /* ABI 9 */
   FQ3C_RELU2 = 131072   /* GEMM / GGEMM on the sequence products: max(z, 0)^2 */,
   FQ3C_CENTER = 262144  /* GNORM / SUM_NORM: subtract the mean, divide by the root of the variance (layer norm) */,
-  FQ3C_ROT_HALF = 524288 /* ROT_APPEND: the turning pairs are (i, i + taps / 2) */
+  FQ3C_ROT_HALF = 524288 /* ROT_APPEND: the turning pairs are (i, i + taps / 2) */,
+  /* ABI 10 */
+  FQ3C_UNIT = 1048576   /* ROT_APPEND: heads are divided by their root mean square, no weights */
 };
 
 typedef struct fq3c_op {

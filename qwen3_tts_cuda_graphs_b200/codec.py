@@ -41,6 +41,7 @@ F_F32, F_NOROUND, F_GELU_TANH, F_SIGMOID, F_A_F32 = 512, 1024, 2048, 4096, 8192
 F_GATE_PRE, F_GATE_POST = 16384, 32768
 F_RAW_WEIGHTS = 65536
 F_RELU2, F_CENTER, F_ROT_HALF = 131072, 262144, 524288
+F_UNIT = 1048576
 
 
 class Op(C.Structure):
@@ -150,7 +151,7 @@ def load_lib():
     lib.fq3c_graph_launch.argtypes = [C.c_void_p, C.c_void_p]
     lib.fq3c_graph_destroy.restype = C.c_int
     lib.fq3c_graph_destroy.argtypes = [C.c_void_p]
-    if lib.fq3c_abi_version() != 9:
+    if lib.fq3c_abi_version() != 10:
         raise CodecError("libfq3codec.so ABI version mismatch")
     _lib = lib
     return lib

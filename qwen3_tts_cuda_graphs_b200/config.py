@@ -368,12 +368,17 @@ class SoftmaxAttentionConfig:
     keep_first: int = 0      # ... or j < keep_first
     sink: bool = False
     gate: bool = False       # one sigmoid gate per head on the head's output
-    bias: bool = False       # q, k, v and output projections have biases
+    bias: bool = False       # q, k, v and (out_bias) output projections have biases
     distance: bool = False   # score -= r1_h ln(1 + r2_h (i - j))
     kv_from: Optional[int] = None   # index of the layer whose cached keys / values this layer reads
     chunk: int = 0           # > 0: position i sees j only inside its own chunk (i // chunk == j // chunk), chunks from position 0
     qk_norm: bool = False    # queries and keys are RMS-normed per head (one weight vector each, shared by the heads)
     zero_sink: bool = False  # a sink of score 0 without a tensor: the softmax denominator holds one more 1
+    out_bias: bool = True    # with `bias`: the output projection has one too
+    rot_factor: float = 1.0  # every rotary frequency is divided by it (linear scaling)
+    qk_unit: bool = False    # queries and keys are divided by their root mean square per head, no weights
+    pool: int = 0            # > 0 (with a window): every block of this many positions that lies wholly before the window is seen
+                             # as one more key and value, the means of its keys and of its values
 
 
 @dataclass(frozen=True)
@@ -631,12 +636,110 @@ class ZudusunConfig:
         return ZudusunConfig(int(raw["vocab"]), int(raw["width"]), float((raw.get("norm") or {}).get("eps", 1e-6)), tuple(layers), tuple(owner))
 
 
+@dataclass(frozen=True)
+class ForgetGateAttentionConfig:
+    """Linear attention whose forget gate per key channel and token also decides what is written (S <- diag(f) S + (1 - f) v^T, f with a
+    learned lower bound); the queries pass through silu, the read-out is RMS-normed per head and projected."""
+
+    heads: int
+    dim: int
+    vdim: int
+
+
+@dataclass(frozen=True)
+class MatrixMemoryConfig:
+    """A [dim, vdim] memory per head with exponential input and forget gates under a running maximum, read out over a normaliser; the
+    read-out is divided by its root mean square per head, weighted, gated by a sigmoid per entry and projected."""
+
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float          # both gates' logits pass cap * tanh(. / cap)
+
+
+@dataclass(frozen=True)
+class LoopConfig:
+    """Layers start .. stop - 1 run `times` times in a row on the same tensors; every pass starts by mixing the embedding output back in."""
+
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class SirodraConfig:
+    """Sirodra: layer norms (weight, no bias) in front of every sublayer; mixers in a configured order: linear attention with written
+    forget gates, a matrix memory with exponential gates, or windowed softmax attention that also sees pooled blocks before its window;
+    dense GELU feed-forwards or none; a range of layers that runs several times with the embedding output mixed in before each pass."""
+
+    architecture = "Sirodra"
+    vocab: int
+    width: int
+    norm_eps: float
+    layers: Tuple[SeqLayerConfig, ...]
+    loop: Optional[LoopConfig] = None
+
+    @property
+    def runs(self) -> Tuple[Tuple[int, bool], ...]:
+        """The layer runs of a step in order: (layer, whether a pass of the loop starts with it)."""
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            return tuple((i, False) for i in range(n))
+        once = [(i, i == lp.start) for i in range(lp.start, lp.stop)]
+        return tuple([(i, False) for i in range(lp.start)] + once * lp.times + [(i, False) for i in range(lp.stop, n)])
+
+    @staticmethod
+    def from_dict(raw: dict) -> "SirodraConfig":
+        layers = []
+        for i, L in enumerate(raw["layers"]):
+            m, kind = L["mixer"], L["type"]
+            if kind == "hgrn2":
+                mixer = ForgetGateAttentionConfig(int(m["heads"]), int(m["dim"]), int(m["vdim"]))
+            elif kind == "mlstm":
+                mixer = MatrixMemoryConfig(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+                if not mixer.gate_cap > 0:
+                    raise ValueError(f"layer {i}: gate_cap must be positive")
+            elif kind == "attention":
+                rot, mask = m.get("rot") or {}, m.get("mask") or {}
+                mixer = SoftmaxAttentionConfig(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                               rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
+                                               window=int(mask.get("size") or 0), gate=True, bias=True, out_bias=False,
+                                               rot_factor=float((rot.get("scaling") or {}).get("factor", 1.0)), qk_unit=True,
+                                               pool=int(mask.get("pool") or 0))
+                if mixer.heads % mixer.kv_heads:
+                    raise ValueError(f"layer {i}: kv_heads must divide heads")
+                if mixer.rot_dims % 2 or mixer.rot_dims > mixer.dim:
+                    raise ValueError(f"layer {i}: rot.dims must be even and at most dim")
+                if mixer.window < 0 or mixer.pool < 0 or (mixer.pool > 0 and mixer.window < 1):
+                    raise ValueError(f"layer {i}: pooled blocks need a window")
+                if not mixer.rot_factor > 0:
+                    raise ValueError(f"layer {i}: the rotary scaling factor must be positive")
+            else:
+                raise ValueError(f"unknown mixer type {kind!r}")
+            f = L.get("mlp")
+            if f is None:
+                mlp = None
+            elif f.get("kind", "dense") == "dense":
+                mlp = DenseFFConfig(int(f["ff"]))
+            else:
+                raise ValueError(f"unknown feed-forward kind {f['kind']!r}")
+            layers.append(SeqLayerConfig(kind, mixer, mlp))
+        lp = raw.get("loop")
+        loop = None
+        if lp is not None:
+            loop = LoopConfig(int(lp["start"]), int(lp["stop"]), int(lp["times"]))
+            if not 0 <= loop.start < loop.stop <= len(layers) or loop.times < 1:
+                raise ValueError("loop: 0 <= start < stop <= layers and at least one pass")
+        return SirodraConfig(int(raw["vocab"]), int(raw["width"]), float((raw.get("norm") or {}).get("eps", 1e-6)), tuple(layers), loop)
+
+
 # config.json "architecture" -> (config class, "module:class" of the model that lowers it to op lists)
 SEQUENCE_ARCHITECTURES = {
     "Sidalorn": (SidalornConfig, "sidalorn:SidalornModel"),
     "Redodra": (RedodraConfig, "redodra:RedodraModel"),
     "Ratizen": (RatizenConfig, "ratizen:RatizenModel"),
     "Zudusun": (ZudusunConfig, "zudusun:ZudusunModel"),
+    "Sirodra": (SirodraConfig, "sirodra:SirodraModel"),
 }
 
 

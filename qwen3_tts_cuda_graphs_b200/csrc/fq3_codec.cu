@@ -1061,6 +1061,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
     case FQ3C_EMBED:
       if (!o.A || !o.B || !o.C) return fail("embed: missing operand");
       if (o.i0 > 1 && o.K < o.N) return fail("embed: copies need a stride of at least N elements");
+      if (o.C2 && o.ldr < o.N * std::max(o.i1, 1)) return fail("embed: the operand copies do not fit their pitch");
       if (o.flags & FQ3C_F32) fq3s_embed_kernel<float><<<o.M, 128, 0, s>>>(o);
       else fq3s_embed_kernel<bf16><<<o.M, 128, 0, s>>>(o);
       return 0;
@@ -1217,12 +1218,23 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       if (!o.A || o.i0 < 0 || o.i1 < 0 || o.i2 < 1 || o.taps < 0 || (o.taps & 1) || o.taps > o.i2 || (o.taps > 0 && !o.B) ||
           (o.i1 > 0 && (!o.C || (o.cin > 0 && !o.C2))))
         return fail("rot_append: bad configuration");
-      if (o.flags & FQ3C_F32) fq3s_rot_append_kernel<float><<<o.M, 256, 0, s>>>(o);
+      if (o.m_begin > 0 && (o.i1 < 1 || o.cin < 1 || !o.norm_out || !o.ws || !o.p0)) return fail("rot_append: pooled blocks need both caches, their pooled rows and a position");
+      if (o.m_begin > 0 && o.M == 1 && (o.flags & FQ3C_F32)) fq3s_rot_append_kernel<float, true><<<1, 256, 0, s>>>(o);
+      else if (o.m_begin > 0 && o.M == 1) fq3s_rot_append_kernel<bf16, true><<<1, 256, 0, s>>>(o);
+      else if (o.flags & FQ3C_F32) fq3s_rot_append_kernel<float><<<o.M, 256, 0, s>>>(o);
       else fq3s_rot_append_kernel<bf16><<<o.M, 256, 0, s>>>(o);
+      if (o.m_begin > 0 && o.M > 1) {
+        const dim3 grid(o.M / o.m_begin + 1, (o.i1 * std::max(o.i2, o.cin) + 255) / 256, 2);
+        if (o.flags & FQ3C_F32) fq3s_pool_append_kernel<float><<<grid, 256, 0, s>>>(o);
+        else fq3s_pool_append_kernel<bf16><<<grid, 256, 0, s>>>(o);
+        count_launches(1);
+      }
       return 0;
     case FQ3C_CACHE_ATTN: {
       if (o.i0 < 1 || o.i1 < 1 || o.i0 % o.i1 || o.i2 < 1 || o.cin < 1 || !o.A || !o.B || !o.p1 || !o.C) return fail("cache_attn: bad configuration");
       const int splits = std::max(1, o.m_begin), HG = o.i0 / o.i1;
+      const bool pool = o.tap_off[1] > 0;
+      if (pool && (o.K < 1 || !o.C2 || !o.norm_out || o.bias || o.tap_off[0] > 0)) return fail("cache_attn: pooled blocks go with a window and their pooled rows, not with a chunked mask or a distance penalty");
       if (splits > 64) return fail("cache_attn: at most 64 key splits");
       if (splits > 1 && (!o.ws || o.ws_bytes < (int64_t)o.M * o.i0 * splits * (o.cin + 2) * 4)) return fail("cache_attn: workspace too small for the splits");
       // bf16 cache and a prompt portion: the tensor-core kernel (FQ3S_ATTN_MMA=0: CUDA cores everywhere)
@@ -1234,7 +1246,8 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         if (!mma_rows && (16 * w) % HG == 0) mma_rows = 16 * w;
       if (use_mma && mma_rows && !(o.flags & FQ3C_F32) && o.M > 8 && o.i2 % 16 == 0 && o.i2 <= 256 &&
           o.cin % 16 == 0 && o.cin <= 128 && o.ldr % 8 == 0 && o.taps % 8 == 0 && !(reinterpret_cast<uintptr_t>(o.B) & 15) &&
-          !(reinterpret_cast<uintptr_t>(o.p1) & 15) && (o.ldc % 2 == 0 || (o.flags & FQ3C_OUT_F32))) {
+          !(reinterpret_cast<uintptr_t>(o.p1) & 15) && (!pool || !((reinterpret_cast<uintptr_t>(o.C2) | reinterpret_cast<uintptr_t>(o.norm_out)) & 15)) &&
+          (o.ldc % 2 == 0 || (o.flags & FQ3C_OUT_F32))) {
         static bool mattr[64] = {};
         int dev = 0;
         cudaGetDevice(&dev);
@@ -1242,12 +1255,19 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
           cudaFuncSetAttribute(fq3s_cache_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
           cudaFuncSetAttribute(fq3s_cache_attn_mma_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
           cudaFuncSetAttribute(fq3s_cache_attn_mma_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+          cudaFuncSetAttribute(fq3s_cache_attn_mma_kernel<4, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+          cudaFuncSetAttribute(fq3s_cache_attn_mma_kernel<8, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+          cudaFuncSetAttribute(fq3s_cache_attn_mma_kernel<16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
           mattr[dev] = true;
         }
         const int ROWS = (mma_rows == 64 && o.M * HG >= 8192 && cache_attn_mma_smem(128, o.i2, o.cin) <= 110 * 1024) ? 128 : mma_rows, QBLK = ROWS / HG;
         dim3 grid((o.M + QBLK - 1) / QBLK, o.i1);
         const size_t smem = cache_attn_mma_smem(ROWS, o.i2, o.cin);
-        if (o.cin <= 32) fq3s_cache_attn_mma_kernel<4><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
+        if (pool) {
+          if (o.cin <= 32) fq3s_cache_attn_mma_kernel<4, true><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
+          else if (o.cin <= 64) fq3s_cache_attn_mma_kernel<8, true><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
+          else fq3s_cache_attn_mma_kernel<16, true><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
+        } else if (o.cin <= 32) fq3s_cache_attn_mma_kernel<4><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
         else if (o.cin <= 64) fq3s_cache_attn_mma_kernel<8><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
         else fq3s_cache_attn_mma_kernel<16><<<grid, ROWS * 2, smem, s>>>(o, ROWS);
         return 0;
@@ -1263,10 +1283,14 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       if (dev >= 0 && dev < 64 && !attr[dev]) {
         cudaFuncSetAttribute(fq3s_cache_attn_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         cudaFuncSetAttribute(fq3s_cache_attn_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(fq3s_cache_attn_kernel<float, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(fq3s_cache_attn_kernel<bf16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         attr[dev] = true;
       }
       dim3 grid((o.M + QB - 1) / QB, o.i1, splits);
-      if (o.flags & FQ3C_F32) fq3s_cache_attn_kernel<float><<<grid, 256, smem, s>>>(o, QB, TJ, splits);
+      if (pool && (o.flags & FQ3C_F32)) fq3s_cache_attn_kernel<float, true><<<grid, 256, smem, s>>>(o, QB, TJ, splits);
+      else if (pool) fq3s_cache_attn_kernel<bf16, true><<<grid, 256, smem, s>>>(o, QB, TJ, splits);
+      else if (o.flags & FQ3C_F32) fq3s_cache_attn_kernel<float><<<grid, 256, smem, s>>>(o, QB, TJ, splits);
       else fq3s_cache_attn_kernel<bf16><<<grid, 256, smem, s>>>(o, QB, TJ, splits);
       if (splits > 1) {
         fq3s_cache_attn_merge_kernel<<<dim3(o.M, o.i0), 128, 0, s>>>(o, splits);
@@ -1296,8 +1320,9 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       return 0;
     case FQ3C_MSTATE_SCAN: {
       if (o.i0 < 1 || o.i1 < 1 || o.i0 % o.i1 || o.i2 < 1 || o.cin < 1 || !o.A || !o.p0 || !o.C || !o.C2) return fail("mstate_scan: bad configuration");
-      if (o.taps < 0 || o.taps > 3)
-        return fail("mstate_scan: taps selects the delta rule (0), the state-space scan (1), a decay per key channel (2) or a fixed decay per head (3)");
+      if (o.taps < 0 || o.taps > 5)
+        return fail("mstate_scan: taps selects the delta rule (0), the state-space scan (1), a decay per key channel (2), a fixed decay per head (3), a forget gate "
+                    "per channel (4) or exponential gates (5)");
       if (o.i2 > 512) return fail("mstate_scan: at most 512 state rows per head");
       if (o.taps <= 1) {
         if (!o.res || !o.scale || !o.ws) return fail("mstate_scan: raw projections, A_log and a workspace required");
@@ -1306,10 +1331,21 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         if (!o.res || !o.ws || !o.B || o.i1 != o.i0 || o.m_begin < 1 || o.m_begin > MS_MAX_RANK)
           return fail("mstate_scan: channel decays need their latent rows, the up-projection (inner size 1 .. 1024), a workspace and one key head per head");
         if (o.ws_bytes < (int64_t)o.M * mstate_decay_cols(o.i0, o.i2) * 4) return fail("mstate_scan: workspace too small");
-      } else if (!o.scale || o.i1 != o.i0) {
-        return fail("mstate_scan: fixed decays need one value and one key head per head");
+      } else if (o.taps == 3) {
+        if (!o.scale || o.i1 != o.i0) return fail("mstate_scan: fixed decays need one value and one key head per head");
+      } else {
+        if (!o.scale || o.i1 != o.i0 || (o.taps == 5 && (!o.res || !o.p1 || !o.norm_out || o.norm_ld < o.i0 || !(o.f1 > 0.f))))
+          return fail("mstate_scan: gates need their bounds or maxima, one key head per head, and exponential gates a cap and room for the divisors");
+        const int cols = o.taps == 4 ? mstate_gate_cols(o.i0, o.i2) : mstate_max_cols(o.i0);
+        if (o.M > MS_CH && (!o.ws || o.ws_bytes < (int64_t)o.M * cols * 4)) return fail("mstate_scan: workspace too small");
       }
-      if (o.taps != 3) {
+      if (o.taps == 4 && o.M > MS_CH) {
+        fq3s_mstate_gate_kernel<<<dim3(o.M, (o.i0 * o.i2 + 255) / 256), 256, 0, s>>>(o);
+        count_launches(1);
+      } else if (o.taps == 5 && o.M > MS_CH) {
+        fq3s_mstate_max_kernel<<<o.i0, 256, 0, s>>>(o);
+        count_launches(1);
+      } else if (o.taps < 3) {
         fq3s_mstate_prep_kernel<<<o.taps == 2 ? (o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS : o.M, 128, 0, s>>>(o);
         count_launches(1);
       }
@@ -1318,16 +1354,24 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       cudaGetDevice(&dev);
       if (dev >= 0 && dev < 64 && !sattr[dev]) {
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<16, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 72 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<16, 3, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 72 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32, 3, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 216 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 3, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 216 * 1024);
         sattr[dev] = true;
       }
       // Long runs of a recurrence whose decays do not depend on the state: pieces walked twice (see the kernel), when the caller's
       // workspace has room behind the per-row coefficients for the pieces' states and decay products.
-      const int64_t base = o.taps == 3 ? 0 : ((int64_t)o.M * (o.taps == 2 ? mstate_decay_cols(o.i0, o.i2) : mstate_ws_cols(o.i0, o.i1, o.i2, false)) + 3) & ~(int64_t)3;
-      const int64_t per_piece = (int64_t)o.i0 * o.i2 * (o.cin + 1);
+      const int sv = o.taps == 5 ? o.cin + 1 : o.cin;      // state columns (exponential gates: the normaliser is one more)
+      const int coef = o.taps == 3 ? 0 : o.taps == 5 ? mstate_max_cols(o.i0) : o.taps == 4 ? mstate_gate_cols(o.i0, o.i2)
+                     : o.taps == 2 ? mstate_decay_cols(o.i0, o.i2) : mstate_ws_cols(o.i0, o.i1, o.i2, false);
+      const int64_t base = ((int64_t)o.M * coef + 3) & ~(int64_t)3;
+      const int64_t per_piece = (int64_t)o.i0 * o.i2 * (sv + 1);
       int pieces = 1, piece = o.M;
       if (o.taps != 0 && o.M >= 512 && o.ws) {
         pieces = (int)std::min<int64_t>(std::min(16, o.M / 128), (o.ws_bytes / 4 - base) / per_piece);
@@ -1338,35 +1382,36 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         if (pieces < 2) { pieces = 1; piece = o.M; }
       }
       float* X = pieces > 1 ? reinterpret_cast<float*>(o.ws) + base : nullptr;
-      float* P = pieces > 1 ? X + (int64_t)pieces * o.i0 * o.i2 * o.cin : nullptr;
-      const dim3 tiles((o.cin + MS_COLS - 1) / MS_COLS, o.i0);
+      float* P = pieces > 1 ? X + (int64_t)pieces * o.i0 * o.i2 * sv : nullptr;
+      const dim3 tiles((sv + MS_COLS - 1) / MS_COLS, o.i0);
+      const int bound = o.i2 <= 32 ? 4 : o.i2 <= 64 ? 8 : o.i2 <= 128 ? 16 : o.i2 <= 256 ? 32 : 64;      // state rows a lane holds
+      const bool three = o.taps == 2 || o.taps == 4, gated = o.taps >= 4;
       auto walk = [&](const int phase, const int nz) {
         const dim3 grid(tiles.x, tiles.y, nz);
-        if (o.taps == 2) {
-          if (o.i2 <= 32) fq3s_mstate_scan_kernel<4, 3><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(4, 3), s>>>(o, phase, piece, X, P);
-          else if (o.i2 <= 64) fq3s_mstate_scan_kernel<8, 3><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(8, 3), s>>>(o, phase, piece, X, P);
-          else if (o.i2 <= 128) fq3s_mstate_scan_kernel<16, 3><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(16, 3), s>>>(o, phase, piece, X, P);
-          else if (o.i2 <= 256) fq3s_mstate_scan_kernel<32, 3><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(32, 3), s>>>(o, phase, piece, X, P);
-          else fq3s_mstate_scan_kernel<64, 3><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(64, 3), s>>>(o, phase, piece, X, P);
-        } else if (o.i2 <= 32) fq3s_mstate_scan_kernel<4><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(4), s>>>(o, phase, piece, X, P);
-        else if (o.i2 <= 64) fq3s_mstate_scan_kernel<8><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(8), s>>>(o, phase, piece, X, P);
-        else if (o.i2 <= 128) fq3s_mstate_scan_kernel<16><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(16), s>>>(o, phase, piece, X, P);
-        else if (o.i2 <= 256) fq3s_mstate_scan_kernel<32><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(32), s>>>(o, phase, piece, X, P);
-        else fq3s_mstate_scan_kernel<64><<<grid, 128, sizeof(float) * 2 * mstate_buf_floats(64), s>>>(o, phase, piece, X, P);
+        const size_t smem = sizeof(float) * 2 * mstate_buf_floats(bound, three ? 3 : 2);
+#define FQ3S_WALK(RPT) \
+  case RPT: \
+    if (three && gated) fq3s_mstate_scan_kernel<RPT, 3, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    else if (three) fq3s_mstate_scan_kernel<RPT, 3><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    else if (gated) fq3s_mstate_scan_kernel<RPT, 2, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    else fq3s_mstate_scan_kernel<RPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    break;
+        switch (bound) { FQ3S_WALK(4) FQ3S_WALK(8) FQ3S_WALK(16) FQ3S_WALK(32) FQ3S_WALK(64) }
+#undef FQ3S_WALK
       };
       if (pieces == 1) {
         walk(0, 1);
         return 0;
       }
       walk(1, pieces - 1);
-      const int64_t n = (int64_t)o.i0 * o.i2 * o.cin;
-      fq3s_mstate_carry_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>(o, pieces, X, P);
+      const int64_t n = (int64_t)o.i0 * o.i2 * sv;
+      fq3s_mstate_carry_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>(o, pieces, X, P, sv);
       walk(3, pieces);
       count_launches(2);
       return 0;
     }
     case FQ3C_SUM_NORM: {
-      if (o.i0 < 1 || !o.A || !o.p0 || !o.C || (o.i0 > 1 && o.K < o.N) || (o.norm_out && !o.norm_w)) return fail("sum_norm: missing operand");
+      if (o.i0 < 1 || !o.A || !o.p0 || !o.C || (o.i0 > 1 && o.K < o.N)) return fail("sum_norm: missing operand");
       if ((size_t)o.N * 4 > 200 * 1024) return fail("sum_norm: row too wide for shared memory");
       static bool nattr[64] = {};
       int dev = 0;
@@ -1386,7 +1431,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
 
 extern "C" {
 
-int fq3c_abi_version(void) { return 9; }
+int fq3c_abi_version(void) { return 10; }
 const char* fq3c_last_error(void) { return g_err.c_str(); }
 int64_t fq3c_launch_count(void) { return g_launches.load(); }
 

@@ -621,6 +621,8 @@ __global__ void fq3s_embed_kernel(const fq3c_op o) {
   for (int i = threadIdx.x; i < o.N; i += blockDim.x) {
     const float v = ldf<TB>(row + i) * sc;
     for (int s = 0; s < copies; ++s) c[(size_t)s * (size_t)o.K + i] = v;
+    if (o.C2)
+      for (int t = 0; t < max(o.i1, 1); ++t) stf(reinterpret_cast<TB*>(o.C2) + (size_t)m * o.ldr + (size_t)t * o.N + i, v);
   }
 }
 
@@ -649,28 +651,32 @@ __global__ void __launch_bounds__(256) fq3s_tconv_kernel(const fq3c_op o) {
   else reinterpret_cast<bf16*>(o.C)[(size_t)m * o.ldc + c] = __float2bfloat16_rn(a);
 }
 
-// grid (M, groups); one block per (row, group).  FQ3C_CENTER: mean and variance instead of the mean square.  An optional silu gate (p1, pitch i1) multiplies the row before the statistics
-// (FQ3C_GATE_PRE) or the finished row (FQ3C_GATE_POST); weights repeat with period i2 when i2 > 0.
+// grid (M, groups); one block per (row, group).  FQ3C_CENTER: mean and variance instead of the mean square.  An optional silu gate (p1, pitch i1;
+// FQ3C_SIGMOID: a sigmoid gate) multiplies the row before the statistics (FQ3C_GATE_PRE) or the finished row (FQ3C_GATE_POST); weights repeat
+// with period i2 when i2 > 0; divisors (bias, pitch cin) divide a group before anything else.
+__device__ __forceinline__ float gate_f(const float z, const bool plain) { return plain ? sigmoid_f(z) : z / (1.f + expf(-z)); }
 __global__ void __launch_bounds__(128) fq3s_gnorm_kernel(const fq3c_op o) {
   __shared__ float red[32];
   const int m = blockIdx.x, gsz = o.N / o.i0, c0 = blockIdx.y * gsz;
   const float* x = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda + c0;
   const bool pre = (o.flags & FQ3C_GATE_PRE) != 0, post = (o.flags & FQ3C_GATE_POST) != 0;
   const float* gate = (pre || post) ? reinterpret_cast<const float*>(o.p1) + (size_t)m * o.i1 + c0 : nullptr;
+  const bool plain = (o.flags & FQ3C_SIGMOID) != 0;
+  const float inv = o.bias ? 1.f / reinterpret_cast<const float*>(o.bias)[(size_t)m * o.cin + blockIdx.y] : 1.f;
   float mean = 0.f;
   if (o.flags & FQ3C_CENTER) {      // layer norm: the mean first, then the squared deviations from it (two passes, no cancellation)
     float sm = 0.f;
     for (int i = threadIdx.x; i < gsz; i += blockDim.x) {
-      float v = x[i];
-      if (pre) { const float z = gate[i]; v *= z / (1.f + expf(-z)); }
+      float v = x[i] * inv;
+      if (pre) v *= gate_f(gate[i], plain);
       sm += v;
     }
     mean = seq_block_sum(sm, red) / (float)gsz;
   }
   float ss = 0.f;
   for (int i = threadIdx.x; i < gsz; i += blockDim.x) {
-    float v = x[i];
-    if (pre) { const float z = gate[i]; v *= z / (1.f + expf(-z)); }
+    float v = x[i] * inv;
+    if (pre) v *= gate_f(gate[i], plain);
     v -= mean;
     ss = fmaf(v, v, ss);
   }
@@ -680,11 +686,11 @@ __global__ void __launch_bounds__(128) fq3s_gnorm_kernel(const fq3c_op o) {
   const int wmod = o.i2 > 0 ? o.i2 : o.N;
   const size_t orow = (size_t)m + (o.p0 ? (size_t)*reinterpret_cast<const int*>(o.p0) : 0);
   for (int i = threadIdx.x; i < gsz; i += blockDim.x) {
-    float v = x[i];
-    if (pre) { const float z = gate[i]; v *= z / (1.f + expf(-z)); }
+    float v = x[i] * inv;
+    if (pre) v *= gate_f(gate[i], plain);
     v = (v - mean) * rs;
     if (w) v *= w[(c0 + i) % wmod];
-    if (post) { const float z = gate[i]; v *= z / (1.f + expf(-z)); }
+    if (post) v *= gate_f(gate[i], plain);
     if (o.flags & FQ3C_RESID) v += reinterpret_cast<const float*>(o.res)[(size_t)m * o.ldr + c0 + i];
     if (o.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(o.C)[orow * o.ldc + c0 + i] = v;
     else reinterpret_cast<bf16*>(o.C)[orow * o.ldc + c0 + i] = __float2bfloat16_rn(v);
@@ -1318,10 +1324,34 @@ __global__ void __launch_bounds__(256) fq3s_xielu_kernel(const fq3c_op o) {
   else reinterpret_cast<bf16*>(o.C)[(size_t)m * o.ldc + c] = __float2bfloat16_rn(v);
 }
 
+// the mean of the P rows of block b of a cache -> row b of its pooled rows, for columns c0, c0 + step, .. below c1
+template <typename TC>
+__device__ __forceinline__ void pool_run(const TC* cache, const int ld, TC* pooled, const int b, const int P, const int c0, const int c1, const int step) {
+  for (int c = c0; c < c1; c += step) {
+    const TC* src = cache + (size_t)b * P * ld + c;
+    float sum = 0.f;
+    for (int r = 0; r < P; ++r) sum += ldf<TC>(src + (size_t)r * ld);
+    stf(pooled + (size_t)b * ld + c, sum / (float)P);
+  }
+}
+// grid (M / P + 1, ceil(i1 * max(i2, cin) / 256), 2): z = 0 keys, 1 values
+template <typename TC>
+__global__ void __launch_bounds__(256) fq3s_pool_append_kernel(const fq3c_op o) {
+  const int pos0 = o.p0 ? *reinterpret_cast<const int*>(o.p0) : 0, P = o.m_begin, b = pos0 / P + blockIdx.x;
+  if ((b + 1) * P > pos0 + o.M) return;
+  const int c = blockIdx.y * blockDim.x + threadIdx.x, n = o.i1 * (blockIdx.z ? o.cin : o.i2);
+  if (blockIdx.z == 0) pool_run<TC>(reinterpret_cast<const TC*>(o.C), o.ldc, reinterpret_cast<TC*>(o.norm_out), b, P, c, min(n, c + 1), 1);
+  else pool_run<TC>(reinterpret_cast<const TC*>(o.C2), o.ldr, reinterpret_cast<TC*>(o.ws), b, P, c, min(n, c + 1), 1);
+}
+
 // grid (M), 256 threads, a warp per query / key head.  Angles in f32: position (exact as a float below 2^24) times the frequency,
 // full-range sincosf; cos and sin times the amplitude f1 when that is set.  With norm weights a head is first divided by its root
-// mean square (eps f0) and multiplied by them.  Queries in place, keys (read from `res` rows when given) into the cache.
-template <typename TC>
+// mean square (eps f0) and multiplied by them; with FQ3C_UNIT it is divided only (a rotation keeps the root mean square, so it does
+// not matter which comes first).  Queries in place, keys (read from `res` rows when given) into the cache.
+// m_begin = P > 0: every run of P positions bP .. bP + P - 1 that the step completes leaves the mean of its P cached keys and values as
+// row b of norm_out / ws.  A single row does it here (POOL; its block has just written the run's last row); more rows take
+// fq3s_pool_append_kernel behind this launch.
+template <typename TC, bool POOL = false>
 __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
   const int m = blockIdx.x, H = o.i0, G = o.i1, d = o.i2, dv = o.cin, half = o.taps >> 1;
   const int pos = (o.p0 ? *reinterpret_cast<const int*>(o.p0) : 0) + m;
@@ -1335,8 +1365,9 @@ __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
     const bool isq = hh < H;
     const float* src = isq ? row + (size_t)hh * d : krow + o.K + (size_t)(hh - H) * d;
     const float* nw = reinterpret_cast<const float*>(isq ? o.scale : o.bias);
+    const bool normed = nw || (o.flags & FQ3C_UNIT);
     float rs = 1.f;
-    if (nw) {
+    if (normed) {
       float ss = 0.f;
       for (int c = lane; c < d; c += 32) ss = fmaf(src[c], src[c], ss);
       rs = 1.f / sqrtf(warp_sum(ss) / (float)d + o.f0);
@@ -1350,14 +1381,16 @@ __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
       sn *= amp; cs *= amp;
       const int ia = halves ? i : 2 * i, ib = halves ? i + half : 2 * i + 1;
       float a = src[ia], b = src[ib];
-      if (nw) { a = a * rs * nw[ia]; b = b * rs * nw[ib]; }
+      if (normed) { a *= rs; b *= rs; }
+      if (nw) { a *= nw[ia]; b *= nw[ib]; }
       const float x = a * cs - b * sn, y = b * cs + a * sn;
       if (isq) { qd[ia] = x; qd[ib] = y; }
       else { stf(kd + ia, x); stf(kd + ib, y); }
     }
-    if (isq && !nw) continue;     // the rest of a query head stays as it is
+    if (isq && !normed) continue;     // the rest of a query head stays as it is
     for (int c = 2 * half + lane; c < d; c += 32) {
-      const float v = nw ? src[c] * rs * nw[c] : src[c];
+      float v = normed ? src[c] * rs : src[c];
+      if (nw) v *= nw[c];
       if (isq) qd[c] = v;
       else stf(kd + c, v);
     }
@@ -1366,12 +1399,19 @@ __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
   TC* vc = reinterpret_cast<TC*>(o.C2) + (size_t)pos * o.ldr;
   const float* v = krow + o.a_rows;
   for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x) stf(vc + idx, v[idx]);
+  if (POOL && (pos + 1) % o.m_begin == 0) {
+    __syncthreads();
+    pool_run<TC>(reinterpret_cast<const TC*>(o.C), o.ldc, reinterpret_cast<TC*>(o.norm_out), pos / o.m_begin, o.m_begin, threadIdx.x, G * d, blockDim.x);
+    pool_run<TC>(reinterpret_cast<const TC*>(o.C2), o.ldr, reinterpret_cast<TC*>(o.ws), pos / o.m_begin, o.m_begin, threadIdx.x, G * dv, blockDim.x);
+  }
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
 // Softmax attention over a key / value cache on the CUDA cores, every sum in f32.  A block takes QB consecutive queries x the HG
 // query heads of one key / value head (R = QB * HG rows that score the same staged key tile), 256 threads, online softmax over
 // tiles of TJ keys; tiles that no row of the block can see (outside the window and beyond the kept first positions) are skipped.
+// Pooled blocks (tap_off[1] = P > 0): the rows of the pooled caches C2 / norm_out (means of P positions each) are keys and values of the
+// same softmax; position i sees the blocks that lie wholly before its window, i.e. the first (i - window + 1) / P.  Their tiles come first.
 // grid (ceil(M / QB), key heads, splits).  One split finishes in place (sink, output gate); several leave (max, sum, out) per
 // (row, split) in ws for fq3s_cache_attn_merge_kernel.
 // Shared memory (f32): q [R][d], keys [TJ][d + 1], values [TJ][dv], p [R][TJ], out [R][dv], max / sum / rescale [3][R].
@@ -1380,7 +1420,8 @@ __host__ __device__ inline size_t cache_attn_smem(int R, int TJ, int d, int dv) 
   return sizeof(float) * ((size_t)R * d + (size_t)TJ * (d + 1) + (size_t)TJ * dv + (size_t)R * TJ + (size_t)R * dv + 3 * (size_t)R);
 }
 struct CacheAttnMask {
-  int window, keep, chunk;
+  int window, keep, chunk, pool;
+  __device__ __forceinline__ int blocks(int i) const { return pool > 0 ? max(0, i - window + 1) / pool : 0; }
   __device__ __forceinline__ bool sees(int i, int j) const {
     return j <= i && (window <= 0 || i - j < window || j < keep) && (chunk <= 0 || j >= i - i % chunk);
   }
@@ -1425,7 +1466,7 @@ __device__ __forceinline__ void ca_stage_rows(float* dst, const int dld, const T
     dst[(size_t)jj * dld + c] = jj < nvalid ? ldf<TC>(src + (size_t)jj * sld + c) : 0.f;
   }
 }
-template <typename TC>
+template <typename TC, bool POOL = false>
 __global__ void __launch_bounds__(256) fq3s_cache_attn_kernel(const fq3c_op o, const int QB, const int TJ, const int splits) {
   extern __shared__ float csm[];
   const int H = o.i0, G = o.i1, d = o.i2, dv = o.cin, HG = H / G, R = QB * HG;
@@ -1441,12 +1482,13 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_kernel(const fq3c_op o, c
   float* al = ls + R;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nwarp = blockDim.x >> 5;
   const int P = o.p0 ? *reinterpret_cast<const int*>(o.p0) : 0;
-  const CacheAttnMask mask{o.K, o.a_rows, o.tap_off[0]};
+  const CacheAttnMask mask{o.K, o.a_rows, o.tap_off[0], o.tap_off[1]};
   const int ifirst = P + m0, ilast = P + m0 + nq - 1;
-  // the splits share the tiles from the first one any query of the block can see
-  const int ntiles = ilast / TJ + 1, tbeg = mask.lowest(ifirst) / TJ;
-  const int per = (ntiles - tbeg + splits - 1) / splits;
-  const int t0 = tbeg + z * per, t1 = min(ntiles, t0 + per);
+  // the splits share the tiles: those of the pooled blocks, then the tokens' from the first one any query of the block can see
+  const int npool = POOL ? mask.blocks(ilast) : 0, npt = (npool + TJ - 1) / TJ;
+  const int tbeg = mask.lowest(ifirst) / TJ, total = npt + ilast / TJ + 1 - tbeg;
+  const int per = (total + splits - 1) / splits;
+  const int u0 = z * per, u1 = min(total, u0 + per);
   for (int idx = tid; idx < R * d; idx += blockDim.x) {
     const int r = idx / d, c = idx - r * d, qi = r / HG, hh = r - qi * HG;
     qs[idx] = qi < nq ? reinterpret_cast<const float*>(o.A)[(size_t)(m0 + qi) * o.lda + (size_t)(g * HG + hh) * d + c] : 0.f;
@@ -1455,21 +1497,24 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_kernel(const fq3c_op o, c
   for (int idx = tid; idx < R; idx += blockDim.x) { mx[idx] = -INFINITY; ls[idx] = 0.f; }
   const TC* kc = reinterpret_cast<const TC*>(o.B) + (size_t)g * d;
   const TC* vc = reinterpret_cast<const TC*>(o.p1) + (size_t)g * dv;
+  const TC* kp = reinterpret_cast<const TC*>(o.C2) + (size_t)g * d;
+  const TC* vp = reinterpret_cast<const TC*>(o.norm_out) + (size_t)g * dv;
   const float* r12 = reinterpret_cast<const float*>(o.bias);
   const float cap = o.f1, icap = o.f1 > 0.f ? 1.f / o.f1 : 0.f;
-  for (int t = t0; t < t1; ++t) {
-    const int j0 = t * TJ, jn = min(TJ, ilast + 1 - j0);
+  for (int u = u0; u < u1; ++u) {
+    const bool pooled = POOL && u < npt;
+    const int j0 = (pooled ? u : tbeg + u - npt) * TJ, jn = min(TJ, (pooled ? npool : ilast + 1) - j0);
     // nothing of this tile is inside the widest window of the block (that of its first query) nor among the kept positions
-    if (mask.window > 0 && j0 + jn <= ifirst - mask.window + 1 && j0 >= mask.keep) continue;
+    if (!pooled && mask.window > 0 && j0 + jn <= ifirst - mask.window + 1 && j0 >= mask.keep) continue;
     if (mask.chunk > 0 && j0 + jn <= ifirst - ifirst % mask.chunk) continue;
     __syncthreads();
-    ca_stage_rows<TC>(kt, d + 1, kc + (size_t)j0 * o.ldr, o.ldr, jn, TJ, d, tid, blockDim.x);
-    ca_stage_rows<TC>(vt, dv, vc + (size_t)j0 * o.taps, o.taps, jn, TJ, dv, tid, blockDim.x);
+    ca_stage_rows<TC>(kt, d + 1, (pooled ? kp : kc) + (size_t)j0 * o.ldr, o.ldr, jn, TJ, d, tid, blockDim.x);
+    ca_stage_rows<TC>(vt, dv, (pooled ? vp : vc) + (size_t)j0 * o.taps, o.taps, jn, TJ, dv, tid, blockDim.x);
     __syncthreads();
     for (int idx = tid; idx < R * TJ; idx += blockDim.x) {
       const int r = idx / TJ, jj = idx - r * TJ, qi = r / HG, i = ifirst + qi, j = j0 + jj;
       float s = -INFINITY;
-      if (qi < nq && jj < jn && mask.sees(i, j)) {
+      if (qi < nq && jj < jn && (pooled ? j < mask.blocks(i) : mask.sees(i, j))) {
         const float* qv = qs + (size_t)r * d;
         const float* kv = kt + (size_t)jj * (d + 1);
         float acc = 0.f;
@@ -1586,7 +1631,7 @@ __device__ __forceinline__ float fast_tanh(float x) {
   return 1.f - __fdividef(2.f, e + 1.f);
 }
 __host__ __device__ inline size_t cache_attn_mma_smem(int rows, int d, int dv) { return 2 * ((size_t)rows * (d + 8) + 2 * (size_t)CM_TJ * (d + 8) + 2 * (size_t)CM_TJ * (dv + 8)); }
-template <int NTM>
+template <int NTM, bool POOL = false>      // POOL: tiles of pooled blocks in front of the tokens' (a variant of its own: the plain one compiles as it always did)
 __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op o, const int ROWS) {
   extern __shared__ __align__(16) unsigned char cm_raw[];
   const int H = o.i0, G = o.i1, d = o.i2, dv = o.cin, HG = H / G, QBLK = ROWS / HG, LDK = d + 8, LDV = dv + 8;
@@ -1598,6 +1643,9 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
   const int P = o.p0 ? *reinterpret_cast<const int*>(o.p0) : 0;
   const int nq = min(QBLK, o.M - m0), ifirst = P + m0, ilast = ifirst + nq - 1;
   const int W = o.K, keep = o.a_rows, chunk = o.tap_off[0];
+  // pooled blocks position i sees, those any query of the block sees, and their tiles (numbered -npt .. -1)
+  auto blocks = [&](const int i) { return POOL ? max(0, i - W + 1) / o.tap_off[1] : 0; };
+  const int npool = blocks(ilast), npt = POOL ? (npool + CM_TJ - 1) / CM_TJ : 0;
   const float* A = reinterpret_cast<const float*>(o.A);
   if (o.lda % 4 == 0 && !(reinterpret_cast<uintptr_t>(A) & 15)) {      // 16-byte loads, four in flight per thread
     const int c4 = d >> 2;
@@ -1617,7 +1665,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
     }
   }
   // the two rows this thread holds of its warp's 16
-  int qpos[2], head[2], clo[2];
+  int qpos[2], head[2], clo[2], nb[2];
   bool live[2];
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -1625,6 +1673,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
     live[e] = qi < nq;
     qpos[e] = ifirst + qi;
     clo[e] = chunk > 0 ? qpos[e] - qpos[e] % chunk : 0;      // first key of the query's chunk
+    nb[e] = blocks(qpos[e]);
     head[e] = kvh * HG + (r - qi * HG);
   }
   const bool wactive = (warp * 16) / HG < nq;
@@ -1632,23 +1681,26 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
   const int ntiles = ilast / CM_TJ + 1;
   const int tkeep = W > 0 ? (keep + CM_TJ - 1) / CM_TJ : 0, tlo = W > 0 ? max(0, ifirst - W + 1) / CM_TJ : 0;
   const int tstart = chunk > 0 ? (ifirst - ifirst % chunk) / CM_TJ : 0;      // tiles below the first query's chunk: nobody sees them
-  auto next_tile = [&](int tt) { ++tt; if (tt < tstart) tt = tstart; if (W > 0 && tt >= tkeep && tt < tlo) tt = tlo; return tt; };
+  auto next_tile = [&](int tt) { ++tt; if (POOL && tt < 0) return tt; if (tt < tstart) tt = tstart; if (W > 0 && tt >= tkeep && tt < tlo) tt = tlo; return tt; };
   const bf16* kc = reinterpret_cast<const bf16*>(o.B) + (size_t)kvh * d;
   const bf16* vc = reinterpret_cast<const bf16*>(o.p1) + (size_t)kvh * dv;
   const int kch = d >> 3, vch = dv >> 3;
   auto fetch_tile = [&](const int tt, const int buf) {       // rows beyond the last needed position arrive as zeros
     bf16* kd = Kt0 + (size_t)buf * CM_TJ * LDK;
     bf16* vd = Vt0 + (size_t)buf * CM_TJ * LDV;
-    const int j0 = tt * CM_TJ;
+    const bool pooled = POOL && tt < 0;
+    const int j0 = (pooled ? tt + npt : tt) * CM_TJ, jend = pooled ? npool - 1 : ilast;
+    const bf16* ks = pooled ? reinterpret_cast<const bf16*>(o.C2) + (size_t)kvh * d : kc;
+    const bf16* vs = pooled ? reinterpret_cast<const bf16*>(o.norm_out) + (size_t)kvh * dv : vc;
     for (int i = tid; i < CM_TJ * kch; i += nth) {
       const int row = i / kch, c = i - row * kch;
-      const bool ok = j0 + row <= ilast;
-      cp_async16(kd + (size_t)row * LDK + c * 8, kc + (size_t)(ok ? j0 + row : 0) * o.ldr + c * 8, ok);
+      const bool ok = j0 + row <= jend;
+      cp_async16(kd + (size_t)row * LDK + c * 8, ks + (size_t)(ok ? j0 + row : 0) * o.ldr + c * 8, ok);
     }
     for (int i = tid; i < CM_TJ * vch; i += nth) {
       const int row = i / vch, c = i - row * vch;
-      const bool ok = j0 + row <= ilast;
-      cp_async16(vd + (size_t)row * LDV + c * 8, vc + (size_t)(ok ? j0 + row : 0) * o.taps + c * 8, ok);
+      const bool ok = j0 + row <= jend;
+      cp_async16(vd + (size_t)row * LDV + c * 8, vs + (size_t)(ok ? j0 + row : 0) * o.taps + c * 8, ok);
     }
     cp_async_commit();
   };
@@ -1662,7 +1714,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
   float r1v[2] = {0.f, 0.f}, r2v[2] = {0.f, 0.f};
   if (r12) { r1v[0] = r12[head[0]]; r1v[1] = r12[head[1]]; r2v[0] = r12[H + head[0]]; r2v[1] = r12[H + head[1]]; }
   const bf16* Qw = Qs + (size_t)warp * 16 * LDK;
-  int tcur = next_tile(-1);
+  int tcur = next_tile(-1 - npt);
   if (tcur < ntiles) fetch_tile(tcur, 0);
   for (int it = 0; tcur < ntiles; ++it) {
     const int tn = next_tile(tcur);
@@ -1673,10 +1725,11 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
       cp_async_wait<0>();
     }
     __syncthreads();
-    const int jt = tcur * CM_TJ;
+    const bool pooled = POOL && tcur < 0;
+    const int jt = (pooled ? tcur + npt : tcur) * CM_TJ;
     const bf16* Kt = Kt0 + (size_t)(it & 1) * CM_TJ * LDK;
     const bf16* Vt = Vt0 + (size_t)(it & 1) * CM_TJ * LDV;
-    if (wactive && jt <= wlast) {
+    if (wactive && (pooled ? jt < blocks(wlast) : jt <= wlast)) {
       float s[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i) { s[i][0] = 0.f; s[i][1] = 0.f; s[i][2] = 0.f; s[i][3] = 0.f; }
@@ -1697,7 +1750,8 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
         }
       }
       // a tile every row of the warp sees whole needs no per-score test (most tiles of a long portion)
-      const bool whole = nq == QBLK && jt + CM_TJ - 1 <= wfirst && (W <= 0 || wlast - jt < W) && (chunk <= 0 || jt >= wlast - wlast % chunk);
+      const bool whole = nq == QBLK && (pooled ? jt + CM_TJ <= blocks(wfirst)
+                                               : jt + CM_TJ - 1 <= wfirst && (W <= 0 || wlast - jt < W) && (chunk <= 0 || jt >= wlast - wlast % chunk));
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
@@ -1705,7 +1759,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
         for (int e = 0; e < 4; ++e) {
           const int key = jt + nt * 8 + t * 2 + (e & 1), hf = e >> 1, i = qpos[hf];
           float v = -INFINITY;
-          if (whole || (live[hf] && key <= i && key >= clo[hf] && (W <= 0 || i - key < W || key < keep))) {
+          if (whole || (live[hf] && (pooled ? key < nb[hf] : key <= i && key >= clo[hf] && (W <= 0 || i - key < W || key < keep)))) {
             v = s[nt][e] * o.f0;
             if (cap > 0.f) v = cap * fast_tanh(v * icap);
             if (r12) v -= r1v[hf] * __logf(fmaf(r2v[hf], (float)(i - key), 1.f));
@@ -1807,11 +1861,17 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
 // product plus three shuffles per reduction; tokens arrive in rounds staged through shared memory.
 // ws row m (padded to a multiple of four floats): [unit q [G * dk] | unit k [G * dk] |] c1[H] | c2[H] [| q.k [G]]  (bracketed parts: delta
 // rule only; delta rule: c1 = decay, c2 = write strength; scan: c1 = decay, c2 = dt)
-// Two more modes share the walk.  Mode 2 (a decay per key channel and token): ws row m = alpha [H * dk], staged beside the token's
+// Four more modes share the walk.  Mode 2 (a decay per key channel and token): ws row m = alpha [H * dk], staged beside the token's
 // key and query as a third vector.  Mode 3 (one fixed decay per head): no per-token coefficients at all, hence no first launch.
+// Mode 4 (a forget gate per channel that also decides what is written): ws row m = silu(q) [H * dk] | 1 - f [H * dk] | f [H * dk], walked
+// like mode 2.  Mode 5 (exponential gates under a running maximum): ws row m = e^(lf + m' - m) [H] | e^(li - m) [H] | e^(-m) [H]; the
+// normaliser is one more state column (index dv) whose value entry is one.
+// Up to MS_CH rows (decoding) the walk forms modes 4 and 5's coefficients itself as it stages the tokens: no first launch.
 // ---------------------------------------------------------------------------------------------------------------------------
 __host__ __device__ inline int mstate_ws_cols(int H, int G, int dk, bool delta) { return ((delta ? 2 * G * dk + G : 0) + 2 * H + 3) & ~3; }
 __host__ __device__ inline int mstate_decay_cols(int H, int dk) { return (H * dk + 3) & ~3; }
+__host__ __device__ inline int mstate_gate_cols(int H, int dk) { return (3 * H * dk + 3) & ~3; }      // mode 4
+__host__ __device__ inline int mstate_max_cols(int H) { return (3 * H + 3) & ~3; }                    // mode 5
 __host__ __device__ inline int mstate_ws_coef(int G, int dk, bool delta) { return delta ? 2 * G * dk : 0; }      // column of c1
 
 constexpr int MS_MAX_RANK = 1024;     // inner size of the decay projection (mode 2)
@@ -1896,6 +1956,68 @@ __global__ void __launch_bounds__(128) fq3s_mstate_prep_kernel(const fq3c_op o) 
 }
 
 constexpr int MS_CH = 16;     // tokens staged per round
+
+// mode 4, one channel: q raw, z the gate's logit, l the lower bound; 1 - f is formed from the mirrored sigmoid, not by a subtraction
+__device__ __forceinline__ void forget_coeffs(const float q, const float z, const float l, float& sq, float& in, float& f) {
+  const float u = 1.f - l;
+  sq = q / (1.f + expf(-q));
+  in = u * sigmoid_f(-z);
+  f = fmaf(u, sigmoid_f(z), l);
+}
+// grid (M, ceil(H * dk / 256)): ws row m of mode 4
+__global__ void __launch_bounds__(256) fq3s_mstate_gate_kernel(const fq3c_op o) {
+  const int m = blockIdx.x, n = o.i0 * o.i2, c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= n) return;
+  const float* raw = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda;
+  float* w = reinterpret_cast<float*>(o.ws) + (size_t)m * mstate_gate_cols(o.i0, o.i2);
+  forget_coeffs(raw[c], raw[o.col_mod + c], reinterpret_cast<const float*>(o.scale)[c], w[c], w[n + c], w[2 * n + c]);
+}
+// mode 5, one token of a head: log input gate and log forget gate from their logits, capped by c tanh(. / c)
+__device__ __forceinline__ void log_gates(const float zi, const float zf, const float cap, float& li, float& lf) {
+  li = cap * tanhf(zi / cap);
+  lf = -softplus_f(-cap * tanhf(zf / cap));
+}
+// grid (H), 256 threads: ws rows of mode 5.  m_t = max(lf_t + m_(t-1), li_t) over a run of tokens is the map m -> max(a + m, b) with
+// a = sum lf and b = the run's own maximum, so every thread folds a share of the rows, the block scans the maps, and every thread walks its
+// share from the maximum it starts with.  The coefficients are differences of the very maxima the walk keeps: whatever the maxima's
+// rounding, numerator, normaliser and e^(-m) refer to the same one.
+__global__ void __launch_bounds__(256) fq3s_mstate_max_kernel(const fq3c_op o) {
+  __shared__ float sa[256], sb[256];
+  const int h = blockIdx.x, H = o.i0, tid = threadIdx.x, per = (o.M + 255) / 256, t0 = min(o.M, tid * per), t1 = min(o.M, t0 + per);
+  const int cols = mstate_max_cols(H);
+  const float* raw = reinterpret_cast<const float*>(o.res);
+  float* w = reinterpret_cast<float*>(o.ws) + h;
+  float a = 0.f, b = -INFINITY;
+  for (int t = t0; t < t1; ++t) {
+    const float* r = raw + (size_t)t * o.ldr + h;
+    float li, lf;
+    log_gates(r[o.col_mod], r[o.m_begin], o.f1, li, lf);
+    float* c = w + (size_t)t * cols;
+    c[0] = lf; c[H] = li;
+    a += lf;
+    b = fmaxf(b + lf, li);
+  }
+  sa[tid] = a; sb[tid] = b;
+  for (int d = 1; d < 256; d <<= 1) {      // inclusive scan of the maps, earlier shares applied first
+    __syncthreads();
+    float pa = 0.f, pb = -INFINITY;
+    if (tid >= d) { pa = sa[tid - d]; pb = sb[tid - d]; }
+    __syncthreads();
+    if (tid >= d) { sb[tid] = fmaxf(sa[tid] + pb, sb[tid]); sa[tid] += pa; }
+  }
+  __syncthreads();
+  float m = reinterpret_cast<const float*>(o.scale)[h];
+  if (tid > 0) m = fmaxf(sa[tid - 1] + m, sb[tid - 1]);
+  for (int t = t0; t < t1; ++t) {
+    float* c = w + (size_t)t * cols;
+    const float lf = c[0], li = c[H], mn = fmaxf(lf + m, li);
+    c[0] = expf(lf + m - mn);
+    c[H] = expf(li - mn);
+    c[2 * H] = expf(-mn);
+    m = mn;
+  }
+  if (t1 == o.M && t0 < t1) reinterpret_cast<float*>(const_cast<void*>(o.p1))[h] = m;
+}
 constexpr int MS_COLS = 16;   // state columns per block (eight lanes each)
 __device__ __forceinline__ void cp_async4(void* dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
@@ -1906,22 +2028,24 @@ __host__ __device__ constexpr int mstate_buf_floats(int rpt, int nv = 2) { retur
 // rows of its state column (RPT * 8 >= dk; rows beyond dk stay zero: their key / query entries are zero padding), reads its slice
 // of the token's key and query with 16-byte shared-memory loads (slices are padded apart by four floats: no bank conflicts),
 // and a product is finished by three shuffles.  The next round's tokens arrive by cp.async while the current round is walked.
-// NV = 3 (mode 2): a third staged vector per token, the decays of the head's key channels.
+// NV = 3 (modes 2 and 4): a third staged vector per token, the decays of the head's key channels.  GATED: modes 4 (NV = 3) and 5 (NV = 2).
 //
-// A long run of rows of a recurrence whose decay does not depend on the state (modes 1-3) is cut into pieces of `piece` rows
+// A long run of rows of a recurrence whose decay does not depend on the state (modes 1-5) is cut into pieces of `piece` rows
 // (grid.z) and walked twice.  phase 1: every piece but the last starts from zero and leaves its own contribution S_loc in
 // X[z + 1] and the product of its decays per state row in P[z]; fq3s_mstate_carry_kernel then turns X into the states the pieces
 // start from (X[0] = the carried state, X[z + 1] = P[z] X[z] + S_loc[z]); phase 3: every piece walks again from X[z] and writes
 // the outputs, the last one also the next state.  phase 0: one pass over all rows (short runs, decoding, the delta rule).
-template <int RPT, int NV = 2>
+template <int RPT, int NV = 2, bool GATED = false>
 __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, const int phase, const int piece, float* X, float* P) {
   extern __shared__ __align__(16) float msm[];
   constexpr int SL = RPT + 4, ROW = 8 * SL;
   const int H = o.i0, G = o.i1, dk = o.i2, dv = o.cin, h = blockIdx.y, g = h / (H / G);
-  const bool delta = o.taps == 0, fixed = o.taps == 3;
-  const int wc = NV == 3 ? mstate_decay_cols(H, dk) : mstate_ws_cols(H, G, dk, delta);
+  const bool delta = o.taps == 0, fixed = o.taps == 3, gates = GATED && NV == 3, memory = GATED && NV == 2;
+  const bool direct = GATED && o.M <= MS_CH;      // the coefficients are formed here
+  const int sv = memory ? dv + 1 : dv;                  // state columns
+  const int wc = NV == 3 ? (gates ? mstate_gate_cols(H, dk) : mstate_decay_cols(H, dk)) : memory ? mstate_max_cols(H) : mstate_ws_cols(H, G, dk, delta);
   const int tid = threadIdx.x, sub = tid & 7, cl = tid >> 3, col = blockIdx.x * MS_COLS + cl;
-  const bool live = col < dv;
+  const bool live = col < sv;
   const int zc = blockIdx.z, tb = phase == 0 ? 0 : zc * piece, te = phase == 0 ? o.M : min(o.M, tb + piece);
   const bool last_piece = phase == 0 || te == o.M;
   constexpr int per = mstate_buf_floats(RPT, NV);
@@ -1933,36 +2057,45 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   float Pd[NV == 3 ? RPT : 1];       // phase 1: the product of the piece's decays (per state row, or one number per head)
 #pragma unroll
   for (int r = 0; r < (NV == 3 ? RPT : 1); ++r) Pd[r] = 1.f;
-  const size_t hstate = (size_t)dk * dv;
+  const size_t hstate = (size_t)dk * sv;
   const float* st = phase == 3 ? X + ((size_t)zc * H + h) * hstate : reinterpret_cast<const float*>(o.p0) + (size_t)h * hstate;
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; S[r] = (phase != 1 && live && i < dk) ? st[(size_t)i * dv + col] : 0.f; }
+  for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; S[r] = (phase != 1 && live && i < dk) ? st[(size_t)i * sv + col] : 0.f; }
   const float D = (o.taps == 1 && o.B) ? reinterpret_cast<const float*>(o.B)[h] : 0.f;
   const float* wsb = reinterpret_cast<const float*>(o.ws);
   const float* rows = reinterpret_cast<const float*>(o.A);
-  const bool qkv_rows = delta || NV == 3 || fixed;       // layout (q | k | v) of the delta rule: queries at column 0, values at a_rows
+  const bool qkv_rows = delta || NV == 3 || fixed || memory;       // layout (q | k | v) of the delta rule: queries at column 0, values at a_rows
   const int vcol = (qkv_rows ? o.a_rows : 0) + h * dv;
   __syncthreads();
   // keys then queries (B then C) of this head's group, as columns of the rows they are staged from
-  const float* vsrc = delta ? wsb : rows;
-  const int vstride = delta ? wc : o.lda, off0 = (delta ? G * dk : o.K) + g * dk, off1 = ((delta || qkv_rows) ? 0 : o.a_rows) + g * dk;
+  const float* vsrc = (delta || gates) ? wsb : rows;
+  const int vstride = (delta || gates) ? wc : o.lda, off0 = ((delta || gates) ? G * dk : o.K) + g * dk, off1 = ((delta || qkv_rows) ? 0 : o.a_rows) + g * dk;
+  const int offa = (gates ? 2 * H * dk : 0) + h * dk;      // the decays' columns (NV == 3)
   const int cfo = mstate_ws_coef(G, dk, delta);
   const bool vec = dk % 4 == 0 && vstride % 4 == 0 && off0 % 4 == 0 && off1 % 4 == 0 && !(reinterpret_cast<uintptr_t>(vsrc) & 15) &&
-                   (NV < 3 || (wc % 4 == 0 && !(reinterpret_cast<uintptr_t>(wsb) & 15)));
+                   (NV < 3 || (wc % 4 == 0 && offa % 4 == 0 && !(reinterpret_cast<uintptr_t>(wsb) & 15)));
   const float fixed_c1 = fixed ? reinterpret_cast<const float*>(o.scale)[h] : 0.f;
   auto fetch = [&](const int t0, float* buf) {
     const int nt = min(MS_CH, te - t0);
     float* kq = buf;
     float* vs = kq + MS_CH * NV * ROW;
     float* cf = vs + MS_CH * MS_COLS;
-    if (vec) {        // 16-byte copies: four consecutive entries never straddle a lane's slice (RPT is a multiple of four)
+    if (NV == 3 && direct) {      // few rows: formed from the raw projections as they are staged
+      const float* low = reinterpret_cast<const float*>(o.scale) + h * dk;
+      for (int idx = tid; idx < nt * dk; idx += 128) {
+        const int tt = idx / dk, c = idx - tt * dk, at = (c / RPT) * SL + (c % RPT);
+        const float* r = rows + (size_t)(t0 + tt) * o.lda + h * dk + c;
+        float* d = kq + tt * NV * ROW + at;
+        forget_coeffs(r[0], r[o.col_mod], low[c], d[ROW], d[0], d[(NV - 1) * ROW]);
+      }
+    } else if (vec) {        // 16-byte copies: four consecutive entries never straddle a lane's slice (RPT is a multiple of four)
       const int n4 = dk >> 2;
       for (int idx = tid; idx < nt * n4; idx += 128) {
         const int tt = idx / n4, c = (idx - tt * n4) * 4, at = (c / RPT) * SL + (c % RPT);
         const float* sr = vsrc + (size_t)(t0 + tt) * vstride;
         cp_async16(kq + tt * NV * ROW + at, sr + off0 + c, true);
         cp_async16(kq + tt * NV * ROW + ROW + at, sr + off1 + c, true);
-        if (NV == 3) cp_async16(kq + tt * NV * ROW + 2 * ROW + at, wsb + (size_t)(t0 + tt) * wc + h * dk + c, true);
+        if (NV == 3) cp_async16(kq + tt * NV * ROW + 2 * ROW + at, wsb + (size_t)(t0 + tt) * wc + offa + c, true);
       }
     } else {
       for (int tt = 0; tt < nt; ++tt) {
@@ -1971,20 +2104,36 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
           const int at = (c / RPT) * SL + (c % RPT);
           cp_async4(kq + tt * NV * ROW + at, sr + off0 + c);
           cp_async4(kq + tt * NV * ROW + ROW + at, sr + off1 + c);
-          if (NV == 3) cp_async4(kq + tt * NV * ROW + 2 * ROW + at, wsb + (size_t)(t0 + tt) * wc + h * dk + c);
+          if (NV == 3) cp_async4(kq + tt * NV * ROW + 2 * ROW + at, wsb + (size_t)(t0 + tt) * wc + offa + c);
         }
       }
     }
     for (int idx = tid; idx < nt * MS_COLS; idx += 128) {
       const int tt = idx / MS_COLS, c = blockIdx.x * MS_COLS + (idx % MS_COLS);
       if (c < dv) cp_async4(vs + idx, rows + (size_t)(t0 + tt) * o.lda + vcol + c);
+      else if (memory && c == dv) vs[idx] = 1.f;
     }
-    if (NV < 3 && !fixed)
+    if (memory && direct) {       // few rows: a lane per token, the running maximum handed from lane to lane
+      if (tid < 32) {
+        float li = 0.f, lf = 0.f, m = reinterpret_cast<const float*>(o.scale)[h], mine = m, next = m;
+        if (tid < nt) {
+          const float* r = reinterpret_cast<const float*>(o.res) + (size_t)(t0 + tid) * o.ldr + h;
+          log_gates(r[o.col_mod], r[o.m_begin], o.f1, li, lf);
+        }
+        for (int tt = 0; tt < nt; ++tt) {
+          const float mn = fmaxf(__shfl_sync(0xffffffffu, lf, tt) + m, __shfl_sync(0xffffffffu, li, tt));
+          if (tt == tid) { mine = m; next = mn; }
+          m = mn;
+        }
+        if (tid < nt) { cf[tid * 4] = expf(lf + mine - next); cf[tid * 4 + 1] = expf(li - next); cf[tid * 4 + 2] = expf(-next); }
+        if (tid == 0 && blockIdx.x == 0) reinterpret_cast<float*>(const_cast<void*>(o.p1))[h] = m;
+      }
+    } else if (NV < 3 && !fixed)
       for (int idx = tid; idx < nt * 3; idx += 128) {
         const int tt = idx / 3, which = idx - tt * 3;
         const float* sr = wsb + (size_t)(t0 + tt) * wc + cfo;
         if (which < 2) cp_async4(cf + tt * 4 + which, sr + which * H + h);
-        else if (delta) cp_async4(cf + tt * 4 + 2, sr + 2 * H + g);
+        else if (delta || memory) cp_async4(cf + tt * 4 + 2, sr + 2 * H + g);
       }
     cp_async_commit();
   };
@@ -2087,6 +2236,13 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
       ot += __shfl_xor_sync(0xffffffffu, ot, 1);
       ot += __shfl_xor_sync(0xffffffffu, ot, 2);
       ot += __shfl_xor_sync(0xffffffffu, ot, 4);
+      if (memory) {
+        ot *= o.f0;
+        if (col == dv && sub == 0)       // the normaliser's column: what the head's read-out is divided by
+          reinterpret_cast<float*>(o.norm_out)[(size_t)(t0 + tt) * o.norm_ld + h] = fmaxf(fabsf(ot), cf[tt * 4 + 2]) + o.norm_eps;
+        if (col < dv && sub == 0) reinterpret_cast<float*>(o.C)[(size_t)(t0 + tt) * o.ldc + (size_t)h * dv + col] = ot;
+        continue;
+      }
       if (!delta) ot = fmaf(D, v, ot);
       if (live && sub == 0) reinterpret_cast<float*>(o.C)[(size_t)(t0 + tt) * o.ldc + (size_t)h * dv + col] = ot;
     }
@@ -2095,7 +2251,7 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   if (phase == 1) {       // this piece's own contribution becomes the next piece's start (after the carry pass); its decay product
     float* nx = X + ((size_t)(zc + 1) * H + h) * hstate;
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live && i < dk) nx[(size_t)i * dv + col] = S[r]; }
+    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live && i < dk) nx[(size_t)i * sv + col] = S[r]; }
     if (blockIdx.x == 0 && cl == 0) {
       float* pz = P + ((size_t)zc * H + h) * dk;
 #pragma unroll
@@ -2106,14 +2262,14 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   if (!last_piece) return;
   float* nst = reinterpret_cast<float*>(o.C2) + (size_t)h * hstate;
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live && i < dk) nst[(size_t)i * dv + col] = S[r]; }
+  for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live && i < dk) nst[(size_t)i * sv + col] = S[r]; }
 }
 
-// grid (ceil(H * dk * dv / 256)): X[0] = the carried state; X[z + 1] = P[z] X[z] + X[z + 1] for the pieces in order.
-__global__ void __launch_bounds__(256) fq3s_mstate_carry_kernel(const fq3c_op o, const int pieces, float* X, const float* P) {
-  const size_t n = (size_t)o.i0 * o.i2 * o.cin, e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+// grid (ceil(H * dk * sv / 256)), sv state columns: X[0] = the carried state; X[z + 1] = P[z] X[z] + X[z + 1] for the pieces in order.
+__global__ void __launch_bounds__(256) fq3s_mstate_carry_kernel(const fq3c_op o, const int pieces, float* X, const float* P, const int sv) {
+  const size_t n = (size_t)o.i0 * o.i2 * sv, e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (e >= n) return;
-  const size_t hi = e / o.cin;        // (head, state row)
+  const size_t hi = e / sv;        // (head, state row)
   float R = reinterpret_cast<const float*>(o.p0)[e];
   X[e] = R;
   for (int z = 0; z + 1 < pieces; ++z) {
@@ -2218,6 +2374,13 @@ __global__ void __launch_bounds__(256) fq3s_sum_norm_kernel(const fq3c_op o) {
     sm += v;
   }
   if (!o.norm_out) return;
+  if (!o.norm_w) {       // no norm: the finished row itself, in the product operands' type
+    for (int i = threadIdx.x; i < o.N; i += blockDim.x) {
+      if (o.flags & FQ3C_F32) reinterpret_cast<float*>(o.norm_out)[(size_t)m * o.norm_ld + i] = snm[i];
+      else reinterpret_cast<bf16*>(o.norm_out)[(size_t)m * o.norm_ld + i] = __float2bfloat16_rn(snm[i]);
+    }
+    return;
+  }
   float mean = 0.f;
   if (o.flags & FQ3C_CENTER) mean = seq_block_sum(sm, red) / (float)o.N;
   float ss = 0.f;

@@ -11,11 +11,13 @@ with its constants as arguments, so another design composes them differently:
   rows and odd shapes), latent_attention (low-rank shared latent cache, absorbed projections, sink softmax; optionally a query
   latent, a rotary key part shared by the heads with a scaled rotary table, a sliding window, an output gate), softmax_attention
   (key / value cache, grouped heads, partial rotary, per-head query / key norms, score cap, window with kept first positions,
-  chunked mask, distance penalty, sink, output gate, borrowed cache), rglru (gated diagonal linear recurrence block), delta_rule and state_space (matrix state per
+  chunked mask, distance penalty, sink, output gate, borrowed cache, pooled blocks before the window), rglru (gated diagonal linear recurrence block), delta_rule and state_space (matrix state per
   head), polynorm_ff, xielu_ff, moe_ff (softmax or sigmoid router with correction, neighbour groups, identity experts, shared
   expert; gelu, relu^2 or gated experts; weights on the experts' outputs or inputs; router bias; gated shared expert), sum_norm (the
   weighted residual sum of sublayers that ran side by side, chained into the next layer norm or RMS norm), channel_decay_attention
-  and retention (linear attentions on the matrix-state scan: a decay per key channel and token, one fixed decay per head).
+  and retention (linear attentions on the matrix-state scan: a decay per key channel and token, one fixed decay per head),
+  forget_gate_attention and matrix_memory (the same scan with gates that also decide what is written, and with exponential gates
+  under a running maximum), gelu_ff.
 
 Precision: `f32=True` runs every product in true 32-bit.  Otherwise weights and product operands are bf16 with f32
 accumulation; the residual stream, norms, softmax, router, recurrence and everything entering it are f32 in both modes.
@@ -27,11 +29,11 @@ from typing import Dict, List, Optional
 import torch
 
 from .codec import (F_A_F32, F_BIAS, F_CENTER, F_SWIGLU, F_F32, F_GATE_POST, F_GATE_PRE, F_GELU, F_NOROUND, F_OUT_F32, F_RAW_WEIGHTS, F_RELU2, F_RESID,
-                    F_ROT_HALF, F_SIGMOID, F_SILU,
+                    F_ROT_HALF, F_SIGMOID, F_SILU, F_UNIT,
                     K_BDGEMM, K_CACHE_ATTN, K_COMMIT, K_DEPTH_MIX, K_DYT, K_EMBED, K_GEMM, K_GGEMM, K_GLU, K_GNORM, K_HYPER, K_LATENT_ATTN,
                     K_LRU_SCAN, K_MOE_COMBINE, K_MOE_SORT, K_MSTATE_SCAN, K_POLYNORM, K_ROT_APPEND, K_ROUTER, K_SUM_NORM, K_TCONV, K_XIELU, Op, _Plan)
-from .config import (ChannelDecayAttentionConfig, DeltaRuleConfig, LatentAttentionConfig, MoEFFConfig, RetentionConfig, RglruConfig,
-                     SoftmaxAttentionConfig, StateSpaceConfig)
+from .config import (ChannelDecayAttentionConfig, DeltaRuleConfig, ForgetGateAttentionConfig, LatentAttentionConfig, MatrixMemoryConfig,
+                     MoEFFConfig, RetentionConfig, RglruConfig, SoftmaxAttentionConfig, StateSpaceConfig)
 from .seq_state import SlotState
 
 
@@ -73,13 +75,18 @@ class StepBuilder:
 
     # ---- mechanisms -----------------------------------------------------------------------------
     def embed(self, ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, rows: Optional[int] = None, scale: float = 0.0,
-              copies: int = 1):
+              copies: int = 1, operand: Optional[torch.Tensor] = None, operand_col: int = 0):
         """out f32 [rows, N] = table[ids] (* scale); also a row gather from an f32 matrix (F_F32).  copies > 1: out is
-        [copies, rows, N] and every slice gets the rows (residual streams that start equal)."""
+        [copies, rows, N] and every slice gets the rows (residual streams that start equal).  operand [rows, ..] of the table's type:
+        the rows also fill its columns from operand_col on, as often as they fit (the operand of a product that reads the embedding)."""
         kw = {}
+        if operand is not None:
+            assert operand.dtype == table.dtype and (operand.shape[1] - operand_col) % table.shape[1] == 0
+            kw.update(C2=_ptr(operand, operand_col), ldr=operand.shape[1], i1=(operand.shape[1] - operand_col) // table.shape[1])
+            self.plan.keep.append(operand)
         if copies > 1:
             assert out.dim() == 3 and out.shape[0] == copies and out.is_contiguous()
-            kw = dict(i0=copies, K=out.shape[1] * out.shape[2])
+            kw.update(i0=copies, K=out.shape[1] * out.shape[2])
         self._op(K_EMBED, M=rows or self.M, N=table.shape[1], A=ids, B=table, C=out, ldc=out.shape[-1], f0=float(scale),
                  flags=F_F32 if table.dtype == torch.float32 else 0, **kw)
         return out
@@ -121,10 +128,12 @@ class StepBuilder:
     def group_norm(self, x: torch.Tensor, w: Optional[torch.Tensor], groups: int, eps: float, out: torch.Tensor, n: Optional[int] = None,
                    col: int = 0, residual: Optional[torch.Tensor] = None, out_bf16: Optional[torch.Tensor] = None,
                    append_at_position: bool = False, gate: Optional[torch.Tensor] = None, gate_col: int = 0, gate_first: bool = False,
-                   weight_period: int = 0, center: bool = False, rows: Optional[int] = None):
+                   weight_period: int = 0, center: bool = False, rows: Optional[int] = None, gate_sigmoid: bool = False,
+                   divisor: Optional[torch.Tensor] = None):
         """out = (residual +) rms_unit_per_group(x) * w.  `gate` (f32 rows, columns from gate_col): the row times silu(gate) before the
         statistics (gate_first) or after the weights.  weight_period > 0: w has that many entries and repeats (a per-head norm).
-        w None: no weights (n required).  center: the statistics are mean and variance (a layer norm without bias)."""
+        w None: no weights (n required).  center: the statistics are mean and variance (a layer norm without bias).  gate_sigmoid: the
+        gate is a sigmoid instead of a silu.  divisor f32 [rows, groups]: a group is divided by its entry first."""
         n = n or w.shape[0]
         kw = dict(M=rows or self.M, N=n, i0=groups, f0=eps, A=_ptr(x, col), lda=x.shape[1], C=out, ldc=out.shape[1], i2=weight_period,
                   flags=self._oflag(out) | (F_RESID if residual is not None else 0) | (F_CENTER if center else 0))
@@ -132,8 +141,10 @@ class StepBuilder:
             kw["scale"] = w
         if gate is not None:
             kw["p1"], kw["i1"] = _ptr(gate, gate_col), gate.shape[1]
-            kw["flags"] |= F_GATE_PRE if gate_first else F_GATE_POST
+            kw["flags"] |= (F_GATE_PRE if gate_first else F_GATE_POST) | (F_SIGMOID if gate_sigmoid else 0)
             self.plan.keep.append(gate)
+        if divisor is not None:
+            kw["bias"], kw["cin"] = divisor, divisor.shape[1]
         if residual is not None:
             kw["res"], kw["ldr"] = residual, residual.shape[1]
         if out_bf16 is not None:
@@ -279,12 +290,15 @@ class StepBuilder:
                  norm_out: Optional[torch.Tensor] = None, eps: float = 0.0, center: bool = False, out: Optional[torch.Tensor] = None):
         """parts f32 [slices, M, N]: out (default parts[0], the residual stream, in place) = sum_(j < count) weights[j] * parts[j],
         weights f32 [count] on the device.  With norm_out: also norm_out = norm(out) * norm_w — RMS, or with `center` mean / variance —
-        in the same launch (the norm that reads the finished stream next)."""
+        in the same launch (the norm that reads the finished stream next); without norm_w norm_out gets the finished row itself (the
+        operand of a product that reads the stream)."""
         out = parts[0] if out is None else out
         kw = dict(M=self.M, N=parts.shape[2], i0=count, K=parts.shape[1] * parts.shape[2], A=parts, lda=parts.shape[2], p0=weights, C=out,
                   ldc=out.shape[1], flags=F_OUT_F32 | (F_CENTER if center else 0))
         if norm_out is not None:
-            kw.update(norm_out=norm_out, norm_w=norm_w, norm_ld=norm_out.shape[1], norm_eps=float(eps))
+            kw.update(norm_out=norm_out, norm_ld=norm_out.shape[1], norm_eps=float(eps))
+            if norm_w is not None:
+                kw["norm_w"] = norm_w
             if norm_out.dtype == torch.float32:
                 kw["flags"] |= F_F32
         self._op(K_SUM_NORM, **kw)
@@ -296,7 +310,8 @@ class StepBuilder:
         """h [M, width] (product-operand dtype) -> out f32 [M, width].  w: wqkv [(H + 2G) dim.. (+ H gate rows), width] — queries, then
         (unless the layer borrows a cache) keys and values, then the gate rows; bqkv f32 or None; freq f32 [rot_dims / 2] or None;
         sink f32 [H] or None; r12 f32 [2H] or None; o [width, H * vdim]; o_b f32 or None; q_norm / k_norm f32 [dim] with qk_norm
-        (eps: their epsilon).  kcache / vcache name the slot's append states to write (own projections) and read."""
+        (eps: their epsilon; qk_unit: no weights).  kcache / vcache name the slot's append states to write (own projections) and read;
+        with pooled blocks (c.pool) kcache + ".pool" and vcache + ".pool" hold one row per complete block."""
         M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
         own = c.kv_from is None
         kcol = H * d
@@ -305,22 +320,28 @@ class StepBuilder:
         proj = self.linear(h, w["wqkv"], self.buf("sa.proj", M, w["wqkv"].shape[0]), bias=w.get("bqkv"))
         kc, vc = self.slot.cur[kcache], self.slot.cur[vcache]
         cf32 = F_F32 if kc.dtype == torch.float32 else 0
-        if own or c.rot_dims > 0 or c.qk_norm:
+        pool = c.pool if c.window > 0 else 0
+        if own or c.rot_dims > 0 or c.qk_norm or c.qk_unit:
             kw = dict(M=M, i0=H, i1=G if own else 0, i2=d, cin=dv, taps=c.rot_dims, K=kcol, a_rows=vcol, A=proj, lda=proj.shape[1],
                       p0=self.slot.pos, flags=cf32)
             if c.rot_dims > 0:
                 kw["B"] = w["freq"]
             if c.qk_norm:   # per-head norms in the same launch, before the rotation
                 kw.update(scale=w["q_norm"], bias=w["k_norm"], f0=float(eps))
+            elif c.qk_unit:
+                kw["f0"] = float(eps)
+                kw["flags"] |= F_UNIT
             if own:
                 kw.update(C=kc, ldc=kc.shape[1], C2=vc, ldr=vc.shape[1])
+                if pool > 0:
+                    kw.update(m_begin=pool, norm_out=self.slot.cur[kcache + ".pool"], ws=self.slot.cur[vcache + ".pool"])
             self._op(K_ROT_APPEND, **kw)
         # key-range splits: many query blocks need none; a few rows (decoding) spread their keys over up to 64 blocks
         HG = H // G
         QB = 1 if M == 1 else max(1, min(16, M, 16 // HG))
         span = self.slot.max_pos        # the most keys a query can see
         if c.window > 0 and c.keep_first == 0:
-            span = min(span, c.window)
+            span = min(span, c.window + (32 + span // pool if pool > 0 else 0))
         if c.chunk > 0:
             span = min(span, c.chunk)
         tiles = max(1, -(-span // 32))
@@ -336,11 +357,13 @@ class StepBuilder:
             kw["bias"] = w["r12"]
         if c.gate:
             kw["res"], kw["col_mod"] = _ptr(proj, gcol), proj.shape[1]
+        if pool > 0:
+            kw["C2"], kw["norm_out"] = self.slot.cur[kcache + ".pool"], self.slot.cur[vcache + ".pool"]
         if splits > 1:
             ws = self.buf("sa.ws", 1, M * H * splits * (dv + 2))
             kw["ws"], kw["ws_bytes"] = ws, ws.numel() * 4
         op = self._op(K_CACHE_ATTN, **kw)
-        op.tap_off[0] = max(c.chunk, 0)
+        op.tap_off[0], op.tap_off[1] = max(c.chunk, 0), pool
         return self.linear(oa, w["o"], out, bias=w.get("o_b"))
 
     # ---- recurrences with a matrix state per head -----------------------------------------------------
@@ -423,6 +446,45 @@ class StepBuilder:
                  ws=ws, ws_bytes=ws.numel() * 4, flags=F_OUT_F32)
         yn = self.group_norm(y, None, H, eps, self.buf("rt.yn", M, H * dv, self.adt), n=H * dv, gate=raw, gate_col=gcol)
         return self.linear(yn, w["o"], out)
+
+    def forget_gate_attention(self, h: torch.Tensor, c: ForgetGateAttentionConfig, w: dict, state: str, eps: float, out: torch.Tensor):
+        """h [M, width] -> out f32 [M, width].  w: win [2 H dim + H vdim (+ padding), width] (q | forget gate | v), bin f32 (its bias: the
+        gate's, zeros elsewhere), lower f32 [H dim], norm f32 [vdim], o [width, H vdim].  Per head, with f = l + (1 - l) sigmoid(gate):
+        S <- diag(f) S + (1 - f) v^T, o = S^T silu(q)."""
+        M, H, d, dv = self.M, c.heads, c.dim, c.vdim
+        raw = self.linear(h, w["win"], self.buf("fg.raw", M, w["win"].shape[0]), bias=w["bin"])
+        y = self.buf("fg.y", M, H * dv)
+        ws = self._scan_ws(-(-(3 * H * d) // 4) * 4, H, d, dv)
+        self._op(K_MSTATE_SCAN, M=M, N=H * dv, taps=4, i0=H, i1=H, i2=d, cin=dv, K=0, a_rows=2 * H * d, A=raw, lda=raw.shape[1], col_mod=H * d,
+                 scale=w["lower"], f0=1.0, p0=self.slot.cur[state], C2=self.slot.next[state], C=y, ldc=y.shape[1], ws=ws, ws_bytes=ws.numel() * 4,
+                 flags=F_OUT_F32)
+        yn = self.group_norm(y, w["norm"], H, eps, self.buf("fg.yn", M, H * dv, self.adt), n=H * dv, weight_period=dv)
+        return self.linear(yn, w["o"], out)
+
+    def matrix_memory(self, h: torch.Tensor, c: MatrixMemoryConfig, w: dict, state: str, eps: float, out: torch.Tensor, floor: float = 1e-6):
+        """h [M, width] -> out f32 [M, width].  w: win [2 H dim + 2 H vdim + 2 H (+ padding), width] (q | k | v | output gate | input gate |
+        forget gate), bin f32 (its bias: the last two's, zeros elsewhere), norm f32 [H vdim], o [width, H vdim].  Per head, under the
+        running maximum m' = max(lf + m, li): S <- e^(lf + m - m') S + e^(li - m') k v^T, n likewise with k alone,
+        o = S^T q / (max(|n . q|, e^(-m')) + floor), q scaled by dim^(-1/2).  States: state + ".s" [H dim, vdim + 1] (the last column is n)
+        and state + ".m" [1, H]."""
+        M, H, d, dv = self.M, c.heads, c.dim, c.vdim
+        gcol = 2 * H * d + H * dv
+        raw = self.linear(h, w["win"], self.buf("mm.raw", M, w["win"].shape[0]), bias=w["bin"])
+        y, den = self.buf("mm.y", M, H * dv), self.buf("mm.den", M, H)
+        ws = self._scan_ws(-(-(3 * H) // 4) * 4, H, d, dv + 1)
+        S, mx = state + ".s", state + ".m"
+        self._op(K_MSTATE_SCAN, M=M, N=H * dv, taps=5, i0=H, i1=H, i2=d, cin=dv, K=H * d, a_rows=2 * H * d, A=raw, lda=raw.shape[1], res=raw,
+                 ldr=raw.shape[1], col_mod=gcol + H * dv, m_begin=gcol + H * dv + H, f0=float(d) ** -0.5, f1=float(c.gate_cap),
+                 scale=self.slot.cur[mx], p1=self.slot.next[mx], norm_out=den, norm_ld=H, norm_eps=float(floor),
+                 p0=self.slot.cur[S], C2=self.slot.next[S], C=y, ldc=y.shape[1], ws=ws, ws_bytes=ws.numel() * 4, flags=F_OUT_F32)
+        yn = self.group_norm(y, w["norm"], H, eps, self.buf("mm.yn", M, H * dv, self.adt), n=H * dv, gate=raw, gate_col=gcol, gate_sigmoid=True,
+                             divisor=den)
+        return self.linear(yn, w["o"], out)
+
+    def gelu_ff(self, x: torch.Tensor, w: dict, out: torch.Tensor):
+        """out f32 = W_down gelu(W_up x) (erf form); w: up [ff, width], down [width, ff].  The activation rides in the first product."""
+        za = self.linear(x, w["up"], self.buf("ff.za", self.M, w["up"].shape[0], self.adt), gelu=True)
+        return self.linear(za, w["down"], out)
 
     def xielu_ff(self, x: torch.Tensor, w: dict, out: torch.Tensor):
         """out f32 = W_down xielu(W_up x); w: up [ff, width], down [width, ff], act f32 [2]."""

@@ -1,7 +1,8 @@
 """Per-sequence state of the sequence models: slots, position counters, caches that grow with the position and fixed-size carries.
 
 A model declares what each of its layers keeps between steps as `StateSpec`s:
-  * kind "append": one row per position (`rows` = capacity in positions): an attention's cached latents / keys / values;
+  * kind "append": one row per position (`rows` = capacity in positions): an attention's cached latents / keys / values; with
+    `every` = P one row per P positions: a reduction over each complete block of P;
   * kind "carry":  a fixed block that a step reads and replaces: the last inputs of a causal convolution, a recurrent state.
 A carry is double-buffered (`cur`, `next`): the step's kernels read `cur` and write `next`, and the step's last op
 (FQ3C_COMMIT, include/fq3_codec.h) copies every `next` to its `cur` and advances the slot's device position counter in one
@@ -24,6 +25,7 @@ class StateSpec:
     cols: int
     rows: int = 1             # carry: rows of the block; append: ignored (capacity comes from the manager)
     dtype: torch.dtype = torch.float32
+    every: int = 1            # append: positions per row
 
 
 class SlotState:
@@ -38,7 +40,7 @@ class SlotState:
         table = []
         for s in specs:
             if s.kind == "append":
-                self.cur[s.name] = torch.zeros(max_pos, s.cols, dtype=s.dtype, device=device)
+                self.cur[s.name] = torch.zeros(max(1, max_pos // s.every), s.cols, dtype=s.dtype, device=device)
             elif s.kind == "carry":
                 if s.rows <= 0:
                     continue
