@@ -1,8 +1,8 @@
 """Throughput of a sequence model at layer sizes that resemble a real model's, beside the closest model of the framework.
 
 `bench.py --seq-model` (the default workload of bench.py is untouched).  Random weights, synthetic tokens.  Sizes w* are Sidalorn
-models, r* Redodra models, z* Ratizen models, u* Zudusun models (`--seq-sizes u1024,z1024,r1024,w1024` puts the designs side by side at
-equal width).  For
+models, r* Redodra models, z* Ratizen models, u* Zudusun models, s* Sirodra models (`--seq-sizes s1024,u1024,z1024,r1024,w1024` puts the
+designs side by side at equal width).  For
 each size:
   * prefill: one step of T prompt tokens through `SequenceEngine.step` (tokens / s), and the same in portions;
   * decode: single-token steps at context T (tokens / s), replayed as CUDA graphs as the generation path does;
@@ -23,9 +23,10 @@ from collections import defaultdict
 import torch
 
 from . import codec as K
-from .config import (ChannelDecayAttentionConfig, DeltaRuleConfig, DenseFFConfig, LatentAttentionConfig, MoEFFConfig, ParallelMixerConfig,
-                     RatizenConfig, RedodraConfig, RetentionConfig, RglruConfig, ScaledPairMixerConfig, SeqLayerConfig, SidalornConfig,
-                     SoftmaxAttentionConfig, StateSpaceConfig, ZudusunConfig)
+from .config import (ChannelDecayAttentionConfig, DeltaRuleConfig, DenseFFConfig, ForgetGateAttentionConfig, LatentAttentionConfig, LoopConfig,
+                     MatrixMemoryConfig, MoEFFConfig, ParallelMixerConfig, RatizenConfig, RedodraConfig, RetentionConfig, RglruConfig,
+                     ScaledPairMixerConfig, SeqLayerConfig, SidalornConfig, SirodraConfig, SoftmaxAttentionConfig, StateSpaceConfig,
+                     ZudusunConfig)
 
 KIND_NAMES = {K.K_GEMM: "gemm (tcgen05 / gemv)", K.K_RMSNORM: "rmsnorm", K.K_ATTN: "attention (prefill, CUDA cores)", 8: "qk-norm + rope + kv",
               K.K_EMBED: "embed / gather", K.K_TCONV: "time conv", K.K_GNORM: "group norm", K.K_BDGEMM: "block-diagonal product",
@@ -89,7 +90,15 @@ def sizes():
         moe = MoEFFConfig(experts, 0, top, 1, 1, 1.0, expert_ff, shared_ff, act="relu2", router_bias=True, shared_gate=True)
         return ZudusunConfig(vocab, width, 1e-5, tuple(SeqLayerConfig(t, mix[t], moe) for t in order), tuple(range(len(order))))
 
-    return {"u1024": zudusun(1024, 16, 4, 8, 16, 2, 768, 1536, ("parallel", "attention", "retention") * 2),
+    def sirodra(width, heads, kv, lin_heads, ff, order, times, window=1024, pool=16, vocab=3072):
+        att = SoftmaxAttentionConfig(heads, kv, 128, 128, 128 ** -0.5, rot_dims=64, rot_base=2e5, window=window, gate=True, bias=True, out_bias=False,
+                                     rot_factor=4.0, qk_unit=True, pool=pool)
+        mix = {"hgrn2": ForgetGateAttentionConfig(lin_heads, 128, 128), "mlstm": MatrixMemoryConfig(lin_heads, 128, 128, 12.0), "attention": att}
+        return SirodraConfig(vocab, width, 1e-5, tuple(SeqLayerConfig(t, mix[t], DenseFFConfig(ff)) for t in order), LoopConfig(0, len(order), times))
+
+    return {"s1024": sirodra(1024, 16, 4, 8, 3072, ("mlstm", "hgrn2", "attention"), 2),
+            "s2048": sirodra(2048, 32, 8, 16, 6144, ("mlstm", "hgrn2", "attention"), 1),
+            "u1024": zudusun(1024, 16, 4, 8, 16, 2, 768, 1536, ("parallel", "attention", "retention") * 2),
             "u2048": zudusun(2048, 32, 8, 16, 32, 4, 1024, 2048, ("parallel", "attention", "retention")),
             "z1024": ratizen(1024, 16, 4, 256, 384, 16, 2, 768, 1536, ("attention", "latent_attention", "latent_attention") * 2),
             "z2048": ratizen(2048, 32, 8, 512, 768, 32, 4, 1024, 2048, ("attention", "latent_attention", "latent_attention")),
@@ -111,6 +120,10 @@ def random_model(cfg, device, seed=0):
         from .zudusun import ZudusunModel, init_synthetic
 
         return ZudusunModel(cfg, init_synthetic(cfg, seed).get, device, f32=False)
+    if isinstance(cfg, SirodraConfig):
+        from .sirodra import SirodraModel, init_synthetic
+
+        return SirodraModel(cfg, init_synthetic(cfg, seed).get, device, f32=False)
     from .sidalorn import SidalornModel, tensor_specs
 
     g = torch.Generator(device=device).manual_seed(seed)
@@ -151,6 +164,8 @@ def op_cost(o, ctx_keys: float):
         return 0.0, M * N * (4 * 4 + outs)
     if k == K.K_CACHE_ATTN:
         keys = min(ctx_keys, o.K + o.a_rows) if o.K > 0 else ctx_keys
+        if o.tap_off[1] > 0:
+            keys += max(0.0, ctx_keys - o.K) / o.tap_off[1]                 # pooled blocks in front of the window
         if o.tap_off[0] > 0:
             keys = min(keys, (o.tap_off[0] + 1) / 2.0)                      # chunked mask: half a chunk on average
         return 2.0 * M * o.i0 * (o.i2 + o.cin) * keys, min(ctx_keys + M / 2, keys + M) * o.i1 * (o.i2 + o.cin) * ws + M * o.i0 * (o.i2 * 4 + o.cin * outs)
@@ -238,7 +253,8 @@ def bench_sequence_model(name, cfg, T, device):
     g = torch.Generator().manual_seed(1)
     toks = torch.randint(0, cfg.vocab, (T + 40,), generator=g).tolist()
     flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
-    out = {"model": f"{cfg.architecture} {name}", "width": cfg.width, "layers": len(cfg.layers), "T": T}
+    runs = len(cfg.runs) if isinstance(cfg, SirodraConfig) else len(cfg.layers)      # layer runs: a looped layer counts each time
+    out = {"model": f"{cfg.architecture} {name}", "width": cfg.width, "layers": runs, "T": T}
 
     def prefill(portion):
         def run():
@@ -270,7 +286,12 @@ def bench_sequence_model(name, cfg, T, device):
         return v.numel() * v.element_size() if isinstance(v, torch.Tensor) and v.dtype == torch.bfloat16 else 0
 
     wb = 0
+    if isinstance(cfg, SirodraConfig):          # every layer run reads its layer's tensors, every pass the product in front of it
+        for i, first in cfg.runs:
+            wb += operand_bytes(model.layers[i]) + (operand_bytes(model.g["loop.in"]) if first else 0)
     for i, (L, w) in enumerate(zip(cfg.layers, model.layers)):
+        if isinstance(cfg, SirodraConfig):
+            break
         if isinstance(cfg, RedodraConfig):
             wb += operand_bytes(w)
             continue
