@@ -1234,7 +1234,8 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       if (o.i0 < 1 || o.i1 < 1 || o.i0 % o.i1 || o.i2 < 1 || o.cin < 1 || !o.A || !o.B || !o.p1 || !o.C) return fail("cache_attn: bad configuration");
       const int splits = std::max(1, o.m_begin), HG = o.i0 / o.i1;
       const bool pool = o.tap_off[1] > 0;
-      if (pool && (o.K < 1 || !o.C2 || !o.norm_out || o.bias || o.tap_off[0] > 0)) return fail("cache_attn: pooled blocks go with a window and their pooled rows, not with a chunked mask or a distance penalty");
+      if (pool && (o.K < 1 || !o.C2 || !o.norm_out || o.bias || o.tap_off[0] > 0 || o.a_rows > 0))
+        return fail("cache_attn: pooled blocks go with a window and their pooled rows, not with kept first positions, a chunked mask or a distance penalty");
       if (splits > 64) return fail("cache_attn: at most 64 key splits");
       if (splits > 1 && (!o.ws || o.ws_bytes < (int64_t)o.M * o.i0 * splits * (o.cin + 2) * 4)) return fail("cache_attn: workspace too small for the splits");
       // bf16 cache and a prompt portion: the tensor-core kernel (FQ3S_ATTN_MMA=0: CUDA cores everywhere)
@@ -1343,7 +1344,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         fq3s_mstate_gate_kernel<<<dim3(o.M, (o.i0 * o.i2 + 255) / 256), 256, 0, s>>>(o);
         count_launches(1);
       } else if (o.taps == 5 && o.M > MS_CH) {
-        fq3s_mstate_max_kernel<<<o.i0, 256, 0, s>>>(o);
+        fq3s_mstate_max_kernel<<<o.i0, MM_THREADS, 0, s>>>(o);
         count_launches(1);
       } else if (o.taps < 3) {
         fq3s_mstate_prep_kernel<<<o.taps == 2 ? (o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS : o.M, 128, 0, s>>>(o);
@@ -1383,20 +1384,29 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       }
       float* X = pieces > 1 ? reinterpret_cast<float*>(o.ws) + base : nullptr;
       float* P = pieces > 1 ? X + (int64_t)pieces * o.i0 * o.i2 * sv : nullptr;
-      const dim3 tiles((sv + MS_COLS - 1) / MS_COLS, o.i0);
       const int bound = o.i2 <= 32 ? 4 : o.i2 <= 64 ? 8 : o.i2 <= 128 ? 16 : o.i2 <= 256 ? 32 : 64;      // state rows a lane holds
       const bool three = o.taps == 2 || o.taps == 4, gated = o.taps >= 4;
+      const int cpt = pieces > 1 && bound <= 16 ? 2 : 1;                                                    // state columns a lane holds
       auto walk = [&](const int phase, const int nz) {
-        const dim3 grid(tiles.x, tiles.y, nz);
-        const size_t smem = sizeof(float) * 2 * mstate_buf_floats(bound, three ? 3 : 2);
-#define FQ3S_WALK(RPT) \
-  case RPT: \
-    if (three && gated) fq3s_mstate_scan_kernel<RPT, 3, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
-    else if (three) fq3s_mstate_scan_kernel<RPT, 3><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
-    else if (gated) fq3s_mstate_scan_kernel<RPT, 2, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
-    else fq3s_mstate_scan_kernel<RPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
-    break;
-        switch (bound) { FQ3S_WALK(4) FQ3S_WALK(8) FQ3S_WALK(16) FQ3S_WALK(32) FQ3S_WALK(64) }
+        const dim3 grid((sv + cpt * MS_COLS - 1) / (cpt * MS_COLS), o.i0, nz);
+        const size_t smem = sizeof(float) * 2 * mstate_buf_floats(bound, three ? 3 : 2, cpt);
+#define FQ3S_WALK(RPT, CPT) \
+    if (three && gated) fq3s_mstate_scan_kernel<RPT, 3, true, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    else if (three) fq3s_mstate_scan_kernel<RPT, 3, false, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    else if (gated) fq3s_mstate_scan_kernel<RPT, 2, true, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
+    else fq3s_mstate_scan_kernel<RPT, 2, false, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P);
+        if (cpt == 2) switch (bound) {
+          case 4: FQ3S_WALK(4, 2) break;
+          case 8: FQ3S_WALK(8, 2) break;
+          default: FQ3S_WALK(16, 2) break;
+        }
+        else switch (bound) {
+          case 4: FQ3S_WALK(4, 1) break;
+          case 8: FQ3S_WALK(8, 1) break;
+          case 16: FQ3S_WALK(16, 1) break;
+          case 32: FQ3S_WALK(32, 1) break;
+          default: FQ3S_WALK(64, 1) break;
+        }
 #undef FQ3S_WALK
       };
       if (pieces == 1) {

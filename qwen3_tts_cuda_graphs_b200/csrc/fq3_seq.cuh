@@ -1646,6 +1646,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
   // pooled blocks position i sees, those any query of the block sees, and their tiles (numbered -npt .. -1)
   auto blocks = [&](const int i) { return POOL ? max(0, i - W + 1) / o.tap_off[1] : 0; };
   const int npool = blocks(ilast), npt = POOL ? (npool + CM_TJ - 1) / CM_TJ : 0;
+  int nb[2] = {0, 0}, wblocks[2] = {0, 0};      // blocks this thread's two rows see; the first and the last row of its warp
   const float* A = reinterpret_cast<const float*>(o.A);
   if (o.lda % 4 == 0 && !(reinterpret_cast<uintptr_t>(A) & 15)) {      // 16-byte loads, four in flight per thread
     const int c4 = d >> 2;
@@ -1665,7 +1666,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
     }
   }
   // the two rows this thread holds of its warp's 16
-  int qpos[2], head[2], clo[2], nb[2];
+  int qpos[2], head[2], clo[2];
   bool live[2];
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -1673,7 +1674,6 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
     live[e] = qi < nq;
     qpos[e] = ifirst + qi;
     clo[e] = chunk > 0 ? qpos[e] - qpos[e] % chunk : 0;      // first key of the query's chunk
-    nb[e] = blocks(qpos[e]);
     head[e] = kvh * HG + (r - qi * HG);
   }
   const bool wactive = (warp * 16) / HG < nq;
@@ -1681,6 +1681,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
   const int ntiles = ilast / CM_TJ + 1;
   const int tkeep = W > 0 ? (keep + CM_TJ - 1) / CM_TJ : 0, tlo = W > 0 ? max(0, ifirst - W + 1) / CM_TJ : 0;
   const int tstart = chunk > 0 ? (ifirst - ifirst % chunk) / CM_TJ : 0;      // tiles below the first query's chunk: nobody sees them
+  if (POOL) { nb[0] = live[0] ? blocks(qpos[0]) : 0; nb[1] = live[1] ? blocks(qpos[1]) : 0; wblocks[0] = blocks(wfirst); wblocks[1] = blocks(wlast); }
   auto next_tile = [&](int tt) { ++tt; if (POOL && tt < 0) return tt; if (tt < tstart) tt = tstart; if (W > 0 && tt >= tkeep && tt < tlo) tt = tlo; return tt; };
   const bf16* kc = reinterpret_cast<const bf16*>(o.B) + (size_t)kvh * d;
   const bf16* vc = reinterpret_cast<const bf16*>(o.p1) + (size_t)kvh * dv;
@@ -1729,7 +1730,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
     const int jt = (pooled ? tcur + npt : tcur) * CM_TJ;
     const bf16* Kt = Kt0 + (size_t)(it & 1) * CM_TJ * LDK;
     const bf16* Vt = Vt0 + (size_t)(it & 1) * CM_TJ * LDV;
-    if (wactive && (pooled ? jt < blocks(wlast) : jt <= wlast)) {
+    if (wactive && (pooled ? jt < wblocks[1] : jt <= wlast)) {
       float s[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i) { s[i][0] = 0.f; s[i][1] = 0.f; s[i][2] = 0.f; s[i][3] = 0.f; }
@@ -1750,8 +1751,16 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
         }
       }
       // a tile every row of the warp sees whole needs no per-score test (most tiles of a long portion)
-      const bool whole = nq == QBLK && (pooled ? jt + CM_TJ <= blocks(wfirst)
+      const bool whole = nq == QBLK && (pooled ? jt + CM_TJ <= wblocks[0]
                                                : jt + CM_TJ - 1 <= wfirst && (W <= 0 || wlast - jt < W) && (chunk <= 0 || jt >= wlast - wlast % chunk));
+      int lo[2], hi[2];      // POOL: the keys of this tile each of the two rows sees lie in [lo, hi)
+      if (POOL) {
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          lo[hf] = (pooled ? 0 : qpos[hf] - W + 1) - jt - t * 2;
+          hi[hf] = (pooled ? nb[hf] : live[hf] ? qpos[hf] + 1 : 0) - jt - t * 2;
+        }
+      }
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
@@ -1759,7 +1768,13 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
         for (int e = 0; e < 4; ++e) {
           const int key = jt + nt * 8 + t * 2 + (e & 1), hf = e >> 1, i = qpos[hf];
           float v = -INFINITY;
-          if (whole || (live[hf] && (pooled ? key < nb[hf] : key <= i && key >= clo[hf] && (W <= 0 || i - key < W || key < keep)))) {
+          if (POOL) {
+            const int at = nt * 8 + (e & 1);
+            if (whole || (at >= lo[hf] && at < hi[hf])) {
+              v = s[nt][e] * o.f0;
+              if (cap > 0.f) v = cap * fast_tanh(v * icap);
+            }
+          } else if (whole || (live[hf] && key <= i && key >= clo[hf] && (W <= 0 || i - key < W || key < keep))) {
             v = s[nt][e] * o.f0;
             if (cap > 0.f) v = cap * fast_tanh(v * icap);
             if (r12) v -= r1v[hf] * __logf(fmaf(r2v[hf], (float)(i - key), 1.f));
@@ -1977,28 +1992,38 @@ __device__ __forceinline__ void log_gates(const float zi, const float zf, const 
   li = cap * tanhf(zi / cap);
   lf = -softplus_f(-cap * tanhf(zf / cap));
 }
-// grid (H), 256 threads: ws rows of mode 5.  m_t = max(lf_t + m_(t-1), li_t) over a run of tokens is the map m -> max(a + m, b) with
+// grid (H), MM_THREADS threads: ws rows of mode 5.  m_t = max(lf_t + m_(t-1), li_t) over a run of tokens is the map m -> max(a + m, b) with
 // a = sum lf and b = the run's own maximum, so every thread folds a share of the rows, the block scans the maps, and every thread walks its
 // share from the maximum it starts with.  The coefficients are differences of the very maxima the walk keeps: whatever the maxima's
-// rounding, numerator, normaliser and e^(-m) refer to the same one.
-__global__ void __launch_bounds__(256) fq3s_mstate_max_kernel(const fq3c_op o) {
-  __shared__ float sa[256], sb[256];
-  const int h = blockIdx.x, H = o.i0, tid = threadIdx.x, per = (o.M + 255) / 256, t0 = min(o.M, tid * per), t1 = min(o.M, t0 + per);
+// rounding, numerator, normaliser and e^(-m) refer to the same one.  Rows are fetched MM_BATCH at a time, ahead of the stores.
+constexpr int MM_THREADS = 512, MM_BATCH = 4;
+__global__ void __launch_bounds__(MM_THREADS) fq3s_mstate_max_kernel(const fq3c_op o) {
+  __shared__ float sa[MM_THREADS], sb[MM_THREADS];
+  const int h = blockIdx.x, H = o.i0, tid = threadIdx.x, per = (o.M + MM_THREADS - 1) / MM_THREADS, t0 = min(o.M, tid * per), t1 = min(o.M, t0 + per);
   const int cols = mstate_max_cols(H);
-  const float* raw = reinterpret_cast<const float*>(o.res);
+  const float* raw = reinterpret_cast<const float*>(o.res) + h;
   float* w = reinterpret_cast<float*>(o.ws) + h;
   float a = 0.f, b = -INFINITY;
-  for (int t = t0; t < t1; ++t) {
-    const float* r = raw + (size_t)t * o.ldr + h;
-    float li, lf;
-    log_gates(r[o.col_mod], r[o.m_begin], o.f1, li, lf);
-    float* c = w + (size_t)t * cols;
-    c[0] = lf; c[H] = li;
-    a += lf;
-    b = fmaxf(b + lf, li);
+  for (int t = t0; t < t1; t += MM_BATCH) {
+    float li[MM_BATCH], lf[MM_BATCH];
+#pragma unroll
+    for (int q = 0; q < MM_BATCH; ++q) {
+      const float* r = raw + (size_t)min(t + q, t1 - 1) * o.ldr;
+      li[q] = __ldg(r + o.col_mod);
+      lf[q] = __ldg(r + o.m_begin);
+    }
+#pragma unroll
+    for (int q = 0; q < MM_BATCH; ++q) {
+      if (t + q >= t1) break;
+      log_gates(li[q], lf[q], o.f1, li[q], lf[q]);
+      float* c = w + (size_t)(t + q) * cols;
+      c[0] = lf[q]; c[H] = li[q];
+      a += lf[q];
+      b = fmaxf(b + lf[q], li[q]);
+    }
   }
   sa[tid] = a; sb[tid] = b;
-  for (int d = 1; d < 256; d <<= 1) {      // inclusive scan of the maps, earlier shares applied first
+  for (int d = 1; d < MM_THREADS; d <<= 1) {      // inclusive scan of the maps, earlier shares applied first
     __syncthreads();
     float pa = 0.f, pb = -INFINITY;
     if (tid >= d) { pa = sa[tid - d]; pb = sb[tid - d]; }
@@ -2008,22 +2033,35 @@ __global__ void __launch_bounds__(256) fq3s_mstate_max_kernel(const fq3c_op o) {
   __syncthreads();
   float m = reinterpret_cast<const float*>(o.scale)[h];
   if (tid > 0) m = fmaxf(sa[tid - 1] + m, sb[tid - 1]);
-  for (int t = t0; t < t1; ++t) {
-    float* c = w + (size_t)t * cols;
-    const float lf = c[0], li = c[H], mn = fmaxf(lf + m, li);
-    c[0] = expf(lf + m - mn);
-    c[H] = expf(li - mn);
-    c[2 * H] = expf(-mn);
-    m = mn;
+  for (int t = t0; t < t1; t += MM_BATCH) {
+    float li[MM_BATCH], lf[MM_BATCH];
+#pragma unroll
+    for (int q = 0; q < MM_BATCH; ++q) {
+      const float* c = w + (size_t)min(t + q, t1 - 1) * cols;
+      lf[q] = c[0]; li[q] = c[H];
+    }
+#pragma unroll
+    for (int q = 0; q < MM_BATCH; ++q) {
+      if (t + q >= t1) break;
+      float* c = w + (size_t)(t + q) * cols;
+      const float mn = fmaxf(lf[q] + m, li[q]);
+      c[0] = expf(lf[q] + m - mn);
+      c[H] = expf(li[q] - mn);
+      c[2 * H] = expf(-mn);
+      m = mn;
+    }
   }
   if (t1 == o.M && t0 < t1) reinterpret_cast<float*>(const_cast<void*>(o.p1))[h] = m;
 }
-constexpr int MS_COLS = 16;   // state columns per block (eight lanes each)
+constexpr int MS_COLS = 16;   // state columns per block (eight lanes each), times the columns a lane holds
 __device__ __forceinline__ void cp_async4(void* dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
-// floats per staging buffer: (k, q) or (B, C) (and the decays) [MS_CH][NV][8 slices of RPT + 4] | v [MS_CH][MS_COLS] | coefficients [MS_CH][4]
-__host__ __device__ constexpr int mstate_buf_floats(int rpt, int nv = 2) { return MS_CH * nv * 8 * (rpt + 4) + MS_CH * MS_COLS + MS_CH * 4; }
+// floats per staging buffer: (k, q) or (B, C) (and the decays) [CH][NV][8 slices of RPT + 4] | v [CH][columns] | coefficients [CH][4]
+__host__ __device__ constexpr int mstate_ch(int cpt) { return MS_CH / cpt; }
+__host__ __device__ constexpr int mstate_buf_floats(int rpt, int nv = 2, int cpt = 1) {
+  return mstate_ch(cpt) * (nv * 8 * (rpt + 4) + MS_COLS * cpt + 4);
+}
 // grid (ceil(dv / 16), H), 128 threads: thread = (column tid / 8 of the tile, lane-of-eight tid % 8).  A lane holds RPT consecutive
 // rows of its state column (RPT * 8 >= dk; rows beyond dk stay zero: their key / query entries are zero padding), reads its slice
 // of the token's key and query with 16-byte shared-memory loads (slices are padded apart by four floats: no bank conflicts),
@@ -2035,32 +2073,42 @@ __host__ __device__ constexpr int mstate_buf_floats(int rpt, int nv = 2) { retur
 // X[z + 1] and the product of its decays per state row in P[z]; fq3s_mstate_carry_kernel then turns X into the states the pieces
 // start from (X[0] = the carried state, X[z + 1] = P[z] X[z] + S_loc[z]); phase 3: every piece walks again from X[z] and writes
 // the outputs, the last one also the next state.  phase 0: one pass over all rows (short runs, decoding, the delta rule).
-template <int RPT, int NV = 2, bool GATED = false>
+//
+// CPT = 2 (pieces of long runs, where blocks are plenty): a lane holds two state columns, so a token's vectors are read from shared memory
+// once for both; rounds of eight tokens keep the blocks small.  Warps without a live column only stage.
+template <int RPT, int NV = 2, bool GATED = false, int CPT = 1>
 __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, const int phase, const int piece, float* X, float* P) {
   extern __shared__ __align__(16) float msm[];
-  constexpr int SL = RPT + 4, ROW = 8 * SL;
+  constexpr int SL = RPT + 4, ROW = 8 * SL, CH = mstate_ch(CPT), COLS = MS_COLS * CPT;
   const int H = o.i0, G = o.i1, dk = o.i2, dv = o.cin, h = blockIdx.y, g = h / (H / G);
-  const bool delta = o.taps == 0, fixed = o.taps == 3, gates = GATED && NV == 3, memory = GATED && NV == 2;
+  const bool delta = !GATED && NV == 2 && CPT == 1 && o.taps == 0, fixed = !GATED && NV == 2 && o.taps == 3;
+  const bool gates = GATED && NV == 3, memory = GATED && NV == 2;
   const bool direct = GATED && o.M <= MS_CH;      // the coefficients are formed here
   const int sv = memory ? dv + 1 : dv;                  // state columns
   const int wc = NV == 3 ? (gates ? mstate_gate_cols(H, dk) : mstate_decay_cols(H, dk)) : memory ? mstate_max_cols(H) : mstate_ws_cols(H, G, dk, delta);
-  const int tid = threadIdx.x, sub = tid & 7, cl = tid >> 3, col = blockIdx.x * MS_COLS + cl;
-  const bool live = col < sv;
+  const int tid = threadIdx.x, sub = tid & 7, cl = tid >> 3;      // this lane's columns: blockIdx.x * COLS + cl (+ MS_COLS)
+  const bool wlive = blockIdx.x * COLS + (cl & ~3) < sv;           // the warp (four neighbouring columns) has one
+  int col[CPT];
+  bool live[CPT];
+#pragma unroll
+  for (int j = 0; j < CPT; ++j) { col[j] = blockIdx.x * COLS + cl + j * MS_COLS; live[j] = col[j] < sv; }
   const int zc = blockIdx.z, tb = phase == 0 ? 0 : zc * piece, te = phase == 0 ? o.M : min(o.M, tb + piece);
   const bool last_piece = phase == 0 || te == o.M;
-  constexpr int per = mstate_buf_floats(RPT, NV);
+  constexpr int per = mstate_buf_floats(RPT, NV, CPT);
   {   // the padding between and behind the slices stays zero for the whole launch (only the token rows that will be used)
-    const int used = min(te - tb, MS_CH) * NV * ROW;
+    const int used = min(te - tb, CH) * NV * ROW;
     for (int i = tid; i < 2 * used; i += 128) msm[(i < used ? 0 : per - used) + i] = 0.f;
   }
-  float S[RPT];
+  float S[CPT][RPT];
   float Pd[NV == 3 ? RPT : 1];       // phase 1: the product of the piece's decays (per state row, or one number per head)
 #pragma unroll
   for (int r = 0; r < (NV == 3 ? RPT : 1); ++r) Pd[r] = 1.f;
   const size_t hstate = (size_t)dk * sv;
   const float* st = phase == 3 ? X + ((size_t)zc * H + h) * hstate : reinterpret_cast<const float*>(o.p0) + (size_t)h * hstate;
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; S[r] = (phase != 1 && live && i < dk) ? st[(size_t)i * sv + col] : 0.f; }
+  for (int j = 0; j < CPT; ++j)
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; S[j][r] = (phase != 1 && live[j] && i < dk) ? st[(size_t)i * sv + col[j]] : 0.f; }
   const float D = (o.taps == 1 && o.B) ? reinterpret_cast<const float*>(o.B)[h] : 0.f;
   const float* wsb = reinterpret_cast<const float*>(o.ws);
   const float* rows = reinterpret_cast<const float*>(o.A);
@@ -2076,10 +2124,10 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
                    (NV < 3 || (wc % 4 == 0 && offa % 4 == 0 && !(reinterpret_cast<uintptr_t>(wsb) & 15)));
   const float fixed_c1 = fixed ? reinterpret_cast<const float*>(o.scale)[h] : 0.f;
   auto fetch = [&](const int t0, float* buf) {
-    const int nt = min(MS_CH, te - t0);
+    const int nt = min(CH, te - t0);
     float* kq = buf;
-    float* vs = kq + MS_CH * NV * ROW;
-    float* cf = vs + MS_CH * MS_COLS;
+    float* vs = kq + CH * NV * ROW;
+    float* cf = vs + CH * COLS;
     if (NV == 3 && direct) {      // few rows: formed from the raw projections as they are staged
       const float* low = reinterpret_cast<const float*>(o.scale) + h * dk;
       for (int idx = tid; idx < nt * dk; idx += 128) {
@@ -2108,8 +2156,8 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
         }
       }
     }
-    for (int idx = tid; idx < nt * MS_COLS; idx += 128) {
-      const int tt = idx / MS_COLS, c = blockIdx.x * MS_COLS + (idx % MS_COLS);
+    for (int idx = tid; idx < nt * COLS; idx += 128) {
+      const int tt = idx / COLS, c = blockIdx.x * COLS + (idx % COLS);
       if (c < dv) cp_async4(vs + idx, rows + (size_t)(t0 + tt) * o.lda + vcol + c);
       else if (memory && c == dv) vs[idx] = 1.f;
     }
@@ -2139,31 +2187,45 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   };
   fetch(tb, msm);
   int it = 0;
-  for (int t0 = tb; t0 < te; t0 += MS_CH, ++it) {
-    const int nt = min(MS_CH, te - t0);
-    if (t0 + MS_CH < te) {
-      fetch(t0 + MS_CH, msm + ((it + 1) & 1) * per);
+  for (int t0 = tb; t0 < te; t0 += CH, ++it) {
+    const int nt = min(CH, te - t0);
+    if (t0 + CH < te) {
+      fetch(t0 + CH, msm + ((it + 1) & 1) * per);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();
     const float* kq = msm + (it & 1) * per;
-    const float* vs = kq + MS_CH * NV * ROW;
-    const float* cf = vs + MS_CH * MS_COLS;
-    for (int tt = 0; tt < nt; ++tt) {
+    const float* vs = kq + CH * NV * ROW;
+    const float* cf = vs + CH * COLS;
+    for (int tt = 0; tt < (wlive ? nt : 0); ++tt) {
       const float4* k4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + sub * SL);
       const float4* q4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + ROW + sub * SL);
-      const float v = vs[tt * MS_COLS + cl];
-      float os[4] = {0.f, 0.f, 0.f, 0.f};       // four chains, so that a product's sum is not one long dependent row of multiply-adds
+      float v[CPT];
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) v[j] = vs[tt * COLS + cl + j * MS_COLS];
+      float os[CPT][4] = {};       // four chains, so that a product's sum is not one long dependent row of multiply-adds
+      // a finished product: its four chains, then the eight lanes of the column
+      auto total = [&](const float (&c)[4]) {
+        float x = (c[0] + c[1]) + (c[2] + c[3]);
+        x += __shfl_xor_sync(0xffffffffu, x, 1);
+        x += __shfl_xor_sync(0xffffffffu, x, 2);
+        x += __shfl_xor_sync(0xffffffffu, x, 4);
+        return x;
+      };
+      float* orow = reinterpret_cast<float*>(o.C) + (size_t)(t0 + tt) * o.ldc + (size_t)h * dv;
       if (NV == 3) {      // S <- diag(alpha) S + k v^T, o = f0 S^T q
         const float4* a4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + 2 * ROW + sub * SL);
         if (phase == 1) {
 #pragma unroll
           for (int r = 0; r < RPT / 4; ++r) {
             const float4 kv = k4[r], av = a4[r];
-            S[4 * r] = fmaf(av.x, S[4 * r], kv.x * v); S[4 * r + 1] = fmaf(av.y, S[4 * r + 1], kv.y * v);
-            S[4 * r + 2] = fmaf(av.z, S[4 * r + 2], kv.z * v); S[4 * r + 3] = fmaf(av.w, S[4 * r + 3], kv.w * v);
+#pragma unroll
+            for (int j = 0; j < CPT; ++j) {
+              S[j][4 * r] = fmaf(av.x, S[j][4 * r], kv.x * v[j]); S[j][4 * r + 1] = fmaf(av.y, S[j][4 * r + 1], kv.y * v[j]);
+              S[j][4 * r + 2] = fmaf(av.z, S[j][4 * r + 2], kv.z * v[j]); S[j][4 * r + 3] = fmaf(av.w, S[j][4 * r + 3], kv.w * v[j]);
+            }
             constexpr int PR = NV == 3 ? 1 : 0;     // (this branch only runs with NV == 3; the index stays legal in the other instantiation)
             Pd[PR * (4 * r)] *= av.x; Pd[PR * (4 * r + 1)] *= av.y; Pd[PR * (4 * r + 2)] *= av.z; Pd[PR * (4 * r + 3)] *= av.w;
           }
@@ -2172,86 +2234,101 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
 #pragma unroll
         for (int r = 0; r < RPT / 4; ++r) {
           const float4 kv = k4[r], qv = q4[r], av = a4[r];
-          S[4 * r] = fmaf(av.x, S[4 * r], kv.x * v); S[4 * r + 1] = fmaf(av.y, S[4 * r + 1], kv.y * v);
-          S[4 * r + 2] = fmaf(av.z, S[4 * r + 2], kv.z * v); S[4 * r + 3] = fmaf(av.w, S[4 * r + 3], kv.w * v);
-          os[0] = fmaf(qv.x, S[4 * r], os[0]); os[1] = fmaf(qv.y, S[4 * r + 1], os[1]);
-          os[2] = fmaf(qv.z, S[4 * r + 2], os[2]); os[3] = fmaf(qv.w, S[4 * r + 3], os[3]);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            S[j][4 * r] = fmaf(av.x, S[j][4 * r], kv.x * v[j]); S[j][4 * r + 1] = fmaf(av.y, S[j][4 * r + 1], kv.y * v[j]);
+            S[j][4 * r + 2] = fmaf(av.z, S[j][4 * r + 2], kv.z * v[j]); S[j][4 * r + 3] = fmaf(av.w, S[j][4 * r + 3], kv.w * v[j]);
+            os[j][0] = fmaf(qv.x, S[j][4 * r], os[j][0]); os[j][1] = fmaf(qv.y, S[j][4 * r + 1], os[j][1]);
+            os[j][2] = fmaf(qv.z, S[j][4 * r + 2], os[j][2]); os[j][3] = fmaf(qv.w, S[j][4 * r + 3], os[j][3]);
+          }
         }
-        float ot = (os[0] + os[1]) + (os[2] + os[3]);
-        ot += __shfl_xor_sync(0xffffffffu, ot, 1);
-        ot += __shfl_xor_sync(0xffffffffu, ot, 2);
-        ot += __shfl_xor_sync(0xffffffffu, ot, 4);
-        if (live && sub == 0) reinterpret_cast<float*>(o.C)[(size_t)(t0 + tt) * o.ldc + (size_t)h * dv + col] = ot * o.f0;
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) {
+          const float ot = total(os[j]);
+          if (live[j] && sub == 0) orow[col[j]] = ot * o.f0;
+        }
         continue;
       }
       const float c1 = fixed ? fixed_c1 : cf[tt * 4], c2 = fixed ? o.f0 : cf[tt * 4 + 1];
       if (delta) {
         // both products with the stored state in one pass and one round of shuffles: with S' = c1 S + k u^T,
         // S'^T q = c1 S^T q + u (k . q), and u = c2 (v - c1 S^T k); k . q comes with the token
-        float ks[4] = {0.f, 0.f, 0.f, 0.f};
-        float4 kv[RPT / 4];
 #pragma unroll
-        for (int r = 0; r < RPT / 4; ++r) {
-          kv[r] = k4[r];
-          const float4 qv = q4[r];
-          ks[0] = fmaf(kv[r].x, S[4 * r], ks[0]); ks[1] = fmaf(kv[r].y, S[4 * r + 1], ks[1]);
-          ks[2] = fmaf(kv[r].z, S[4 * r + 2], ks[2]); ks[3] = fmaf(kv[r].w, S[4 * r + 3], ks[3]);
-          os[0] = fmaf(qv.x, S[4 * r], os[0]); os[1] = fmaf(qv.y, S[4 * r + 1], os[1]);
-          os[2] = fmaf(qv.z, S[4 * r + 2], os[2]); os[3] = fmaf(qv.w, S[4 * r + 3], os[3]);
-        }
-        float kt = (ks[0] + ks[1]) + (ks[2] + ks[3]), qt = (os[0] + os[1]) + (os[2] + os[3]);
-        kt += __shfl_xor_sync(0xffffffffu, kt, 1); qt += __shfl_xor_sync(0xffffffffu, qt, 1);
-        kt += __shfl_xor_sync(0xffffffffu, kt, 2); qt += __shfl_xor_sync(0xffffffffu, qt, 2);
-        kt += __shfl_xor_sync(0xffffffffu, kt, 4); qt += __shfl_xor_sync(0xffffffffu, qt, 4);
-        const float u = c2 * (v - c1 * kt);
+        for (int j = 0; j < CPT; ++j) {
+          float ks[4] = {0.f, 0.f, 0.f, 0.f};
+          float4 kv[RPT / 4];
 #pragma unroll
-        for (int r = 0; r < RPT / 4; ++r) {
-          S[4 * r] = fmaf(kv[r].x, u, c1 * S[4 * r]); S[4 * r + 1] = fmaf(kv[r].y, u, c1 * S[4 * r + 1]);
-          S[4 * r + 2] = fmaf(kv[r].z, u, c1 * S[4 * r + 2]); S[4 * r + 3] = fmaf(kv[r].w, u, c1 * S[4 * r + 3]);
+          for (int r = 0; r < RPT / 4; ++r) {
+            kv[r] = k4[r];
+            const float4 qv = q4[r];
+            ks[0] = fmaf(kv[r].x, S[j][4 * r], ks[0]); ks[1] = fmaf(kv[r].y, S[j][4 * r + 1], ks[1]);
+            ks[2] = fmaf(kv[r].z, S[j][4 * r + 2], ks[2]); ks[3] = fmaf(kv[r].w, S[j][4 * r + 3], ks[3]);
+            os[j][0] = fmaf(qv.x, S[j][4 * r], os[j][0]); os[j][1] = fmaf(qv.y, S[j][4 * r + 1], os[j][1]);
+            os[j][2] = fmaf(qv.z, S[j][4 * r + 2], os[j][2]); os[j][3] = fmaf(qv.w, S[j][4 * r + 3], os[j][3]);
+          }
+          float kt = (ks[0] + ks[1]) + (ks[2] + ks[3]), qt = (os[j][0] + os[j][1]) + (os[j][2] + os[j][3]);
+          kt += __shfl_xor_sync(0xffffffffu, kt, 1); qt += __shfl_xor_sync(0xffffffffu, qt, 1);
+          kt += __shfl_xor_sync(0xffffffffu, kt, 2); qt += __shfl_xor_sync(0xffffffffu, qt, 2);
+          kt += __shfl_xor_sync(0xffffffffu, kt, 4); qt += __shfl_xor_sync(0xffffffffu, qt, 4);
+          const float u = c2 * (v[j] - c1 * kt);
+#pragma unroll
+          for (int r = 0; r < RPT / 4; ++r) {
+            S[j][4 * r] = fmaf(kv[r].x, u, c1 * S[j][4 * r]); S[j][4 * r + 1] = fmaf(kv[r].y, u, c1 * S[j][4 * r + 1]);
+            S[j][4 * r + 2] = fmaf(kv[r].z, u, c1 * S[j][4 * r + 2]); S[j][4 * r + 3] = fmaf(kv[r].w, u, c1 * S[j][4 * r + 3]);
+          }
+          if (live[j] && sub == 0) orow[col[j]] = fmaf(u, cf[tt * 4 + 2], c1 * qt);
         }
-        if (live && sub == 0) reinterpret_cast<float*>(o.C)[(size_t)(t0 + tt) * o.ldc + (size_t)h * dv + col] = fmaf(u, cf[tt * 4 + 2], c1 * qt);
         continue;
-      } else if (phase == 1) {
-        const float dx = c2 * v;
+      }
+      float dx[CPT];
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) dx[j] = c2 * v[j];
+      if (phase == 1) {
 #pragma unroll
         for (int r = 0; r < RPT / 4; ++r) {
           const float4 bv = k4[r];
-          S[4 * r] = fmaf(c1, S[4 * r], bv.x * dx); S[4 * r + 1] = fmaf(c1, S[4 * r + 1], bv.y * dx);
-          S[4 * r + 2] = fmaf(c1, S[4 * r + 2], bv.z * dx); S[4 * r + 3] = fmaf(c1, S[4 * r + 3], bv.w * dx);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            S[j][4 * r] = fmaf(c1, S[j][4 * r], bv.x * dx[j]); S[j][4 * r + 1] = fmaf(c1, S[j][4 * r + 1], bv.y * dx[j]);
+            S[j][4 * r + 2] = fmaf(c1, S[j][4 * r + 2], bv.z * dx[j]); S[j][4 * r + 3] = fmaf(c1, S[j][4 * r + 3], bv.w * dx[j]);
+          }
         }
         Pd[0] *= c1;
         continue;
-      } else {
-        const float dx = c2 * v;
+      }
 #pragma unroll
-        for (int r = 0; r < RPT / 4; ++r) {
-          const float4 bv = k4[r], qv = q4[r];
-          S[4 * r] = fmaf(c1, S[4 * r], bv.x * dx); S[4 * r + 1] = fmaf(c1, S[4 * r + 1], bv.y * dx);
-          S[4 * r + 2] = fmaf(c1, S[4 * r + 2], bv.z * dx); S[4 * r + 3] = fmaf(c1, S[4 * r + 3], bv.w * dx);
-          os[0] = fmaf(qv.x, S[4 * r], os[0]); os[1] = fmaf(qv.y, S[4 * r + 1], os[1]);
-          os[2] = fmaf(qv.z, S[4 * r + 2], os[2]); os[3] = fmaf(qv.w, S[4 * r + 3], os[3]);
+      for (int r = 0; r < RPT / 4; ++r) {
+        const float4 bv = k4[r], qv = q4[r];
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) {
+          S[j][4 * r] = fmaf(c1, S[j][4 * r], bv.x * dx[j]); S[j][4 * r + 1] = fmaf(c1, S[j][4 * r + 1], bv.y * dx[j]);
+          S[j][4 * r + 2] = fmaf(c1, S[j][4 * r + 2], bv.z * dx[j]); S[j][4 * r + 3] = fmaf(c1, S[j][4 * r + 3], bv.w * dx[j]);
+          os[j][0] = fmaf(qv.x, S[j][4 * r], os[j][0]); os[j][1] = fmaf(qv.y, S[j][4 * r + 1], os[j][1]);
+          os[j][2] = fmaf(qv.z, S[j][4 * r + 2], os[j][2]); os[j][3] = fmaf(qv.w, S[j][4 * r + 3], os[j][3]);
         }
       }
-      float ot = (os[0] + os[1]) + (os[2] + os[3]);
-      ot += __shfl_xor_sync(0xffffffffu, ot, 1);
-      ot += __shfl_xor_sync(0xffffffffu, ot, 2);
-      ot += __shfl_xor_sync(0xffffffffu, ot, 4);
-      if (memory) {
-        ot *= o.f0;
-        if (col == dv && sub == 0)       // the normaliser's column: what the head's read-out is divided by
-          reinterpret_cast<float*>(o.norm_out)[(size_t)(t0 + tt) * o.norm_ld + h] = fmaxf(fabsf(ot), cf[tt * 4 + 2]) + o.norm_eps;
-        if (col < dv && sub == 0) reinterpret_cast<float*>(o.C)[(size_t)(t0 + tt) * o.ldc + (size_t)h * dv + col] = ot;
-        continue;
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) {
+        float ot = total(os[j]);
+        if (memory) {
+          ot *= o.f0;
+          if (col[j] == dv && sub == 0)       // the normaliser's column: what the head's read-out is divided by
+            reinterpret_cast<float*>(o.norm_out)[(size_t)(t0 + tt) * o.norm_ld + h] = fmaxf(fabsf(ot), cf[tt * 4 + 2]) + o.norm_eps;
+          if (col[j] < dv && sub == 0) orow[col[j]] = ot;
+        } else {
+          ot = fmaf(D, v[j], ot);
+          if (live[j] && sub == 0) orow[col[j]] = ot;
+        }
       }
-      if (!delta) ot = fmaf(D, v, ot);
-      if (live && sub == 0) reinterpret_cast<float*>(o.C)[(size_t)(t0 + tt) * o.ldc + (size_t)h * dv + col] = ot;
     }
     __syncthreads();
   }
   if (phase == 1) {       // this piece's own contribution becomes the next piece's start (after the carry pass); its decay product
     float* nx = X + ((size_t)(zc + 1) * H + h) * hstate;
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live && i < dk) nx[(size_t)i * sv + col] = S[r]; }
+    for (int j = 0; j < CPT; ++j)
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live[j] && i < dk) nx[(size_t)i * sv + col[j]] = S[j][r]; }
     if (blockIdx.x == 0 && cl == 0) {
       float* pz = P + ((size_t)zc * H + h) * dk;
 #pragma unroll
@@ -2262,7 +2339,9 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   if (!last_piece) return;
   float* nst = reinterpret_cast<float*>(o.C2) + (size_t)h * hstate;
 #pragma unroll
-  for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live && i < dk) nst[(size_t)i * sv + col] = S[r]; }
+  for (int j = 0; j < CPT; ++j)
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live[j] && i < dk) nst[(size_t)i * sv + col[j]] = S[j][r]; }
 }
 
 // grid (ceil(H * dk * sv / 256)), sv state columns: X[0] = the carried state; X[z + 1] = P[z] X[z] + X[z + 1] for the pieces in order.

@@ -209,7 +209,7 @@ class RedodraModel:
             if isinstance(m, DeltaRuleConfig):
                 if m.conv > 1:
                     out.append(StateSpec(f"l{i}.dr.conv", "carry", 2 * m.kv_heads * m.dim + m.heads * m.vdim, m.conv - 1))
-                out.append(StateSpec(f"l{i}.dr.s", "carry", m.vdim, m.heads * m.dim))
+                out.append(StateSpec(f"l{i}.dr.s", "carry", m.vdim, m.heads * m.dim, in_place=True))
             elif isinstance(m, SoftmaxAttentionConfig):
                 cache(i, m)
             else:
@@ -217,7 +217,7 @@ class RedodraModel:
                 r = m.right
                 if r.conv > 1:
                     out.append(StateSpec(f"l{i}.ss.conv", "carry", r.inner + 2 * r.groups * r.state, r.conv - 1))
-                out.append(StateSpec(f"l{i}.ss.s", "carry", r.vdim, r.heads * r.state))
+                out.append(StateSpec(f"l{i}.ss.s", "carry", r.vdim, r.heads * r.state, in_place=True))
         return out
 
     # ---- one step of M tokens -----------------------------------------------------------------------

@@ -6,7 +6,8 @@ A model declares what each of its layers keeps between steps as `StateSpec`s:
   * kind "carry":  a fixed block that a step reads and replaces: the last inputs of a causal convolution, a recurrent state.
 A carry is double-buffered (`cur`, `next`): the step's kernels read `cur` and write `next`, and the step's last op
 (FQ3C_COMMIT, include/fq3_codec.h) copies every `next` to its `cur` and advances the slot's device position counter in one
-launch.  All addresses are fixed for the life of the manager, so a captured op list replays at any position of any request
+launch.  A carry with `in_place` has one buffer under both names and nothing to install: for large states whose kernel reads every
+entry before the same thread (or a later launch) writes it.  All addresses are fixed for the life of the manager, so a captured op list replays at any position of any request
 that later occupies the slot.  A slot is handed to one request at a time; releasing it gives everything back, and acquiring
 zeroes the carries and the counter (a cache needs no clearing: rows at or beyond the counter are never read).
 """
@@ -26,6 +27,7 @@ class StateSpec:
     rows: int = 1             # carry: rows of the block; append: ignored (capacity comes from the manager)
     dtype: torch.dtype = torch.float32
     every: int = 1            # append: positions per row
+    in_place: bool = False    # carry: the step updates the block where it lies
 
 
 class SlotState:
@@ -45,6 +47,9 @@ class SlotState:
                 if s.rows <= 0:
                     continue
                 a = torch.zeros(s.rows, s.cols, dtype=s.dtype, device=device)
+                if s.in_place:
+                    self.cur[s.name] = self.next[s.name] = a
+                    continue
                 b = torch.zeros(s.rows, s.cols, dtype=s.dtype, device=device)
                 self.cur[s.name], self.next[s.name] = a, b
                 table.append([a.data_ptr(), b.data_ptr(), a.numel() * a.element_size()])
@@ -62,7 +67,8 @@ class SlotState:
         self.length = 0
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in list(self.cur.values()) + list(self.next.values()))
+        own = {t.data_ptr(): t.numel() * t.element_size() for t in list(self.cur.values()) + list(self.next.values())}
+        return sum(own.values())
 
 
 class SequenceStateManager:

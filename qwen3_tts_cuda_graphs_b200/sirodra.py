@@ -158,9 +158,9 @@ class SirodraModel:
         for r, (i, _) in enumerate(self.cfg.runs):       # every layer run has a state of its own, also the later passes of a loop
             m, p = self.cfg.layers[i].mixer, f"r{r}."
             if isinstance(m, ForgetGateAttentionConfig):
-                out.append(StateSpec(p + "fg", "carry", m.vdim, m.heads * m.dim))
+                out.append(StateSpec(p + "fg", "carry", m.vdim, m.heads * m.dim, in_place=True))
             elif isinstance(m, MatrixMemoryConfig):
-                out += [StateSpec(p + "mm.s", "carry", m.vdim + 1, m.heads * m.dim), StateSpec(p + "mm.m", "carry", m.heads)]
+                out += [StateSpec(p + "mm.s", "carry", m.vdim + 1, m.heads * m.dim, in_place=True), StateSpec(p + "mm.m", "carry", m.heads)]
             else:
                 for n, cols in (("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
                     out.append(StateSpec(p + n, "append", cols, dtype=self.wdt))

@@ -203,11 +203,11 @@ class ZudusunModel:
             m = L.mixer
             if isinstance(m, ScaledPairMixerConfig):
                 cache(i, m.left)
-                out.append(StateSpec(f"l{i}.cd.s", "carry", m.right.vdim, m.right.heads * m.right.dim))
+                out.append(StateSpec(f"l{i}.cd.s", "carry", m.right.vdim, m.right.heads * m.right.dim, in_place=True))
             elif isinstance(m, SoftmaxAttentionConfig):
                 cache(i, m)
             else:
-                out.append(StateSpec(f"l{i}.rt.s", "carry", m.vdim, m.heads * m.dim))
+                out.append(StateSpec(f"l{i}.rt.s", "carry", m.vdim, m.heads * m.dim, in_place=True))
         return out
 
     # ---- one step of M tokens -----------------------------------------------------------------------
