@@ -1055,6 +1055,9 @@ int launch_seq_gemm(const SeqGemm& g, bool a_f32, bool b_f32, bool exact, int zc
   return 0;
 }
 
+// threads of a block that works on one row of n entries: with a few rows (decoding) one per entry, so that the row's loads are one round trip
+int row_threads(int rows, int n, int many) { return rows <= 8 ? std::max(32, std::min(1024, (n + 31) / 32 * 32)) : many; }
+
 // returns 1 when the kind is not a sequence-model op
 int seq_run(const fq3c_op& o, cudaStream_t s) {
   switch (o.kind) {
@@ -1062,8 +1065,8 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       if (!o.A || !o.B || !o.C) return fail("embed: missing operand");
       if (o.i0 > 1 && o.K < o.N) return fail("embed: copies need a stride of at least N elements");
       if (o.C2 && o.ldr < o.N * std::max(o.i1, 1)) return fail("embed: the operand copies do not fit their pitch");
-      if (o.flags & FQ3C_F32) fq3s_embed_kernel<float><<<o.M, 128, 0, s>>>(o);
-      else fq3s_embed_kernel<bf16><<<o.M, 128, 0, s>>>(o);
+      if (o.flags & FQ3C_F32) fq3s_embed_kernel<float><<<o.M, row_threads(o.M, o.N, 128), 0, s>>>(o);
+      else fq3s_embed_kernel<bf16><<<o.M, row_threads(o.M, o.N, 128), 0, s>>>(o);
       return 0;
     case FQ3C_TCONV:
       if (o.taps < 1 || !o.A || !o.B || !o.C || (o.taps > 1 && (!o.p0 || !o.p1))) return fail("tconv: missing operand");
@@ -1072,7 +1075,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
     case FQ3C_GNORM:
       if (o.i0 < 1 || o.N % o.i0 || ((o.flags & FQ3C_RESID) && !o.res)) return fail("gnorm: groups must divide N");
       if ((o.flags & (FQ3C_GATE_PRE | FQ3C_GATE_POST)) && !o.p1) return fail("gnorm: gate rows required");
-      fq3s_gnorm_kernel<<<dim3(o.M, o.i0), 128, 0, s>>>(o);
+      fq3s_gnorm_kernel<<<dim3(o.M, o.i0), row_threads(o.M, o.N / o.i0, 128), 0, s>>>(o);
       return 0;
     case FQ3C_POLYNORM:
       if (!o.p0) return fail("polynorm: coefficients required");
@@ -1430,7 +1433,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         cudaFuncSetAttribute(fq3s_sum_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         nattr[dev] = true;
       }
-      fq3s_sum_norm_kernel<<<o.M, 256, (size_t)o.N * 4, s>>>(o);
+      fq3s_sum_norm_kernel<<<o.M, row_threads(o.M, o.N, 256), (size_t)o.N * 4, s>>>(o);
       return 0;
     }
     default: return 1;

@@ -651,11 +651,11 @@ __global__ void __launch_bounds__(256) fq3s_tconv_kernel(const fq3c_op o) {
   else reinterpret_cast<bf16*>(o.C)[(size_t)m * o.ldc + c] = __float2bfloat16_rn(a);
 }
 
-// grid (M, groups); one block per (row, group).  FQ3C_CENTER: mean and variance instead of the mean square.  An optional silu gate (p1, pitch i1;
+// grid (M, groups); one block per (row, group): 128 threads, or up to 1024 for a few rows (decoding).  FQ3C_CENTER: mean and variance instead of the mean square.  An optional silu gate (p1, pitch i1;
 // FQ3C_SIGMOID: a sigmoid gate) multiplies the row before the statistics (FQ3C_GATE_PRE) or the finished row (FQ3C_GATE_POST); weights repeat
 // with period i2 when i2 > 0; divisors (bias, pitch cin) divide a group before anything else.
 __device__ __forceinline__ float gate_f(const float z, const bool plain) { return plain ? sigmoid_f(z) : z / (1.f + expf(-z)); }
-__global__ void __launch_bounds__(128) fq3s_gnorm_kernel(const fq3c_op o) {
+__global__ void __launch_bounds__(1024) fq3s_gnorm_kernel(const fq3c_op o) {
   __shared__ float red[32];
   const int m = blockIdx.x, gsz = o.N / o.i0, c0 = blockIdx.y * gsz;
   const float* x = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda + c0;
@@ -1606,6 +1606,7 @@ __global__ void __launch_bounds__(128) fq3s_cache_attn_merge_kernel(const fq3c_o
   const float sc = gate / den;
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
     float acc = 0.f;
+#pragma unroll 8
     for (int s = 0; s < splits; ++s) acc = fmaf(wsm[s], src[(size_t)s * (dv + 2) + 2 + c], acc);
     const float v = acc * sc;
     if (o.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(o.C)[(size_t)m * o.ldc + (size_t)h * dv + c] = v;
@@ -2433,10 +2434,10 @@ __global__ void __launch_bounds__(256) fq3s_glu_kernel(const fq3c_op o) {
 // ABI 9 (kind 32): the residual sum of a layer whose sublayers run side by side on one normed input, fused with the norm that
 // reads the finished stream (a layer norm without bias, or an RMS norm).
 // ===========================================================================================================================
-// grid (M), 256 threads, dynamic shared memory N floats (the finished row).  Pass 1 forms the weighted sum of the slices, writes it
+// grid (M), 256 threads (up to 1024 for a few rows), dynamic shared memory N floats (the finished row).  Pass 1 forms the weighted sum of the slices, writes it
 // and keeps it; passes 2 and 3 take the mean and the mean squared deviation from the kept row; pass 4 writes the normed row.
 // A thread only ever reads back entries it wrote itself, and C may be slice 0 (every entry is read before it is written).
-__global__ void __launch_bounds__(256) fq3s_sum_norm_kernel(const fq3c_op o) {
+__global__ void __launch_bounds__(1024) fq3s_sum_norm_kernel(const fq3c_op o) {
   extern __shared__ float snm[];
   __shared__ float red[32];
   const int m = blockIdx.x;
@@ -2446,7 +2447,14 @@ __global__ void __launch_bounds__(256) fq3s_sum_norm_kernel(const fq3c_op o) {
   float sm = 0.f;
   for (int i = threadIdx.x; i < o.N; i += blockDim.x) {
     float v = 0.f;
-    for (int j = 0; j < o.i0; ++j) v = fmaf(w[j], a[(size_t)j * (size_t)o.K + i], v);
+    for (int j = 0; j < o.i0; j += 4) {       // four slices' loads in flight
+      float wv[4], av[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) { const bool ok = j + q < o.i0; wv[q] = ok ? w[j + q] : 0.f; av[q] = ok ? a[(size_t)(j + q) * (size_t)o.K + i] : 0.f; }
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+        if (j + q < o.i0) v = fmaf(wv[q], av[q], v);
+    }
     c[i] = v;
     if (o.C2) reinterpret_cast<bf16*>(o.C2)[(size_t)m * o.ldc + i] = __float2bfloat16_rn(v);
     snm[i] = v;
