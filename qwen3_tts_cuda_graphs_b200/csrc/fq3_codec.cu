@@ -107,6 +107,23 @@ __device__ __forceinline__ void epilogue_pair(const fq3c_op& o, int row, int col
 // Epilogue for eight consecutive columns of one row (the tcgen05 path: a thread owns a row of the accumulator, so it
 // must move whole 16-byte pieces or every store is a partial sector).  Same arithmetic and order as epilogue_pair.
 __device__ __forceinline__ void epilogue_row8(const fq3c_op& o, int row, int col, const float (&acc)[8]) {
+  // unrounded f32 rows (the sequence models' projections): two 16-byte stores, one whole sector
+  if ((o.flags & (FQ3C_OUT_F32 | FQ3C_NOROUND)) == (FQ3C_OUT_F32 | FQ3C_NOROUND) && !(o.flags & ~(FQ3C_OUT_F32 | FQ3C_NOROUND | FQ3C_BIAS)) &&
+      col + 8 <= o.N && (o.ldc & 3) == 0 && o.col_mod == o.N && !(reinterpret_cast<uintptr_t>(o.C) & 15)) {
+    if (row >= o.M) return;
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = acc[j];
+    if (o.flags & FQ3C_BIAS) {
+      const float* b = reinterpret_cast<const float*>(o.bias) + col;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] += b[j];
+    }
+    float4* c = reinterpret_cast<float4*>(reinterpret_cast<float*>(o.C) + (size_t)row * o.ldc + col);
+    c[0] = make_float4(v[0], v[1], v[2], v[3]);
+    c[1] = make_float4(v[4], v[5], v[6], v[7]);
+    return;
+  }
   const bool vec = (col + 8 <= o.N) && !(o.flags & (FQ3C_SWIGLU | FQ3C_OUT_F32)) && ((o.ldc & 7) == 0) &&
                    (!(o.flags & FQ3C_RESID) || (o.ldr & 7) == 0);
   if (!vec) {
