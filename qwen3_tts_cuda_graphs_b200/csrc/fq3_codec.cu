@@ -69,7 +69,10 @@ __device__ __forceinline__ void epilogue_pair(const fq3c_op& o, int row, int col
     reinterpret_cast<bf16*>(o.C)[(size_t)row * o.ldc + (col >> 1)] = __float2bfloat16_rn(y);
     return;
   }
-  if (o.flags & FQ3C_GELU) { v0 = bf16r(gelu_f(v0)); v1 = bf16r(gelu_f(v1)); }
+  if (o.flags & FQ3C_GELU) {
+    v0 = gelu_f(v0); v1 = gelu_f(v1);
+    if (!(o.flags & FQ3C_NOROUND)) { v0 = bf16r(v0); v1 = bf16r(v1); }
+  }
   if (o.flags & FQ3C_SILU) { v0 = bf16r(silu_f(v0)); v1 = bf16r(silu_f(v1)); }
   if (o.flags & FQ3C_SCALE) {
     const float* s = reinterpret_cast<const float*>(o.scale);
@@ -107,9 +110,10 @@ __device__ __forceinline__ void epilogue_pair(const fq3c_op& o, int row, int col
 // Epilogue for eight consecutive columns of one row (the tcgen05 path: a thread owns a row of the accumulator, so it
 // must move whole 16-byte pieces or every store is a partial sector).  Same arithmetic and order as epilogue_pair.
 __device__ __forceinline__ void epilogue_row8(const fq3c_op& o, int row, int col, const float (&acc)[8]) {
-  // unrounded f32 rows (the sequence models' projections): two 16-byte stores, one whole sector
-  if ((o.flags & (FQ3C_OUT_F32 | FQ3C_NOROUND)) == (FQ3C_OUT_F32 | FQ3C_NOROUND) && !(o.flags & ~(FQ3C_OUT_F32 | FQ3C_NOROUND | FQ3C_BIAS)) &&
-      col + 8 <= o.N && (o.ldc & 3) == 0 && o.col_mod == o.N && !(reinterpret_cast<uintptr_t>(o.C) & 15)) {
+  // the sequence models' products: unrounded f32 rows as two 16-byte stores (one whole sector), or an activation taken on the f32 sum
+  // and rounded once
+  if ((o.flags & FQ3C_NOROUND) && !(o.flags & ~(FQ3C_OUT_F32 | FQ3C_NOROUND | FQ3C_BIAS | FQ3C_GELU)) && col + 8 <= o.N &&
+      (o.ldc & ((o.flags & FQ3C_OUT_F32) ? 3 : 7)) == 0 && o.col_mod == o.N && !(reinterpret_cast<uintptr_t>(o.C) & 15)) {
     if (row >= o.M) return;
     float v[8];
 #pragma unroll
@@ -118,6 +122,20 @@ __device__ __forceinline__ void epilogue_row8(const fq3c_op& o, int row, int col
       const float* b = reinterpret_cast<const float*>(o.bias) + col;
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[j] += b[j];
+    }
+    if (o.flags & FQ3C_GELU) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] = gelu_f(v[j]);
+    }
+    if (!(o.flags & FQ3C_OUT_F32)) {
+      uint32_t w[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+        w[j] = *reinterpret_cast<const uint32_t*>(&h);
+      }
+      *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(o.C) + (size_t)row * o.ldc + col) = make_uint4(w[0], w[1], w[2], w[3]);
+      return;
     }
     float4* c = reinterpret_cast<float4*>(reinterpret_cast<float*>(o.C) + (size_t)row * o.ldc + col);
     c[0] = make_float4(v[0], v[1], v[2], v[3]);
@@ -1092,6 +1110,14 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
     case FQ3C_GNORM:
       if (o.i0 < 1 || o.N % o.i0 || ((o.flags & FQ3C_RESID) && !o.res)) return fail("gnorm: groups must divide N");
       if ((o.flags & (FQ3C_GATE_PRE | FQ3C_GATE_POST)) && !o.p1) return fail("gnorm: gate rows required");
+      // many (row, group) pairs of a size a warp holds in registers, 16-byte rows: a warp per pair
+      if ((int64_t)o.M * o.i0 >= 1024 && o.N / o.i0 % 4 == 0 && o.N / o.i0 <= 4 * 32 * GN_VECS && o.i2 % 4 == 0 && !((o.lda | o.ldc | o.ldr) & 3) &&
+          (!(o.flags & (FQ3C_GATE_PRE | FQ3C_GATE_POST)) || o.i1 % 4 == 0) &&
+          !((reinterpret_cast<uintptr_t>(o.A) | reinterpret_cast<uintptr_t>(o.C) | reinterpret_cast<uintptr_t>(o.C2) | reinterpret_cast<uintptr_t>(o.p1) |
+             reinterpret_cast<uintptr_t>(o.res) | reinterpret_cast<uintptr_t>(o.scale)) & 15)) {
+        fq3s_gnorm_warp_kernel<<<(unsigned)(((int64_t)o.M * o.i0 + 3) / 4), 128, 0, s>>>(o);
+        return 0;
+      }
       fq3s_gnorm_kernel<<<dim3(o.M, o.i0), row_threads(o.M, o.N / o.i0, 128), 0, s>>>(o);
       return 0;
     case FQ3C_POLYNORM:
@@ -1449,6 +1475,12 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       if (dev >= 0 && dev < 64 && !nattr[dev]) {
         cudaFuncSetAttribute(fq3s_sum_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         nattr[dev] = true;
+      }
+      // rows of whole 16-byte pieces that a block of 256 holds in registers
+      if (o.N % 4 == 0 && o.N <= 1024 * SN_VECS && !((o.lda | o.ldc | o.norm_ld | o.K) & 3) && !o.C2 &&
+          !((reinterpret_cast<uintptr_t>(o.A) | reinterpret_cast<uintptr_t>(o.C) | reinterpret_cast<uintptr_t>(o.norm_out) | reinterpret_cast<uintptr_t>(o.norm_w)) & 15)) {
+        fq3s_sum_norm_vec_kernel<<<o.M, std::max(32, std::min(256, (o.N / 4 + 31) / 32 * 32)), 0, s>>>(o);
+        return 0;
       }
       fq3s_sum_norm_kernel<<<o.M, row_threads(o.M, o.N, 256), (size_t)o.N * 4, s>>>(o);
       return 0;

@@ -698,6 +698,73 @@ __global__ void __launch_bounds__(1024) fq3s_gnorm_kernel(const fq3c_op o) {
   }
 }
 
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void st4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void st4(bf16* p, const float (&v)[4]) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+// The same norm for many (row, group) pairs: a warp each, the group in registers, 16-byte loads.  grid (ceil(M * groups / 4)), 128 threads.
+constexpr int GN_VECS = 4;
+__global__ void __launch_bounds__(128) fq3s_gnorm_warp_kernel(const fq3c_op o) {
+  const long long pair = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (pair >= (long long)o.M * o.i0) return;
+  const int lane = threadIdx.x & 31, m = (int)(pair / o.i0), gi = (int)(pair - (long long)m * o.i0), gsz = o.N / o.i0, c0 = gi * gsz;
+  const float* x = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda + c0;
+  const bool pre = (o.flags & FQ3C_GATE_PRE) != 0, post = (o.flags & FQ3C_GATE_POST) != 0, plain = (o.flags & FQ3C_SIGMOID) != 0;
+  const float* gate = (pre || post) ? reinterpret_cast<const float*>(o.p1) + (size_t)m * o.i1 + c0 : nullptr;
+  const float inv = o.bias ? 1.f / reinterpret_cast<const float*>(o.bias)[(size_t)m * o.cin + gi] : 1.f;
+  float v[GN_VECS][4], g[GN_VECS][4];
+#pragma unroll
+  for (int q = 0; q < GN_VECS; ++q) {
+    const int i = (q * 32 + lane) * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+    if (i < gsz) { a = ld4(x + i); if (gate) b = ld4(gate + i); }
+    v[q][0] = a.x * inv; v[q][1] = a.y * inv; v[q][2] = a.z * inv; v[q][3] = a.w * inv;
+    g[q][0] = b.x; g[q][1] = b.y; g[q][2] = b.z; g[q][3] = b.w;
+  }
+  float sm = 0.f, ss = 0.f;
+#pragma unroll
+  for (int q = 0; q < GN_VECS; ++q)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (gate) g[q][e] = gate_f(g[q][e], plain);
+      if (pre) v[q][e] *= g[q][e];
+      sm += v[q][e];
+    }
+  const float mean = (o.flags & FQ3C_CENTER) ? warp_sum(sm) / (float)gsz : 0.f;
+#pragma unroll
+  for (int q = 0; q < GN_VECS; ++q)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[q][e] -= mean;
+      if ((q * 32 + lane) * 4 < gsz) ss = fmaf(v[q][e], v[q][e], ss);
+    }
+  const float rs = 1.f / sqrtf(warp_sum(ss) / (float)gsz + o.f0);
+  const float* w = reinterpret_cast<const float*>(o.scale);
+  const int wmod = o.i2 > 0 ? o.i2 : o.N;
+  const size_t orow = (size_t)m + (o.p0 ? (size_t)*reinterpret_cast<const int*>(o.p0) : 0);
+#pragma unroll
+  for (int q = 0; q < GN_VECS; ++q) {
+    const int i = (q * 32 + lane) * 4;
+    if (i >= gsz) continue;
+    float4 wv = make_float4(1.f, 1.f, 1.f, 1.f), r = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (w) wv = ld4(w + (c0 + i) % wmod);
+    if (o.flags & FQ3C_RESID) r = ld4(reinterpret_cast<const float*>(o.res) + (size_t)m * o.ldr + c0 + i);
+    const float ww[4] = {wv.x, wv.y, wv.z, wv.w}, rr[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[q][e] *= rs;
+      if (w) v[q][e] *= ww[e];
+      if (post) v[q][e] *= g[q][e];
+      if (o.flags & FQ3C_RESID) v[q][e] += rr[e];
+    }
+    if (o.flags & FQ3C_OUT_F32) st4(reinterpret_cast<float*>(o.C) + orow * o.ldc + c0 + i, v[q]);
+    else st4(reinterpret_cast<bf16*>(o.C) + orow * o.ldc + c0 + i, v[q]);
+    if (o.C2) st4(reinterpret_cast<bf16*>(o.C2) + orow * o.ldc + c0 + i, v[q]);
+  }
+}
+
 __global__ void __launch_bounds__(256) fq3s_polynorm_kernel(const fq3c_op o) {
   __shared__ float red[32];
   const int m = blockIdx.x;
@@ -2200,6 +2267,7 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
     const float* kq = msm + (it & 1) * per;
     const float* vs = kq + CH * NV * ROW;
     const float* cf = vs + CH * COLS;
+#pragma unroll CPT
     for (int tt = 0; tt < (wlive ? nt : 0); ++tt) {
       const float4* k4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + sub * SL);
       const float4* q4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + ROW + sub * SL);
@@ -2478,5 +2546,69 @@ __global__ void __launch_bounds__(1024) fq3s_sum_norm_kernel(const fq3c_op o) {
     const float n = (snm[i] - mean) * rs * nw[i];
     if (o.flags & FQ3C_F32) reinterpret_cast<float*>(o.norm_out)[(size_t)m * o.norm_ld + i] = n;
     else reinterpret_cast<bf16*>(o.norm_out)[(size_t)m * o.norm_ld + i] = __float2bfloat16_rn(n);
+  }
+}
+
+// The same for rows of whole 16-byte pieces: the row stays in registers.  grid (M), up to 256 threads.
+constexpr int SN_VECS = 4;
+__global__ void __launch_bounds__(256) fq3s_sum_norm_vec_kernel(const fq3c_op o) {
+  __shared__ float red[32];
+  const int m = blockIdx.x, tid = threadIdx.x, nth = blockDim.x;
+  const float* a = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda;
+  const float* w = reinterpret_cast<const float*>(o.p0);
+  float* c = reinterpret_cast<float*>(o.C) + (size_t)m * o.ldc;
+  float v[SN_VECS][4];
+#pragma unroll
+  for (int q = 0; q < SN_VECS; ++q) { v[q][0] = 0.f; v[q][1] = 0.f; v[q][2] = 0.f; v[q][3] = 0.f; }
+  for (int j = 0; j < o.i0; j += 2) {       // two slices' loads in flight
+    float4 s0[SN_VECS], s1[SN_VECS];
+    const bool two = j + 1 < o.i0;
+    const float w0 = w[j], w1 = two ? w[j + 1] : 0.f;
+#pragma unroll
+    for (int q = 0; q < SN_VECS; ++q) {
+      const int i = (q * nth + tid) * 4;
+      if (i < o.N) {
+        s0[q] = ld4(a + (size_t)j * (size_t)o.K + i);
+        if (two) s1[q] = ld4(a + (size_t)(j + 1) * (size_t)o.K + i);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < SN_VECS; ++q) {
+      if ((q * nth + tid) * 4 >= o.N) continue;
+      v[q][0] = fmaf(w0, s0[q].x, v[q][0]); v[q][1] = fmaf(w0, s0[q].y, v[q][1]); v[q][2] = fmaf(w0, s0[q].z, v[q][2]); v[q][3] = fmaf(w0, s0[q].w, v[q][3]);
+      if (two) { v[q][0] = fmaf(w1, s1[q].x, v[q][0]); v[q][1] = fmaf(w1, s1[q].y, v[q][1]); v[q][2] = fmaf(w1, s1[q].z, v[q][2]); v[q][3] = fmaf(w1, s1[q].w, v[q][3]); }
+    }
+  }
+  float sm = 0.f;
+#pragma unroll
+  for (int q = 0; q < SN_VECS; ++q) {
+    const int i = (q * nth + tid) * 4;
+    if (i >= o.N) continue;
+    st4(c + i, v[q]);
+    sm += (v[q][0] + v[q][1]) + (v[q][2] + v[q][3]);
+  }
+  if (!o.norm_out) return;
+  float rs = 1.f, mean = 0.f;
+  if (o.norm_w) {
+    if (o.flags & FQ3C_CENTER) mean = seq_block_sum(sm, red) / (float)o.N;
+    float ss = 0.f;
+#pragma unroll
+    for (int q = 0; q < SN_VECS; ++q) {
+      if ((q * nth + tid) * 4 >= o.N) continue;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { const float d = v[q][e] - mean; ss = fmaf(d, d, ss); }
+    }
+    rs = 1.f / sqrtf(seq_block_sum(ss, red) / (float)o.N + o.norm_eps);
+  }
+#pragma unroll
+  for (int q = 0; q < SN_VECS; ++q) {
+    const int i = (q * nth + tid) * 4;
+    if (i >= o.N) continue;
+    if (o.norm_w) {
+      const float4 nw = ld4(reinterpret_cast<const float*>(o.norm_w) + i);
+      v[q][0] = (v[q][0] - mean) * rs * nw.x; v[q][1] = (v[q][1] - mean) * rs * nw.y; v[q][2] = (v[q][2] - mean) * rs * nw.z; v[q][3] = (v[q][3] - mean) * rs * nw.w;
+    }
+    if (o.flags & FQ3C_F32) st4(reinterpret_cast<float*>(o.norm_out) + (size_t)m * o.norm_ld + i, v[q]);
+    else st4(reinterpret_cast<bf16*>(o.norm_out) + (size_t)m * o.norm_ld + i, v[q]);
   }
 }

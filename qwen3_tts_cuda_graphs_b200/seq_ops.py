@@ -165,8 +165,8 @@ class StepBuilder:
         f32 = w.dtype == torch.float32
         assert x.dtype == w.dtype, (x.dtype, w.dtype)
         flags = self._oflag(out) | (F_BIAS if bias is not None else 0) | (F_GELU if gelu else 0) | (F_F32 if f32 else 0) | (F_RELU2 if relu2 else 0)
-        if out.dtype == torch.float32 or M <= 4 or glu:
-            flags |= F_NOROUND      # f32 results stay unrounded; with a few rows the flag also picks the weight-streaming product
+        if out.dtype == torch.float32 or M <= 4 or glu or gelu:
+            flags |= F_NOROUND      # f32 results and the activation's argument stay unrounded; with a few rows the flag also picks the weight-streaming product
         if glu:
             flags |= F_SWIGLU
         kw = dict(M=M, N=N, K=K, taps=1, cin=K, a_rows=x.shape[0], lda=x.shape[1], ldc=out.shape[1], col_mod=N, A=x, B=w, C=out, flags=flags)
