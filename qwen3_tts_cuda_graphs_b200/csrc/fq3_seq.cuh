@@ -2125,6 +2125,26 @@ constexpr int MS_COLS = 16;   // state columns per block (eight lanes each), tim
 __device__ __forceinline__ void cp_async4(void* dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
+// two f32 values side by side: one instruction multiplies (adds) both, each rounded as the scalar operation rounds
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) { f32x2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
+__device__ __forceinline__ float lo2(f32x2 v) { float a, b; asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); return a; }
+__device__ __forceinline__ float hi2(f32x2 v) { float a, b; asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); return b; }
+// PACKED false: the same two operations as scalar instructions (for code that is bound by registers or shared memory, not by issue)
+template <bool PACKED>
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  if (!PACKED) return pack2(fmaf(lo2(a), lo2(b), lo2(c)), fmaf(hi2(a), hi2(b), hi2(c)));
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+template <bool PACKED>
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  if (!PACKED) return pack2(lo2(a) * lo2(b), hi2(a) * hi2(b));
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
 // floats per staging buffer: (k, q) or (B, C) (and the decays) [CH][NV][8 slices of RPT + 4] | v [CH][columns] | coefficients [CH][4]
 __host__ __device__ constexpr int mstate_ch(int cpt) { return MS_CH / cpt; }
 __host__ __device__ constexpr int mstate_buf_floats(int rpt, int nv = 2, int cpt = 1) {
@@ -2148,6 +2168,7 @@ template <int RPT, int NV = 2, bool GATED = false, int CPT = 1>
 __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, const int phase, const int piece, float* X, float* P) {
   extern __shared__ __align__(16) float msm[];
   constexpr int SL = RPT + 4, ROW = 8 * SL, CH = mstate_ch(CPT), COLS = MS_COLS * CPT;
+  constexpr bool PK = NV == 2;      // with three staged vectors the walk is bound by shared memory, and pairs only cost registers
   const int H = o.i0, G = o.i1, dk = o.i2, dv = o.cin, h = blockIdx.y, g = h / (H / G);
   const bool delta = !GATED && NV == 2 && CPT == 1 && o.taps == 0, fixed = !GATED && NV == 2 && o.taps == 3;
   const bool gates = GATED && NV == 3, memory = GATED && NV == 2;
@@ -2167,16 +2188,20 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
     const int used = min(te - tb, CH) * NV * ROW;
     for (int i = tid; i < 2 * used; i += 128) msm[(i < used ? 0 : per - used) + i] = 0.f;
   }
-  float S[CPT][RPT];
-  float Pd[NV == 3 ? RPT : 1];       // phase 1: the product of the piece's decays (per state row, or one number per head)
+  f32x2 S[CPT][RPT / 2];
+  f32x2 Pd[NV == 3 ? RPT / 2 : 1];   // phase 1: the product of the piece's decays (per state row, or one number per head)
 #pragma unroll
-  for (int r = 0; r < (NV == 3 ? RPT : 1); ++r) Pd[r] = 1.f;
+  for (int r = 0; r < (NV == 3 ? RPT / 2 : 1); ++r) Pd[r] = pack2(1.f, 1.f);
   const size_t hstate = (size_t)dk * sv;
   const float* st = phase == 3 ? X + ((size_t)zc * H + h) * hstate : reinterpret_cast<const float*>(o.p0) + (size_t)h * hstate;
 #pragma unroll
   for (int j = 0; j < CPT; ++j)
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; S[j][r] = (phase != 1 && live[j] && i < dk) ? st[(size_t)i * sv + col[j]] : 0.f; }
+    for (int r = 0; r < RPT / 2; ++r) {
+      const int i = sub * RPT + 2 * r;
+      const bool ok = phase != 1 && live[j];
+      S[j][r] = pack2(ok && i < dk ? st[(size_t)i * sv + col[j]] : 0.f, ok && i + 1 < dk ? st[(size_t)(i + 1) * sv + col[j]] : 0.f);
+    }
   const float D = (o.taps == 1 && o.B) ? reinterpret_cast<const float*>(o.B)[h] : 0.f;
   const float* wsb = reinterpret_cast<const float*>(o.ws);
   const float* rows = reinterpret_cast<const float*>(o.A);
@@ -2269,15 +2294,17 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
     const float* cf = vs + CH * COLS;
 #pragma unroll CPT
     for (int tt = 0; tt < (wlive ? nt : 0); ++tt) {
-      const float4* k4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + sub * SL);
-      const float4* q4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + ROW + sub * SL);
+      const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(kq + tt * NV * ROW + sub * SL);      // four entries: two pairs
+      const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(kq + tt * NV * ROW + ROW + sub * SL);
       float v[CPT];
 #pragma unroll
       for (int j = 0; j < CPT; ++j) v[j] = vs[tt * COLS + cl + j * MS_COLS];
-      float os[CPT][4] = {};       // four chains, so that a product's sum is not one long dependent row of multiply-adds
+      f32x2 os[CPT][2];            // four chains, so that a product's sum is not one long dependent row of multiply-adds
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) { os[j][0] = 0ull; os[j][1] = 0ull; }
       // a finished product: its four chains, then the eight lanes of the column
-      auto total = [&](const float (&c)[4]) {
-        float x = (c[0] + c[1]) + (c[2] + c[3]);
+      auto total = [&](const f32x2 (&c)[2]) {
+        float x = (lo2(c[0]) + hi2(c[0])) + (lo2(c[1]) + hi2(c[1]));
         x += __shfl_xor_sync(0xffffffffu, x, 1);
         x += __shfl_xor_sync(0xffffffffu, x, 2);
         x += __shfl_xor_sync(0xffffffffu, x, 4);
@@ -2285,30 +2312,34 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
       };
       float* orow = reinterpret_cast<float*>(o.C) + (size_t)(t0 + tt) * o.ldc + (size_t)h * dv;
       if (NV == 3) {      // S <- diag(alpha) S + k v^T, o = f0 S^T q
-        const float4* a4 = reinterpret_cast<const float4*>(kq + tt * NV * ROW + 2 * ROW + sub * SL);
+        const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(kq + tt * NV * ROW + 2 * ROW + sub * SL);
+        f32x2 vv[CPT];
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) vv[j] = pack2(v[j], v[j]);
         if (phase == 1) {
 #pragma unroll
           for (int r = 0; r < RPT / 4; ++r) {
-            const float4 kv = k4[r], av = a4[r];
+            const ulonglong2 kv = k4[r], av = a4[r];
 #pragma unroll
             for (int j = 0; j < CPT; ++j) {
-              S[j][4 * r] = fmaf(av.x, S[j][4 * r], kv.x * v[j]); S[j][4 * r + 1] = fmaf(av.y, S[j][4 * r + 1], kv.y * v[j]);
-              S[j][4 * r + 2] = fmaf(av.z, S[j][4 * r + 2], kv.z * v[j]); S[j][4 * r + 3] = fmaf(av.w, S[j][4 * r + 3], kv.w * v[j]);
+              S[j][2 * r] = fma2<PK>(av.x, S[j][2 * r], mul2<PK>(kv.x, vv[j]));
+              S[j][2 * r + 1] = fma2<PK>(av.y, S[j][2 * r + 1], mul2<PK>(kv.y, vv[j]));
             }
             constexpr int PR = NV == 3 ? 1 : 0;     // (this branch only runs with NV == 3; the index stays legal in the other instantiation)
-            Pd[PR * (4 * r)] *= av.x; Pd[PR * (4 * r + 1)] *= av.y; Pd[PR * (4 * r + 2)] *= av.z; Pd[PR * (4 * r + 3)] *= av.w;
+            Pd[PR * (2 * r)] = mul2<PK>(Pd[PR * (2 * r)], av.x);
+            Pd[PR * (2 * r + 1)] = mul2<PK>(Pd[PR * (2 * r + 1)], av.y);
           }
           continue;
         }
 #pragma unroll
         for (int r = 0; r < RPT / 4; ++r) {
-          const float4 kv = k4[r], qv = q4[r], av = a4[r];
+          const ulonglong2 kv = k4[r], qv = q4[r], av = a4[r];
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
-            S[j][4 * r] = fmaf(av.x, S[j][4 * r], kv.x * v[j]); S[j][4 * r + 1] = fmaf(av.y, S[j][4 * r + 1], kv.y * v[j]);
-            S[j][4 * r + 2] = fmaf(av.z, S[j][4 * r + 2], kv.z * v[j]); S[j][4 * r + 3] = fmaf(av.w, S[j][4 * r + 3], kv.w * v[j]);
-            os[j][0] = fmaf(qv.x, S[j][4 * r], os[j][0]); os[j][1] = fmaf(qv.y, S[j][4 * r + 1], os[j][1]);
-            os[j][2] = fmaf(qv.z, S[j][4 * r + 2], os[j][2]); os[j][3] = fmaf(qv.w, S[j][4 * r + 3], os[j][3]);
+            S[j][2 * r] = fma2<PK>(av.x, S[j][2 * r], mul2<PK>(kv.x, vv[j]));
+            S[j][2 * r + 1] = fma2<PK>(av.y, S[j][2 * r + 1], mul2<PK>(kv.y, vv[j]));
+            os[j][0] = fma2<PK>(qv.x, S[j][2 * r], os[j][0]);
+            os[j][1] = fma2<PK>(qv.y, S[j][2 * r + 1], os[j][1]);
           }
         }
 #pragma unroll
@@ -2319,61 +2350,63 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
         continue;
       }
       const float c1 = fixed ? fixed_c1 : cf[tt * 4], c2 = fixed ? o.f0 : cf[tt * 4 + 1];
+      const f32x2 cc = pack2(c1, c1);
       if (delta) {
         // both products with the stored state in one pass and one round of shuffles: with S' = c1 S + k u^T,
         // S'^T q = c1 S^T q + u (k . q), and u = c2 (v - c1 S^T k); k . q comes with the token
 #pragma unroll
         for (int j = 0; j < CPT; ++j) {
-          float ks[4] = {0.f, 0.f, 0.f, 0.f};
-          float4 kv[RPT / 4];
+          f32x2 ks[2] = {0ull, 0ull};
+          ulonglong2 kv[RPT / 4];
 #pragma unroll
           for (int r = 0; r < RPT / 4; ++r) {
             kv[r] = k4[r];
-            const float4 qv = q4[r];
-            ks[0] = fmaf(kv[r].x, S[j][4 * r], ks[0]); ks[1] = fmaf(kv[r].y, S[j][4 * r + 1], ks[1]);
-            ks[2] = fmaf(kv[r].z, S[j][4 * r + 2], ks[2]); ks[3] = fmaf(kv[r].w, S[j][4 * r + 3], ks[3]);
-            os[j][0] = fmaf(qv.x, S[j][4 * r], os[j][0]); os[j][1] = fmaf(qv.y, S[j][4 * r + 1], os[j][1]);
-            os[j][2] = fmaf(qv.z, S[j][4 * r + 2], os[j][2]); os[j][3] = fmaf(qv.w, S[j][4 * r + 3], os[j][3]);
+            const ulonglong2 qv = q4[r];
+            ks[0] = fma2<PK>(kv[r].x, S[j][2 * r], ks[0]);
+            ks[1] = fma2<PK>(kv[r].y, S[j][2 * r + 1], ks[1]);
+            os[j][0] = fma2<PK>(qv.x, S[j][2 * r], os[j][0]);
+            os[j][1] = fma2<PK>(qv.y, S[j][2 * r + 1], os[j][1]);
           }
-          float kt = (ks[0] + ks[1]) + (ks[2] + ks[3]), qt = (os[j][0] + os[j][1]) + (os[j][2] + os[j][3]);
+          float kt = (lo2(ks[0]) + hi2(ks[0])) + (lo2(ks[1]) + hi2(ks[1])), qt = (lo2(os[j][0]) + hi2(os[j][0])) + (lo2(os[j][1]) + hi2(os[j][1]));
           kt += __shfl_xor_sync(0xffffffffu, kt, 1); qt += __shfl_xor_sync(0xffffffffu, qt, 1);
           kt += __shfl_xor_sync(0xffffffffu, kt, 2); qt += __shfl_xor_sync(0xffffffffu, qt, 2);
           kt += __shfl_xor_sync(0xffffffffu, kt, 4); qt += __shfl_xor_sync(0xffffffffu, qt, 4);
           const float u = c2 * (v[j] - c1 * kt);
+          const f32x2 uu = pack2(u, u);
 #pragma unroll
           for (int r = 0; r < RPT / 4; ++r) {
-            S[j][4 * r] = fmaf(kv[r].x, u, c1 * S[j][4 * r]); S[j][4 * r + 1] = fmaf(kv[r].y, u, c1 * S[j][4 * r + 1]);
-            S[j][4 * r + 2] = fmaf(kv[r].z, u, c1 * S[j][4 * r + 2]); S[j][4 * r + 3] = fmaf(kv[r].w, u, c1 * S[j][4 * r + 3]);
+            S[j][2 * r] = fma2<PK>(kv[r].x, uu, mul2<PK>(cc, S[j][2 * r]));
+            S[j][2 * r + 1] = fma2<PK>(kv[r].y, uu, mul2<PK>(cc, S[j][2 * r + 1]));
           }
           if (live[j] && sub == 0) orow[col[j]] = fmaf(u, cf[tt * 4 + 2], c1 * qt);
         }
         continue;
       }
-      float dx[CPT];
+      f32x2 dx[CPT];
 #pragma unroll
-      for (int j = 0; j < CPT; ++j) dx[j] = c2 * v[j];
+      for (int j = 0; j < CPT; ++j) { const float x = c2 * v[j]; dx[j] = pack2(x, x); }
       if (phase == 1) {
 #pragma unroll
         for (int r = 0; r < RPT / 4; ++r) {
-          const float4 bv = k4[r];
+          const ulonglong2 bv = k4[r];
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
-            S[j][4 * r] = fmaf(c1, S[j][4 * r], bv.x * dx[j]); S[j][4 * r + 1] = fmaf(c1, S[j][4 * r + 1], bv.y * dx[j]);
-            S[j][4 * r + 2] = fmaf(c1, S[j][4 * r + 2], bv.z * dx[j]); S[j][4 * r + 3] = fmaf(c1, S[j][4 * r + 3], bv.w * dx[j]);
+            S[j][2 * r] = fma2<PK>(cc, S[j][2 * r], mul2<PK>(bv.x, dx[j]));
+            S[j][2 * r + 1] = fma2<PK>(cc, S[j][2 * r + 1], mul2<PK>(bv.y, dx[j]));
           }
         }
-        Pd[0] *= c1;
+        Pd[0] = mul2<PK>(Pd[0], cc);
         continue;
       }
 #pragma unroll
       for (int r = 0; r < RPT / 4; ++r) {
-        const float4 bv = k4[r], qv = q4[r];
+        const ulonglong2 bv = k4[r], qv = q4[r];
 #pragma unroll
         for (int j = 0; j < CPT; ++j) {
-          S[j][4 * r] = fmaf(c1, S[j][4 * r], bv.x * dx[j]); S[j][4 * r + 1] = fmaf(c1, S[j][4 * r + 1], bv.y * dx[j]);
-          S[j][4 * r + 2] = fmaf(c1, S[j][4 * r + 2], bv.z * dx[j]); S[j][4 * r + 3] = fmaf(c1, S[j][4 * r + 3], bv.w * dx[j]);
-          os[j][0] = fmaf(qv.x, S[j][4 * r], os[j][0]); os[j][1] = fmaf(qv.y, S[j][4 * r + 1], os[j][1]);
-          os[j][2] = fmaf(qv.z, S[j][4 * r + 2], os[j][2]); os[j][3] = fmaf(qv.w, S[j][4 * r + 3], os[j][3]);
+          S[j][2 * r] = fma2<PK>(cc, S[j][2 * r], mul2<PK>(bv.x, dx[j]));
+          S[j][2 * r + 1] = fma2<PK>(cc, S[j][2 * r + 1], mul2<PK>(bv.y, dx[j]));
+          os[j][0] = fma2<PK>(qv.x, S[j][2 * r], os[j][0]);
+          os[j][1] = fma2<PK>(qv.y, S[j][2 * r + 1], os[j][1]);
         }
       }
 #pragma unroll
@@ -2397,11 +2430,11 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
 #pragma unroll
     for (int j = 0; j < CPT; ++j)
 #pragma unroll
-      for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live[j] && i < dk) nx[(size_t)i * sv + col[j]] = S[j][r]; }
+      for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live[j] && i < dk) nx[(size_t)i * sv + col[j]] = r & 1 ? hi2(S[j][r / 2]) : lo2(S[j][r / 2]); }
     if (blockIdx.x == 0 && cl == 0) {
       float* pz = P + ((size_t)zc * H + h) * dk;
 #pragma unroll
-      for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (i < dk) pz[i] = Pd[NV == 3 ? r : 0]; }
+      for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (i < dk) pz[i] = NV == 3 && (r & 1) ? hi2(Pd[NV == 3 ? r / 2 : 0]) : lo2(Pd[NV == 3 ? r / 2 : 0]); }
     }
     return;
   }
@@ -2410,7 +2443,7 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
 #pragma unroll
   for (int j = 0; j < CPT; ++j)
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live[j] && i < dk) nst[(size_t)i * sv + col[j]] = S[j][r]; }
+    for (int r = 0; r < RPT; ++r) { const int i = sub * RPT + r; if (live[j] && i < dk) nst[(size_t)i * sv + col[j]] = r & 1 ? hi2(S[j][r / 2]) : lo2(S[j][r / 2]); }
 }
 
 // grid (ceil(H * dk * sv / 256)), sv state columns: X[0] = the carried state; X[z + 1] = P[z] X[z] + X[z + 1] for the pieces in order.
