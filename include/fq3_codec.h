@@ -178,7 +178,7 @@ enum fq3c_kind {
    *   FQ3C_GNORM: bias (f32 [M, cin], one divisor per row and group), when given: the group is divided by it first; FQ3C_SIGMOID: the gate
    *     p1 is a sigmoid instead of a silu.
    *   FQ3C_SUM_NORM: norm_out without norm_w: the finished row itself.
-   *   FQ3C_ROT_APPEND: FQ3C_UNIT: heads are divided by their root mean square over i2 entries (eps f0), no weights (a rotation keeps it).
+   *   FQ3C_ROT_APPEND: p1 (f32 [taps / 2]), when given: what the frequencies B lost to rounding, added to the angle.  FQ3C_UNIT: heads are divided by their root mean square over i2 entries (eps f0), no weights (a rotation keeps it).
    *     m_begin = P > 0: every block of P positions bP .. bP + P - 1 that the step completes leaves the mean of its P rows of the caches
    *     as row b of norm_out (keys, pitch ldc) and ws (values, pitch ldr), in the caches' type.
    *   FQ3C_CACHE_ATTN: tap_off[1] = P > 0 (with a window K): C2 / norm_out = those pooled rows; beside its tokens, position i sees the

@@ -1425,6 +1425,7 @@ __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
   float* row = const_cast<float*>(reinterpret_cast<const float*>(o.A)) + (size_t)m * o.lda;
   const float* krow = o.res ? reinterpret_cast<const float*>(o.res) + (size_t)m * o.norm_ld : row;
   const float* freq = reinterpret_cast<const float*>(o.B);
+  const float* flo = reinterpret_cast<const float*>(o.p1);
   const float fp = (float)pos, amp = o.f1 != 0.f ? o.f1 : 1.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
   TC* kc = G > 0 ? reinterpret_cast<TC*>(o.C) + (size_t)pos * o.ldc : nullptr;
@@ -1444,8 +1445,13 @@ __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
     const bool halves = (o.flags & FQ3C_ROT_HALF) != 0;      // pairs (i, i + half) instead of (2i, 2i + 1)
     for (int i = lane; i < half; i += 32) {
       float sn, cs;
-      sincosf(fp * freq[i], &sn, &cs);
-      sn *= amp; cs *= amp;
+      const float ang = fp * freq[i];
+      sincosf(ang, &sn, &cs);
+      // what the product (and, with p1, the frequency) lost to rounding turns the pair a little further: at large angles it would show
+      float rest = fmaf(fp, freq[i], -ang);
+      if (flo) rest = fmaf(fp, flo[i], rest);
+      const float s1 = fmaf(cs, rest, sn), c1 = fmaf(-sn, rest, cs);
+      sn = s1 * amp; cs = c1 * amp;
       const int ia = halves ? i : 2 * i, ib = halves ? i + half : 2 * i + 1;
       float a = src[ia], b = src[ib];
       if (normed) { a *= rs; b *= rs; }

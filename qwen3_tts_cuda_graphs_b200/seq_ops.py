@@ -308,8 +308,8 @@ class StepBuilder:
     def softmax_attention(self, h: torch.Tensor, c: SoftmaxAttentionConfig, w: dict, kcache: str, vcache: str, out: torch.Tensor,
                           eps: float = 1e-6):
         """h [M, width] (product-operand dtype) -> out f32 [M, width].  w: wqkv [(H + 2G) dim.. (+ H gate rows), width] — queries, then
-        (unless the layer borrows a cache) keys and values, then the gate rows; bqkv f32 or None; freq f32 [rot_dims / 2] or None;
-        sink f32 [H] or None; r12 f32 [2H] or None; o [width, H * vdim]; o_b f32 or None; q_norm / k_norm f32 [dim] with qk_norm
+        (unless the layer borrows a cache) keys and values, then the gate rows; bqkv f32 or None; freq f32 [rot_dims / 2] or None (freq_lo: what its
+        entries lost to rounding, or None); sink f32 [H] or None; r12 f32 [2H] or None; o [width, H * vdim]; o_b f32 or None; q_norm / k_norm f32 [dim] with qk_norm
         (eps: their epsilon; qk_unit: no weights).  kcache / vcache name the slot's append states to write (own projections) and read;
         with pooled blocks (c.pool) kcache + ".pool" and vcache + ".pool" hold one row per complete block."""
         M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
@@ -326,6 +326,8 @@ class StepBuilder:
                       p0=self.slot.pos, flags=cf32)
             if c.rot_dims > 0:
                 kw["B"] = w["freq"]
+                if w.get("freq_lo") is not None:
+                    kw["p1"] = w["freq_lo"]
             if c.qk_norm:   # per-head norms in the same launch, before the rotation
                 kw.update(scale=w["q_norm"], bias=w["k_norm"], f0=float(eps))
             elif c.qk_unit:

@@ -104,8 +104,12 @@ class Packer:
 
     def attention(self, p: str, m: SoftmaxAttentionConfig) -> dict:
         w, b = self.stack(p, ("q", "k", "v", "g"), ("q", "k", "v"))
-        return {"wqkv": w, "bqkv": b, "o": self.W(self.raw(p + "o")), "o_b": None, "sink": None, "r12": None,
-                "freq": self.F(rotary_frequencies(m.rot_dims, m.rot_base, m.rot_factor)) if m.rot_dims > 0 else None}
+        d = {"wqkv": w, "bqkv": b, "o": self.W(self.raw(p + "o")), "o_b": None, "sink": None, "r12": None, "freq": None}
+        if m.rot_dims > 0:
+            f = rotary_frequencies(m.rot_dims, m.rot_base, m.rot_factor)
+            d["freq"] = self.F(f)
+            d["freq_lo"] = self.F(f - f.to(torch.float32).to(torch.float64))
+        return d
 
     def forget_gate(self, p: str) -> dict:
         w, b = self.stack(p, ("q", "f", "v"), ("f",))

@@ -448,6 +448,25 @@ def test_a_single_token_just_inside_and_just_outside_the_window(f32):
         assert float(row_errors(got, want).max()) < (TOL[True] if f32 else TOL[False]), portions
 
 
+def test_angles_stay_exact_thousands_of_positions_on():
+    """Scores of +-60 between keys that turn fast, 2400 positions in: an angle that is only as good as one 32-bit product (an error of
+    1e-4 at 2400 rad) would show tenfold above the tolerance, in the window and in the pooled keys far away."""
+    from qwen3_tts_cuda_graphs_b200.seq_state import StateSpec
+
+    H, G, d, dv, width, T, window, pool = 1, 1, 32, 8, 16, 2400, 40, 2
+    cfg = cases.config(8, width, [cases.layer(cases.attn(H, G, d, dv, window, pool, 2.0, 32, base=7.0, factor=0.7))])
+    W = sub_weights(cfg, "l0.mix.", seed=31)
+    torch.manual_seed(14)
+    h = bf(torch.randn(T, width))
+    want = so.attention(h.to(F64), {k: v.to(F64) for k, v in W.items()}, "", cfg["layers"][0]["mixer"], 1e-6)
+    c = layer_config(cfg).mixer
+    bench = Bench([StateSpec("k", "append", G * d), StateSpec("v", "append", G * dv),
+                   StateSpec("k.pool", "append", G * d, every=pool), StateSpec("v.pool", "append", G * dv, every=pool)], True, max_pos=T)
+    w = packer(W, True).attention("", c)
+    got = bench.portions(h, [2390, 2], lambda b, rows, out: b.softmax_attention(rows, c, w, "k", "v", out, eps=1e-6), width)
+    assert float(row_errors(got, want).max()) < 1e-4, float(row_errors(got, want).max())
+
+
 # ---------------------------------------------------------------------------------------------------------------------------
 # whole models
 # ---------------------------------------------------------------------------------------------------------------------------
