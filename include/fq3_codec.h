@@ -192,6 +192,23 @@ enum fq3c_kind {
    *     norm_out[row, h] (f32, pitch norm_ld) = max(|f0 n . q|, e^(-m')) + norm_eps, what the read-out is to be divided by.  The state p0 / C2
    *     is f32 [i0, i2, cin + 1] (column cin = n), the maxima are read from scale (f32 [i0]) and written to p1;
    *     ws = f32 [M, round_up(3 * i0, 4)].  Both: no workspace up to 16 rows; pieces as above, with states of cin + 1 columns for taps = 5.   */
+  /* ABI 11 adds to existing kinds:
+   *   FQ3C_GEMM / FQ3C_GGEMM: FQ3C_SWIGLU with FQ3C_GELU_TANH: the gated unit is gelu_tanh(w gate) * (w up).
+   *   FQ3C_GNORM: RESID with ldr = 0 adds the one row `res` to every row (a norm's bias).
+   *   FQ3C_SUM_NORM: bias (f32 [N]), when given, is added behind the norm's weights.  FQ3C_POST: C is the normed row instead of the sum
+   *     (a norm behind the residual sum); norm_out then is a copy of C in its own type and may be NULL.
+   *   FQ3C_TCONV: with FQ3C_SILU only columns from i0 on pass silu.
+   *   FQ3C_ROT_APPEND: f3 = E > 0: queries at position p are multiplied by 1 + f2 ln(floor((p + 1) / E) + 1).  The value heads may be
+   *     the key heads (a_rows = K, cin = i2): what is cached as values are the keys before norm and rotation.
+   *   FQ3C_CACHE_ATTN: FQ3C_GATE_ENTRY: res (f32 [M, col_mod]) holds a gate per output entry, head h at column h * cin; f2 != 0 multiplies
+   *     the output.
+   *   FQ3C_MSTATE_SCAN: taps = 6 (delta rule with a decay per key channel): rows A = queries of group g at column g * i2, keys at
+   *     K + g * i2, values of head h at a_rows + h * cin; raw rows res (f32, pitch ldr): decay latent (tap_off[0] entries) at column col_mod,
+   *     write-strength input of head h at m_begin + h;  z = B lat + bias with B [i0 * i2, tap_off[0]] (bf16; FQ3C_F32: f32), bias f32 [i0 * i2];
+   *       q, k <- unit vectors as for taps = 0;  g = exp(-exp(scale[h]) softplus(z)) per head and key channel;  beta = sigmoid(b);
+   *       S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  C = S^T q.
+   *     tap_off[2] = R > 0: a second up-projection in the same launch: norm_out (f32 [M, i0 * cin], pitch norm_ld) = p1 lat2 with p1
+   *     [i0 * cin, R] (B's type) and lat2 at column tap_off[1] of the rows res.  ws = f32 [M, round_up(2 * i1 * i2 + i0 * i2 + i0 + i1, 4)].  */
 };
 
 enum fq3c_flags {
@@ -214,7 +231,10 @@ enum fq3c_flags {
   FQ3C_CENTER = 262144  /* GNORM / SUM_NORM: subtract the mean, divide by the root of the variance (layer norm) */,
   FQ3C_ROT_HALF = 524288 /* ROT_APPEND: the turning pairs are (i, i + taps / 2) */,
   /* ABI 10 */
-  FQ3C_UNIT = 1048576   /* ROT_APPEND: heads are divided by their root mean square, no weights */
+  FQ3C_UNIT = 1048576   /* ROT_APPEND: heads are divided by their root mean square, no weights */,
+  /* ABI 11 */
+  FQ3C_POST = 2097152   /* SUM_NORM: C receives the normed row (a norm after the residual sum) */,
+  FQ3C_GATE_ENTRY = 4194304 /* CACHE_ATTN: res holds one gate per head and entry instead of one per head */
 };
 
 typedef struct fq3c_op {
@@ -248,6 +268,7 @@ typedef struct fq3c_op {
   const void* norm_w;
   int32_t norm_ld;
   float norm_eps;
+  float f2, f3;          /* ABI 11 */
 } fq3c_op;
 
 int fq3c_abi_version(void);

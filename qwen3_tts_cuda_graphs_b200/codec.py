@@ -42,6 +42,7 @@ F_GATE_PRE, F_GATE_POST = 16384, 32768
 F_RAW_WEIGHTS = 65536
 F_RELU2, F_CENTER, F_ROT_HALF = 131072, 262144, 524288
 F_UNIT = 1048576
+F_POST, F_GATE_ENTRY = 2097152, 4194304
 
 
 class Op(C.Structure):
@@ -53,7 +54,7 @@ class Op(C.Structure):
         ("A", C.c_void_p), ("B", C.c_void_p), ("bias", C.c_void_p), ("res", C.c_void_p), ("scale", C.c_void_p),
         ("p0", C.c_void_p), ("p1", C.c_void_p), ("C", C.c_void_p), ("C2", C.c_void_p),
         ("ws", C.c_void_p), ("ws_bytes", C.c_int64), ("m_begin", C.c_int32), ("reserved", C.c_int32),
-        ("norm_out", C.c_void_p), ("norm_w", C.c_void_p), ("norm_ld", C.c_int32), ("norm_eps", C.c_float),
+        ("norm_out", C.c_void_p), ("norm_w", C.c_void_p), ("norm_ld", C.c_int32), ("norm_eps", C.c_float), ("f2", C.c_float), ("f3", C.c_float),
     ]
 
 
@@ -151,7 +152,7 @@ def load_lib():
     lib.fq3c_graph_launch.argtypes = [C.c_void_p, C.c_void_p]
     lib.fq3c_graph_destroy.restype = C.c_int
     lib.fq3c_graph_destroy.argtypes = [C.c_void_p]
-    if lib.fq3c_abi_version() != 10:
+    if lib.fq3c_abi_version() != 11:
         raise CodecError("libfq3codec.so ABI version mismatch")
     _lib = lib
     return lib

@@ -379,6 +379,11 @@ class SoftmaxAttentionConfig:
     qk_unit: bool = False    # queries and keys are divided by their root mean square per head, no weights
     pool: int = 0            # > 0 (with a window): every block of this many positions that lies wholly before the window is seen
                              # as one more key and value, the means of its keys and of its values
+    rot_scaling: Optional[Tuple[float, float, float, float]] = None   # (factor, original, fast, slow): scaled rotary table
+    conv: int = 0            # > 0: taps of a causal convolution over time on every projected query, key and value channel
+    q_temp: Optional[Tuple[float, float]] = None   # (coef, every): queries at position p times 1 + coef ln(floor((p + 1) / every) + 1)
+    entry_gate: bool = False     # one sigmoid gate per entry of the concatenated heads
+    keys_as_values: bool = False     # the values are the projected keys, before norm and rotation (no value projection)
 
 
 @dataclass(frozen=True)
@@ -555,11 +560,26 @@ class RetentionConfig:
 
 
 @dataclass(frozen=True)
+class ChannelDeltaRuleConfig:
+    """Delta rule whose [dim, vdim] state per head decays per key channel and token (low-rank decay projection) before it is corrected
+    towards the new value along the new key; queries, keys and values pass a causal convolution and silu; the read-out is RMS-normed per
+    head, gated by a sigmoid per entry (low-rank) and projected."""
+
+    heads: int
+    kv_heads: int            # query / key heads
+    dim: int
+    vdim: int
+    conv: int                # taps of the causal convolution on q, k, v
+    decay_rank: int = 0      # inner sizes of the low-rank decay and gate projections; 0: whatever the checkpoint's tensors have
+    gate_rank: int = 0
+
+
+@dataclass(frozen=True)
 class ScaledPairMixerConfig:
     """Two mixers reading the same input; the result is left_scale * left + right_scale * right."""
 
     left: SoftmaxAttentionConfig
-    right: ChannelDecayAttentionConfig
+    right: object            # ChannelDecayAttentionConfig | ChannelDeltaRuleConfig
     left_scale: float
     right_scale: float
 
@@ -733,6 +753,67 @@ class SirodraConfig:
         return SirodraConfig(int(raw["vocab"]), int(raw["width"]), float((raw.get("norm") or {}).get("eps", 1e-6)), tuple(layers), loop)
 
 
+@dataclass(frozen=True)
+class MatidraConfig:
+    """Matidra: layer norms (weight and bias) behind the residual sums, x <- norm(alpha x + sublayer(x)); mixers in a configured order:
+    softmax attention with short convolutions, head norms, a query temperature and a gate per entry beside a delta rule with a decay per key
+    channel, or attention whose values are its projected keys, with head norms and a scaled rotary table; dense gated feed-forwards or none."""
+
+    architecture = "Matidra"
+    vocab: int
+    width: int
+    norm_eps: float
+    alpha: float             # multiplies the stream in every residual sum
+    layers: Tuple[SeqLayerConfig, ...]
+
+    @staticmethod
+    def from_dict(raw: dict) -> "MatidraConfig":
+        layers = []
+        for i, L in enumerate(raw["layers"]):
+            m, kind = L["mixer"], L["type"]
+            if kind == "parallel":
+                a, r = m["left"], m["right"]
+                t = a.get("q_temp")
+                att = SoftmaxAttentionConfig(int(a["heads"]), int(a.get("kv_heads", a["heads"])), int(a["dim"]), int(a["vdim"]), float(a["scale"]),
+                                             qk_norm=True, conv=int(a["conv"]), q_temp=(float(t["coef"]), float(t["every"])) if t else None,
+                                             entry_gate=True)
+                right = ChannelDeltaRuleConfig(int(r["heads"]), int(r.get("kv_heads", r["heads"])), int(r["dim"]), int(r["vdim"]), int(r["conv"]))
+                mixer = ScaledPairMixerConfig(att, right, float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0)))
+                if right.heads % right.kv_heads:
+                    raise ValueError(f"layer {i}: kv_heads must divide heads")
+                if not (1 <= att.conv <= 64 and 1 <= right.conv <= 64):
+                    raise ValueError(f"layer {i}: a convolution has 1 to 64 taps")
+                if att.q_temp is not None and not att.q_temp[1] > 0:
+                    raise ValueError(f"layer {i}: q_temp.every must be positive")
+            elif kind == "attention":
+                rot = m.get("rot") or {}
+                sc = rot.get("scaling")
+                mixer = att = SoftmaxAttentionConfig(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m.get("vdim", m["dim"])),
+                                                     float(m["scale"]), rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
+                                                     rot_scaling=(float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"])) if sc else None,
+                                                     qk_norm=True, keys_as_values=True)
+                if att.vdim != att.dim:
+                    raise ValueError(f"layer {i}: values that are keys have the keys' size")
+                if att.rot_dims % 2 or att.rot_dims > att.dim:
+                    raise ValueError(f"layer {i}: rot.dims must be even and at most dim")
+                if sc and not (float(sc["factor"]) > 0 and float(sc["original"]) > 0 and float(sc["fast"]) > 0 and float(sc["slow"]) > 0):
+                    raise ValueError(f"layer {i}: rot.scaling needs positive entries")
+            else:
+                raise ValueError(f"unknown mixer type {kind!r}")
+            if att.heads % att.kv_heads:
+                raise ValueError(f"layer {i}: kv_heads must divide heads")
+            f = L.get("mlp")
+            if f is None:
+                mlp = None
+            elif f.get("kind", "dense") == "dense":
+                mlp = DenseFFConfig(int(f["ff"]))
+            else:
+                raise ValueError(f"unknown feed-forward kind {f['kind']!r}")
+            layers.append(SeqLayerConfig(kind, mixer, mlp))
+        return MatidraConfig(int(raw["vocab"]), int(raw["width"]), float((raw.get("norm") or {}).get("eps", 1e-6)), float(raw.get("postln_alpha", 1.0)),
+                             tuple(layers))
+
+
 # config.json "architecture" -> (config class, "module:class" of the model that lowers it to op lists)
 SEQUENCE_ARCHITECTURES = {
     "Sidalorn": (SidalornConfig, "sidalorn:SidalornModel"),
@@ -740,6 +821,7 @@ SEQUENCE_ARCHITECTURES = {
     "Ratizen": (RatizenConfig, "ratizen:RatizenModel"),
     "Zudusun": (ZudusunConfig, "zudusun:ZudusunModel"),
     "Sirodra": (SirodraConfig, "sirodra:SirodraModel"),
+    "Matidra": (MatidraConfig, "matidra:MatidraModel"),
 }
 
 

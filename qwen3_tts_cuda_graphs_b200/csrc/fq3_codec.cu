@@ -48,7 +48,18 @@ constexpr int BM = 64, BN = 64, BK = 32, PAD = 8, LDS = BK + PAD;
 
 __device__ __forceinline__ float gelu_f(float x) { return 0.5f * x * (1.f + erff(x * 0.70710678118654752f)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+// a gated unit: silu(gate) * up, or with FQ3C_GELU_TANH gelu_tanh(gate) * up
+__device__ __forceinline__ float glu_f(const int flags, const float gate, const float up) {
+  return (flags & FQ3C_GELU_TANH) ? gelu_tanh_f(gate) * up : silu_f(gate) * up;
+}
 
+__device__ __forceinline__ void stf_any(const fq3c_op& o, const size_t at, const float v) {
+  if (o.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(o.C)[at] = v;
+  else reinterpret_cast<bf16*>(o.C)[at] = __float2bfloat16_rn(v);
+}
 // Epilogue for one (row, even col) pair of accumulators; order documented in include/fq3_codec.h / DESIGN.md §5.
 __device__ __forceinline__ void epilogue_pair(const fq3c_op& o, int row, int col, float v0, float v1) {
   if (row >= o.M || col >= o.N) return;
@@ -65,6 +76,10 @@ __device__ __forceinline__ void epilogue_pair(const fq3c_op& o, int row, int col
     v1 = bf16r(v1);
   }
   if (o.flags & FQ3C_SWIGLU) {  // interleaved (gate, up) columns -> one output column
+    if (o.flags & FQ3C_NOROUND) {
+      if (has1) stf_any(o, (size_t)row * o.ldc + (col >> 1), glu_f(o.flags, v0, v1));
+      return;
+    }
     const float y = bf16r(bf16r(silu_f(v0)) * v1);
     reinterpret_cast<bf16*>(o.C)[(size_t)row * o.ldc + (col >> 1)] = __float2bfloat16_rn(y);
     return;
@@ -140,6 +155,18 @@ __device__ __forceinline__ void epilogue_row8(const fq3c_op& o, int row, int col
     float4* c = reinterpret_cast<float4*>(reinterpret_cast<float*>(o.C) + (size_t)row * o.ldc + col);
     c[0] = make_float4(v[0], v[1], v[2], v[3]);
     c[1] = make_float4(v[4], v[5], v[6], v[7]);
+    return;
+  }
+  // a gated unit on the unrounded sums: four outputs, one 8-byte store
+  if ((o.flags & FQ3C_SWIGLU) && (o.flags & FQ3C_NOROUND) && !(o.flags & ~(FQ3C_SWIGLU | FQ3C_NOROUND | FQ3C_GELU_TANH)) && col + 8 <= o.N &&
+      (o.ldc & 3) == 0 && !(reinterpret_cast<uintptr_t>(o.C) & 7)) {
+    if (row >= o.M) return;
+    float v[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = glu_f(o.flags, acc[2 * j], acc[2 * j + 1]);
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(o.C) + (size_t)row * o.ldc + (col >> 1)) =
+        make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
     return;
   }
   const bool vec = (col + 8 <= o.N) && !(o.flags & (FQ3C_SWIGLU | FQ3C_OUT_F32)) && ((o.ldc & 7) == 0) &&
@@ -1034,7 +1061,7 @@ int launch_seq_gemm(const SeqGemm& g, bool a_f32, bool b_f32, bool exact, int zc
   if (g.flags & ~SEQ_GEMM_FLAGS) return fail("sequence product: unsupported epilogue flag");
   if (b_f32 && !a_f32) return fail("sequence product: f32 weights need f32 rows");
   if (g.M <= 0 || g.N <= 0 || g.K <= 0 || zcount <= 0) return 0;
-  if ((g.flags & FQ3C_SWIGLU) && ((g.N & 1) || (g.flags & (FQ3C_BIAS | FQ3C_GELU | FQ3C_GELU_TANH | FQ3C_SIGMOID | FQ3C_RELU2)) || zcount != 1))
+  if ((g.flags & FQ3C_SWIGLU) && ((g.N & 1) || (g.flags & (FQ3C_BIAS | FQ3C_GELU | FQ3C_SIGMOID | FQ3C_RELU2)) || zcount != 1))
     return fail("sequence product: a gated-unit epilogue takes an even number of alternating gate / up columns and no other epilogue");
   const size_t gemv_smem = (size_t)g.M * g.K * sizeof(float);
   if (!g.seg && g.M <= 8 && gemv_smem <= 96 * 1024) {
@@ -1093,6 +1120,13 @@ int launch_seq_gemm(const SeqGemm& g, bool a_f32, bool b_f32, bool exact, int zc
 // threads of a block that works on one row of n entries: with a few rows (decoding) one per entry, so that the row's loads are one round trip
 int row_threads(int rows, int n, int many) { return rows <= 8 ? std::max(32, std::min(1024, (n + 31) / 32 * 32)) : many; }
 
+// the convolution over many rows of whole 16-byte pieces: four columns and TC_ROWS rows per thread
+bool tconv_vec_ok(const fq3c_op& o) {
+  return o.M >= 64 && o.taps > 1 && o.taps <= 8 && o.N % 4 == 0 && o.lda % 4 == 0 && o.ldc % 4 == 0 && !(o.flags & FQ3C_RESID) &&
+         !((reinterpret_cast<uintptr_t>(o.A) | reinterpret_cast<uintptr_t>(o.C) | reinterpret_cast<uintptr_t>(o.p0) | reinterpret_cast<uintptr_t>(o.p1)) & 15) &&
+         (!(o.flags & FQ3C_SILU) || o.i0 % 4 == 0);
+}
+
 // returns 1 when the kind is not a sequence-model op
 int seq_run(const fq3c_op& o, cudaStream_t s) {
   switch (o.kind) {
@@ -1105,6 +1139,12 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       return 0;
     case FQ3C_TCONV:
       if (o.taps < 1 || !o.A || !o.B || !o.C || (o.taps > 1 && (!o.p0 || !o.p1))) return fail("tconv: missing operand");
+      if (tconv_vec_ok(o)) {
+        const dim3 grid((o.N / 4 + 127) / 128, (o.M + o.taps - 1 + TC_ROWS - 1) / TC_ROWS);
+        if (o.taps <= 4) fq3s_tconv_vec_kernel<4><<<grid, 128, 0, s>>>(o);
+        else fq3s_tconv_vec_kernel<8><<<grid, 128, 0, s>>>(o);
+        return 0;
+      }
       fq3s_tconv_kernel<<<dim3((o.N + 255) / 256, o.M + o.taps - 1), 256, 0, s>>>(o);
       return 0;
     case FQ3C_GNORM:
@@ -1367,9 +1407,9 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       return 0;
     case FQ3C_MSTATE_SCAN: {
       if (o.i0 < 1 || o.i1 < 1 || o.i0 % o.i1 || o.i2 < 1 || o.cin < 1 || !o.A || !o.p0 || !o.C || !o.C2) return fail("mstate_scan: bad configuration");
-      if (o.taps < 0 || o.taps > 5)
+      if (o.taps < 0 || o.taps > 6)
         return fail("mstate_scan: taps selects the delta rule (0), the state-space scan (1), a decay per key channel (2), a fixed decay per head (3), a forget gate "
-                    "per channel (4) or exponential gates (5)");
+                    "per channel (4), exponential gates (5) or the delta rule with a decay per key channel (6)");
       if (o.i2 > 512) return fail("mstate_scan: at most 512 state rows per head");
       if (o.taps <= 1) {
         if (!o.res || !o.scale || !o.ws) return fail("mstate_scan: raw projections, A_log and a workspace required");
@@ -1378,6 +1418,11 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         if (!o.res || !o.ws || !o.B || o.i1 != o.i0 || o.m_begin < 1 || o.m_begin > MS_MAX_RANK)
           return fail("mstate_scan: channel decays need their latent rows, the up-projection (inner size 1 .. 1024), a workspace and one key head per head");
         if (o.ws_bytes < (int64_t)o.M * mstate_decay_cols(o.i0, o.i2) * 4) return fail("mstate_scan: workspace too small");
+      } else if (o.taps == 6) {
+        if (!o.res || !o.ws || !o.B || !o.scale || !o.bias || o.tap_off[0] < 1 || o.tap_off[0] > MS_MAX_RANK || o.tap_off[2] < 0 || o.tap_off[2] > MS_MAX_RANK ||
+            (o.tap_off[2] > 0 && (!o.p1 || !o.norm_out || o.norm_ld < o.i0 * o.cin)))
+          return fail("mstate_scan: channel decays of the delta rule need their latent rows, the up-projections (inner sizes 1 .. 1024), A_log, dt_bias and a workspace");
+        if (o.ws_bytes < (int64_t)o.M * mstate_cdelta_cols(o.i0, o.i1, o.i2) * 4) return fail("mstate_scan: workspace too small");
       } else if (o.taps == 3) {
         if (!o.scale || o.i1 != o.i0) return fail("mstate_scan: fixed decays need one value and one key head per head");
       } else {
@@ -1391,6 +1436,12 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         count_launches(1);
       } else if (o.taps == 5 && o.M > MS_CH) {
         fq3s_mstate_max_kernel<<<o.i0, MM_THREADS, 0, s>>>(o);
+        count_launches(1);
+      } else if (o.taps == 6) {
+        const dim3 grid((o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS, (o.i0 * o.i2 + 255) / 256 + (o.tap_off[2] > 0 ? (o.i0 * o.cin + 255) / 256 : 0) + 1);
+        const size_t smem = sizeof(float) * MS_PREP_ROWS * (size_t)std::max(o.tap_off[0], o.tap_off[2]);
+        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, 256, smem, s>>>(o);
+        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, 256, smem, s>>>(o);
         count_launches(1);
       } else if (o.taps < 3) {
         fq3s_mstate_prep_kernel<<<o.taps == 2 ? (o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS : o.M, 128, 0, s>>>(o);
@@ -1410,6 +1461,9 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32, 3, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 216 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 3, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 216 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<16, 3, false, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 72 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32, 3, false, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
+        cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 3, false, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 216 * 1024);
         sattr[dev] = true;
       }
       // Long runs of a recurrence whose decays do not depend on the state: pieces walked twice (see the kernel), when the caller's
@@ -1420,7 +1474,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       const int64_t base = ((int64_t)o.M * coef + 3) & ~(int64_t)3;
       const int64_t per_piece = (int64_t)o.i0 * o.i2 * (sv + 1);
       int pieces = 1, piece = o.M;
-      if (o.taps != 0 && o.M >= 512 && o.ws) {
+      if (o.taps != 0 && o.taps != 6 && o.M >= 512 && o.ws) {
         pieces = (int)std::min<int64_t>(std::min(16, o.M / 128), (o.ws_bytes / 4 - base) / per_piece);
         if (pieces >= 2) {
           piece = (((o.M + pieces - 1) / pieces) + MS_CH - 1) / MS_CH * MS_CH;
@@ -1431,7 +1485,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       float* X = pieces > 1 ? reinterpret_cast<float*>(o.ws) + base : nullptr;
       float* P = pieces > 1 ? X + (int64_t)pieces * o.i0 * o.i2 * sv : nullptr;
       const int bound = o.i2 <= 32 ? 4 : o.i2 <= 64 ? 8 : o.i2 <= 128 ? 16 : o.i2 <= 256 ? 32 : 64;      // state rows a lane holds
-      const bool three = o.taps == 2 || o.taps == 4, gated = o.taps >= 4;
+      const bool cdelta = o.taps == 6, three = o.taps == 2 || o.taps == 4 || cdelta, gated = o.taps == 4 || o.taps == 5;
       const int cpt = pieces > 1 && bound <= 16 ? 2 : 1;                                                    // state columns a lane holds
       auto walk = [&](const int phase, const int nz) {
         const dim3 grid((sv + cpt * MS_COLS - 1) / (cpt * MS_COLS), o.i0, nz);
@@ -1441,7 +1495,14 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
     else if (three) fq3s_mstate_scan_kernel<RPT, 3, false, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
     else if (gated) fq3s_mstate_scan_kernel<RPT, 2, true, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P); \
     else fq3s_mstate_scan_kernel<RPT, 2, false, CPT><<<grid, 128, smem, s>>>(o, phase, piece, X, P);
-        if (cpt == 2) switch (bound) {
+        if (cdelta) switch (bound) {
+          case 4: fq3s_mstate_scan_kernel<4, 3, false, 1, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); break;
+          case 8: fq3s_mstate_scan_kernel<8, 3, false, 1, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); break;
+          case 16: fq3s_mstate_scan_kernel<16, 3, false, 1, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); break;
+          case 32: fq3s_mstate_scan_kernel<32, 3, false, 1, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); break;
+          default: fq3s_mstate_scan_kernel<64, 3, false, 1, true><<<grid, 128, smem, s>>>(o, phase, piece, X, P); break;
+        }
+        else if (cpt == 2) switch (bound) {
           case 4: FQ3S_WALK(4, 2) break;
           case 8: FQ3S_WALK(8, 2) break;
           default: FQ3S_WALK(16, 2) break;
@@ -1467,7 +1528,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       return 0;
     }
     case FQ3C_SUM_NORM: {
-      if (o.i0 < 1 || !o.A || !o.p0 || !o.C || (o.i0 > 1 && o.K < o.N)) return fail("sum_norm: missing operand");
+      if (o.i0 < 1 || !o.A || !o.p0 || !o.C || (o.i0 > 1 && o.K < o.N) || ((o.flags & FQ3C_POST) && (!o.norm_w || o.C2))) return fail("sum_norm: missing operand");
       if ((size_t)o.N * 4 > 200 * 1024) return fail("sum_norm: row too wide for shared memory");
       static bool nattr[64] = {};
       int dev = 0;
@@ -1478,7 +1539,8 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       }
       // rows of whole 16-byte pieces that a block of 256 holds in registers
       if (o.N % 4 == 0 && o.N <= 1024 * SN_VECS && !((o.lda | o.ldc | o.norm_ld | o.K) & 3) && !o.C2 &&
-          !((reinterpret_cast<uintptr_t>(o.A) | reinterpret_cast<uintptr_t>(o.C) | reinterpret_cast<uintptr_t>(o.norm_out) | reinterpret_cast<uintptr_t>(o.norm_w)) & 15)) {
+          !((reinterpret_cast<uintptr_t>(o.A) | reinterpret_cast<uintptr_t>(o.C) | reinterpret_cast<uintptr_t>(o.norm_out) | reinterpret_cast<uintptr_t>(o.norm_w) |
+            reinterpret_cast<uintptr_t>(o.bias)) & 15)) {
         fq3s_sum_norm_vec_kernel<<<o.M, std::max(32, std::min(256, (o.N / 4 + 31) / 32 * 32)), 0, s>>>(o);
         return 0;
       }
@@ -1493,7 +1555,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
 
 extern "C" {
 
-int fq3c_abi_version(void) { return 10; }
+int fq3c_abi_version(void) { return 11; }
 const char* fq3c_last_error(void) { return g_err.c_str(); }
 int64_t fq3c_launch_count(void) { return g_launches.load(); }
 

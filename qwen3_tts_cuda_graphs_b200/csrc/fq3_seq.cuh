@@ -10,9 +10,6 @@ template <> __device__ __forceinline__ float ldf<bf16>(const bf16* p) { return _
 __device__ __forceinline__ void stf(float* p, float v) { *p = v; }
 __device__ __forceinline__ void stf(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
@@ -48,7 +45,7 @@ struct SeqGemm {
   int a_mod, a_zstride, c_zstride; long long b_zstride;   // grid.z: A columns (z % a_mod) * a_zstride, B + z * b_zstride, C columns z * c_zstride
   const int* seg; const int* rows; int E; long long b_estride;
   // FQ3C_SWIGLU: the weight rows alternate (gate_n, up_n), so columns (2n, 2n + 1) of the product are one gated unit and the output
-  // is C[r, n] = silu(w gate) * (w up), N / 2 columns wide.  w = 1, or rs_w[r], or (rs_pos given: a router's choices) the weight
+  // is C[r, n] = silu(w gate) * (w up) (FQ3C_GELU_TANH: gelu_tanh(w gate) * (w up)), N / 2 columns wide.  w = 1, or rs_w[r], or (rs_pos given: a router's choices) the weight
   // rs_w[m, j] of the choice j of token m = rows[r] whose sorted position rs_pos[m, j] is r.
   const float* rs_w; const int* rs_pos; int rs_top;
 };
@@ -62,8 +59,7 @@ __device__ __forceinline__ float sg_row_scale(const SeqGemm& g, const int r) {
 }
 __device__ __forceinline__ void sg_store_glu(const SeqGemm& g, const int r, const int ccol, const int n_even, const float gate, const float up,
                                              const float w) {
-  const float a = w * gate, b = w * up;
-  const float v = a / (1.f + expf(-a)) * b;
+  const float v = glu_f(g.flags, w * gate, w * up);
   const size_t ci = (size_t)r * g.ldc + ccol + (n_even >> 1);
   if (g.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(g.C)[ci] = v;
   else reinterpret_cast<bf16*>(g.C)[ci] = __float2bfloat16_rn(v);
@@ -646,9 +642,66 @@ __global__ void __launch_bounds__(256) fq3s_tconv_kernel(const fq3c_op o) {
     a = fmaf(w[j], v, a);
   }
   if (o.flags & FQ3C_RESID) a += x[(size_t)m * o.lda + c];
-  if (o.flags & FQ3C_SILU) a = a / (1.f + expf(-a));
+  if ((o.flags & FQ3C_SILU) && c >= o.i0) a = a / (1.f + expf(-a));
   if (o.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(o.C)[(size_t)m * o.ldc + c] = a;
   else reinterpret_cast<bf16*>(o.C)[(size_t)m * o.ldc + c] = __float2bfloat16_rn(a);
+}
+
+// The same for many rows of whole 16-byte pieces: a thread takes four columns of TC_ROWS consecutive rows and keeps the last TAPS inputs in
+// registers, so that an input is loaded once.  TAPS >= o.taps: the taps in front are zero.  Rows M .. M + taps - 2 are the next history.
+// grid (ceil(N / 512), ceil((M + taps - 1) / TC_ROWS)), 128 threads.
+constexpr int TC_ROWS = 8;
+template <int TAPS>
+__global__ void __launch_bounds__(128) fq3s_tconv_vec_kernel(const fq3c_op o) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= o.N) return;
+  const int h = o.taps - 1, m0 = blockIdx.y * TC_ROWS;
+  const float* x = reinterpret_cast<const float*>(o.A) + c;
+  const float* hist = reinterpret_cast<const float*>(o.p0) + c;
+  auto input = [&](const int pos) {       // pos in [-h, M); beyond: not used
+    if (pos < -h || pos >= o.M) return make_float4(0.f, 0.f, 0.f, 0.f);
+    return *reinterpret_cast<const float4*>(pos >= 0 ? x + (size_t)pos * o.lda : hist + (size_t)(h + pos) * o.N);
+  };
+  float w[4][TAPS];
+#pragma unroll
+  for (int e = 0; e < 4; ++e)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const int t = j - (TAPS - o.taps);
+      w[e][j] = t >= 0 ? reinterpret_cast<const float*>(o.B)[(size_t)(c + e) * o.taps + t] : 0.f;
+    }
+  float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (o.flags & FQ3C_BIAS) { const float* bp = reinterpret_cast<const float*>(o.bias) + c; b = make_float4(bp[0], bp[1], bp[2], bp[3]); }
+  const bool act = (o.flags & FQ3C_SILU) && c >= o.i0;
+  float4 v[TAPS + TC_ROWS - 1];      // v[i] = input at position m0 + i - (TAPS - 1)
+#pragma unroll
+  for (int i = 0; i < TAPS + TC_ROWS - 1; ++i) v[i] = input(m0 + i - (TAPS - 1));
+#pragma unroll
+  for (int r = 0; r < TC_ROWS; ++r) {
+    const int m = m0 + r;
+    if (m >= o.M + h) return;
+    if (m >= o.M) {       // next history row s holds the input at M - h + s = m - h
+      const int s = m - o.M, pos = m - h;
+      *reinterpret_cast<float4*>(reinterpret_cast<float*>(const_cast<void*>(o.p1)) + (size_t)s * o.N + c) = input(pos);
+      continue;
+    }
+    float a[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const float4 u = v[r + j];
+      a[0] = fmaf(w[0][j], u.x, a[0]); a[1] = fmaf(w[1][j], u.y, a[1]); a[2] = fmaf(w[2][j], u.z, a[2]); a[3] = fmaf(w[3][j], u.w, a[3]);
+    }
+    if (act) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) a[e] = a[e] / (1.f + expf(-a[e]));
+    }
+    if (o.flags & FQ3C_OUT_F32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(o.C) + (size_t)m * o.ldc + c) = make_float4(a[0], a[1], a[2], a[3]);
+    else {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1]), hi = __floats2bfloat162_rn(a[2], a[3]);
+      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(o.C) + (size_t)m * o.ldc + c) =
+          make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+  }
 }
 
 // grid (M, groups); one block per (row, group): 128 threads, or up to 1024 for a few rows (decoding).  FQ3C_CENTER: mean and variance instead of the mean square.  An optional silu gate (p1, pitch i1;
@@ -1427,19 +1480,22 @@ __global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
   const float* freq = reinterpret_cast<const float*>(o.B);
   const float* flo = reinterpret_cast<const float*>(o.p1);
   const float fp = (float)pos, amp = o.f1 != 0.f ? o.f1 : 1.f;
+  // query temperature: grows with every f3 positions (the quotient of two integers below 2^24 never rounds up to the next integer)
+  const float temp = o.f3 > 0.f ? fmaf(o.f2, logf(floorf((fp + 1.f) / o.f3) + 1.f), 1.f) : 1.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
   TC* kc = G > 0 ? reinterpret_cast<TC*>(o.C) + (size_t)pos * o.ldc : nullptr;
   for (int hh = warp; hh < H + G; hh += nwarp) {
     const bool isq = hh < H;
     const float* src = isq ? row + (size_t)hh * d : krow + o.K + (size_t)(hh - H) * d;
     const float* nw = reinterpret_cast<const float*>(isq ? o.scale : o.bias);
-    const bool normed = nw || (o.flags & FQ3C_UNIT);
+    const bool unit = nw || (o.flags & FQ3C_UNIT), normed = unit || (isq && o.f3 > 0.f);
     float rs = 1.f;
-    if (normed) {
+    if (unit) {
       float ss = 0.f;
       for (int c = lane; c < d; c += 32) ss = fmaf(src[c], src[c], ss);
       rs = 1.f / sqrtf(warp_sum(ss) / (float)d + o.f0);
     }
+    if (isq) rs *= temp;
     float* qd = isq ? row + (size_t)hh * d : nullptr;
     TC* kd = isq ? nullptr : kc + (size_t)(hh - H) * d;
     const bool halves = (o.flags & FQ3C_ROT_HALF) != 0;      // pairs (i, i + half) instead of (2i, 2i + 1)
@@ -1634,6 +1690,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_kernel(const fq3c_op o, c
   __syncthreads();
   const float* sink = reinterpret_cast<const float*>(o.scale);
   const float* gate = reinterpret_cast<const float*>(o.res);
+  const bool entry = (o.flags & FQ3C_GATE_ENTRY) != 0;
   for (int idx = tid; idx < R * dv; idx += blockDim.x) {
     const int r = idx / dv, c = idx - r * dv, qi = r / HG, h = g * HG + (r - qi * HG), m = m0 + qi;
     if (qi >= nq) continue;
@@ -1650,7 +1707,8 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_kernel(const fq3c_op o, c
       den = den * f + expf(sink[h] - mm);
     }
     float v = oa[idx] * f / den;
-    if (gate) v *= sigmoid_f(gate[(size_t)m * o.col_mod + h]);
+    if (gate) v *= sigmoid_f(gate[(size_t)m * o.col_mod + (entry ? h * dv + c : h)]);
+    if (o.f2 != 0.f) v *= o.f2;
     if (o.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(o.C)[(size_t)m * o.ldc + (size_t)h * dv + c] = v;
     else reinterpret_cast<bf16*>(o.C)[(size_t)m * o.ldc + (size_t)h * dv + c] = __float2bfloat16_rn(v);
   }
@@ -1675,13 +1733,16 @@ __global__ void __launch_bounds__(128) fq3s_cache_attn_merge_kernel(const fq3c_o
   if ((int)threadIdx.x < splits) wsm[threadIdx.x] = w;
   float den = seq_block_sum(w * lv, red);
   if (sink) den += expf(sink[h] - mm);
-  const float gate = o.res ? sigmoid_f(reinterpret_cast<const float*>(o.res)[(size_t)m * o.col_mod + h]) : 1.f;
-  const float sc = gate / den;
+  const bool entry = (o.flags & FQ3C_GATE_ENTRY) != 0;
+  const float* gr = o.res ? reinterpret_cast<const float*>(o.res) + (size_t)m * o.col_mod : nullptr;
+  const float gate = (gr && !entry) ? sigmoid_f(gr[h]) : 1.f;
+  const float sc = gate * (o.f2 != 0.f ? o.f2 : 1.f) / den;
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
     float acc = 0.f;
 #pragma unroll 8
     for (int s = 0; s < splits; ++s) acc = fmaf(wsm[s], src[(size_t)s * (dv + 2) + 2 + c], acc);
-    const float v = acc * sc;
+    float v = acc * sc;
+    if (entry) v *= sigmoid_f(gr[(size_t)h * dv + c]);
     if (o.flags & FQ3C_OUT_F32) reinterpret_cast<float*>(o.C)[(size_t)m * o.ldc + (size_t)h * dv + c] = v;
     else reinterpret_cast<bf16*>(o.C)[(size_t)m * o.ldc + (size_t)h * dv + c] = __float2bfloat16_rn(v);
   }
@@ -1920,6 +1981,7 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
   }
   const float* sink = reinterpret_cast<const float*>(o.scale);
   const float* gate = reinterpret_cast<const float*>(o.res);
+  const bool entry = gate && (o.flags & FQ3C_GATE_ENTRY);
 #pragma unroll
   for (int hf = 0; hf < 2; ++hf) {
     if (!live[hf]) continue;
@@ -1931,12 +1993,15 @@ __global__ void __launch_bounds__(256) fq3s_cache_attn_mma_kernel(const fq3c_op 
       den = den * f + expf(sink[h] - mm);
     }
     float sc = f / den;
-    if (gate) sc *= sigmoid_f(gate[(size_t)m * o.col_mod + h]);
+    if (gate && !entry) sc *= sigmoid_f(gate[(size_t)m * o.col_mod + h]);
+    if (o.f2 != 0.f) sc *= o.f2;
+    const float* ge = entry ? gate + (size_t)m * o.col_mod + (size_t)h * dv : nullptr;
     const size_t at = (size_t)m * o.ldc + (size_t)h * dv;
 #pragma unroll
     for (int nt = 0; nt < NTM; ++nt) {
       if (nt >= nt_o) continue;
-      const float v0 = oacc[nt][hf * 2] * sc, v1 = oacc[nt][hf * 2 + 1] * sc;
+      float v0 = oacc[nt][hf * 2] * sc, v1 = oacc[nt][hf * 2 + 1] * sc;
+      if (entry) { v0 *= sigmoid_f(ge[nt * 8 + t * 2]); v1 *= sigmoid_f(ge[nt * 8 + t * 2 + 1]); }
       if (o.flags & FQ3C_OUT_F32) { reinterpret_cast<float*>(o.C)[at + nt * 8 + t * 2] = v0; reinterpret_cast<float*>(o.C)[at + nt * 8 + t * 2 + 1] = v1; }
       else *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf16*>(o.C) + at + nt * 8 + t * 2) = __floats2bfloat162_rn(v0, v1);
     }
@@ -2041,6 +2106,104 @@ __global__ void __launch_bounds__(128) fq3s_mstate_prep_kernel(const fq3c_op o) 
     for (int c = lane; c < dk; c += 32) dot = fmaf(qn[c], kn[c], dot);
     dot = warp_sum(dot);
     if (lane == 0) cf[2 * H + g] = dot;
+  }
+}
+
+// mode 6: ws row m = unit q [G * dk] | unit k [G * dk] | decays [H * dk] | write strengths [H] | q.k [G].  A block takes MS_PREP_ROWS rows (ROWS:
+// how many of them it computes, 1 in decoding) and one share of the columns (grid.y): 256 channels of the decays' up-projection, 256 channels of
+// the gate's, or, the last one, the unit vectors with their products and the write strengths.  A row of an up-projection is loaded once for all
+// rows of the block, whose latents lie transposed in shared memory (sixteen-byte broadcasts).  Dynamic shared memory: 8 x the larger inner size.
+__host__ __device__ inline int mstate_cdelta_cols(int H, int G, int dk) { return ((2 * G + H) * dk + H + G + 3) & ~3; }
+template <int ROWS>
+__device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, const void* U, const int c, const int R, float (&z)[ROWS]) {
+#pragma unroll
+  for (int j = 0; j < ROWS; ++j) z[j] = 0.f;
+  auto add = [&](const float uv, const int r) {
+    if (ROWS == 8) {
+      const float4 a = *reinterpret_cast<const float4*>(lat + r * 8), b = *reinterpret_cast<const float4*>(lat + r * 8 + 4);
+      const float l[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int j = 0; j < ROWS; ++j) z[j] = fmaf(l[j], uv, z[j]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < ROWS; ++j) z[j] = fmaf(lat[r * 8 + j], uv, z[j]);
+    }
+  };
+  if (o.flags & FQ3C_F32) {
+    const float* u = reinterpret_cast<const float*>(U) + (size_t)c * R;
+#pragma unroll 4
+    for (int r = 0; r < R; ++r) add(u[r], r);
+    return;
+  }
+  const bf16* u = reinterpret_cast<const bf16*>(U) + (size_t)c * R;
+  if (R % 8 == 0 && !(reinterpret_cast<uintptr_t>(U) & 15)) {
+#pragma unroll 2
+    for (int r = 0; r < R; r += 8) {
+      const uint4 p = __ldg(reinterpret_cast<const uint4*>(u + r));
+      const uint32_t w[4] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+      for (int q = 0; q < 4; ++q) { add(__uint_as_float(w[q] << 16), r + 2 * q); add(__uint_as_float(w[q] & 0xffff0000u), r + 2 * q + 1); }
+    }
+  } else {
+    for (int r = 0; r < R; ++r) add(__bfloat162float(u[r]), r);
+  }
+}
+template <int ROWS>
+__global__ void __launch_bounds__(256) fq3s_mstate_cdelta_prep_kernel(const fq3c_op o) {
+  extern __shared__ __align__(16) float cd_lat[];       // [inner size][8]
+  const int H = o.i0, G = o.i1, dk = o.i2, m0 = blockIdx.x * MS_PREP_ROWS, nr = min(ROWS, o.M - m0), tid = threadIdx.x;
+  const int nd = (H * dk + 255) / 256, ng = o.tap_off[2] > 0 ? (H * o.cin + 255) / 256 : 0, y = blockIdx.y;
+  const int cols = mstate_cdelta_cols(H, G, dk);
+  const float* raw = reinterpret_cast<const float*>(o.res) + (size_t)m0 * o.ldr;
+  float* w = reinterpret_cast<float*>(o.ws) + (size_t)m0 * cols;
+  if (y < nd + ng) {
+    const bool decay = y < nd;
+    const int R = o.tap_off[decay ? 0 : 2], lcol = decay ? o.col_mod : o.tap_off[1], c = (decay ? y : y - nd) * 256 + tid;
+    for (int i = tid; i < ROWS * R; i += 256) {
+      const int j = i / R, r = i - j * R;
+      cd_lat[r * 8 + j] = j < nr ? raw[(size_t)j * o.ldr + lcol + r] : 0.f;
+    }
+    __syncthreads();
+    float z[ROWS];
+    if (decay) {
+      if (c >= H * dk) return;
+      cdelta_up<ROWS>(o, cd_lat, o.B, c, R, z);
+      const float db = reinterpret_cast<const float*>(o.bias)[c], rate = expf(reinterpret_cast<const float*>(o.scale)[c / dk]);
+#pragma unroll
+      for (int j = 0; j < ROWS; ++j)
+        if (j < nr) w[(size_t)j * cols + 2 * G * dk + c] = expf(-rate * softplus_f(z[j] + db));
+    } else {
+      if (c >= H * o.cin) return;
+      cdelta_up<ROWS>(o, cd_lat, o.p1, c, R, z);
+      float* gr = reinterpret_cast<float*>(o.norm_out) + (size_t)m0 * o.norm_ld + c;
+#pragma unroll
+      for (int j = 0; j < ROWS; ++j)
+        if (j < nr) gr[(size_t)j * o.norm_ld] = z[j];
+    }
+    return;
+  }
+  float* cf = w + (2 * G + H) * dk;
+  for (int i = tid; i < nr * H; i += 256) {
+    const int j = i / H, h = i - j * H;
+    cf[(size_t)j * cols + h] = sigmoid_f(raw[(size_t)j * o.ldr + o.m_begin + h]);
+  }
+  const int warp = tid >> 5, lane = tid & 31;
+  const float qs = 1.f / sqrtf((float)dk);
+  for (int i = warp; i < nr * G; i += 8) {          // a warp per (row, group): both unit vectors and their product
+    const int j = i / G, g = i - j * G;
+    const float* q = reinterpret_cast<const float*>(o.A) + (size_t)(m0 + j) * o.lda + (size_t)g * dk;
+    const float* k = q + o.K;
+    float sq = 0.f, sk = 0.f, qk = 0.f;
+    for (int c = lane; c < dk; c += 32) { const float a = q[c], b = k[c]; sq = fmaf(a, a, sq); sk = fmaf(b, b, sk); }
+    const float fq = qs / sqrtf(warp_sum(sq) + 1e-6f), fk = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
+    float* d = w + (size_t)j * cols + (size_t)g * dk;
+    for (int c = lane; c < dk; c += 32) {
+      const float a = q[c] * fq, b = k[c] * fk;
+      d[c] = a; d[(size_t)G * dk + c] = b;
+      qk = fmaf(a, b, qk);
+    }
+    qk = warp_sum(qk);
+    if (lane == 0) cf[(size_t)j * cols + H + g] = qk;
   }
 }
 
@@ -2170,7 +2333,10 @@ __host__ __device__ constexpr int mstate_buf_floats(int rpt, int nv = 2, int cpt
 //
 // CPT = 2 (pieces of long runs, where blocks are plenty): a lane holds two state columns, so a token's vectors are read from shared memory
 // once for both; rounds of eight tokens keep the blocks small.  Warps without a live column only stage.
-template <int RPT, int NV = 2, bool GATED = false, int CPT = 1>
+//
+// CDELTA (NV = 3): the delta rule with a decay per key channel (mode 6), one pass.  With S' = diag(g) S: u = beta (v - S'^T k) and
+// o = S'^T q + u (q . k), so both products run in the pass that decays the state, with one round of shuffles.
+template <int RPT, int NV = 2, bool GATED = false, int CPT = 1, bool CDELTA = false>
 __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, const int phase, const int piece, float* X, float* P) {
   extern __shared__ __align__(16) float msm[];
   constexpr int SL = RPT + 4, ROW = 8 * SL, CH = mstate_ch(CPT), COLS = MS_COLS * CPT;
@@ -2180,7 +2346,7 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   const bool gates = GATED && NV == 3, memory = GATED && NV == 2;
   const bool direct = GATED && o.M <= MS_CH;      // the coefficients are formed here
   const int sv = memory ? dv + 1 : dv;                  // state columns
-  const int wc = NV == 3 ? (gates ? mstate_gate_cols(H, dk) : mstate_decay_cols(H, dk)) : memory ? mstate_max_cols(H) : mstate_ws_cols(H, G, dk, delta);
+  const int wc = CDELTA ? mstate_cdelta_cols(H, G, dk) : NV == 3 ? (gates ? mstate_gate_cols(H, dk) : mstate_decay_cols(H, dk)) : memory ? mstate_max_cols(H) : mstate_ws_cols(H, G, dk, delta);
   const int tid = threadIdx.x, sub = tid & 7, cl = tid >> 3;      // this lane's columns: blockIdx.x * COLS + cl (+ MS_COLS)
   const bool wlive = blockIdx.x * COLS + (cl & ~3) < sv;           // the warp (four neighbouring columns) has one
   int col[CPT];
@@ -2215,10 +2381,11 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
   const int vcol = (qkv_rows ? o.a_rows : 0) + h * dv;
   __syncthreads();
   // keys then queries (B then C) of this head's group, as columns of the rows they are staged from
-  const float* vsrc = (delta || gates) ? wsb : rows;
-  const int vstride = (delta || gates) ? wc : o.lda, off0 = ((delta || gates) ? G * dk : o.K) + g * dk, off1 = ((delta || qkv_rows) ? 0 : o.a_rows) + g * dk;
-  const int offa = (gates ? 2 * H * dk : 0) + h * dk;      // the decays' columns (NV == 3)
-  const int cfo = mstate_ws_coef(G, dk, delta);
+  const bool staged_ws = delta || gates || CDELTA;      // keys and queries come from the first launch's rows
+  const float* vsrc = staged_ws ? wsb : rows;
+  const int vstride = staged_ws ? wc : o.lda, off0 = (staged_ws ? G * dk : o.K) + g * dk, off1 = ((delta || qkv_rows) ? 0 : o.a_rows) + g * dk;
+  const int offa = (CDELTA ? 2 * G * dk : gates ? 2 * H * dk : 0) + h * dk;      // the decays' columns (NV == 3)
+  const int cfo = CDELTA ? (2 * G + H) * dk : mstate_ws_coef(G, dk, delta);
   const bool vec = dk % 4 == 0 && vstride % 4 == 0 && off0 % 4 == 0 && off1 % 4 == 0 && !(reinterpret_cast<uintptr_t>(vsrc) & 15) &&
                    (NV < 3 || (wc % 4 == 0 && offa % 4 == 0 && !(reinterpret_cast<uintptr_t>(wsb) & 15)));
   const float fixed_c1 = fixed ? reinterpret_cast<const float*>(o.scale)[h] : 0.f;
@@ -2275,6 +2442,11 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
         if (tid < nt) { cf[tid * 4] = expf(lf + mine - next); cf[tid * 4 + 1] = expf(li - next); cf[tid * 4 + 2] = expf(-next); }
         if (tid == 0 && blockIdx.x == 0) reinterpret_cast<float*>(const_cast<void*>(o.p1))[h] = m;
       }
+    } else if (CDELTA) {       // write strength and q . k
+      for (int idx = tid; idx < nt * 2; idx += 128) {
+        const int tt = idx >> 1, which = idx & 1;
+        cp_async4(cf + tt * 4 + which, wsb + (size_t)(t0 + tt) * wc + cfo + (which ? H + g : h));
+      }
     } else if (NV < 3 && !fixed)
       for (int idx = tid; idx < nt * 3; idx += 128) {
         const int tt = idx / 3, which = idx - tt * 3;
@@ -2317,6 +2489,35 @@ __global__ void __launch_bounds__(128) fq3s_mstate_scan_kernel(const fq3c_op o, 
         return x;
       };
       float* orow = reinterpret_cast<float*>(o.C) + (size_t)(t0 + tt) * o.ldc + (size_t)h * dv;
+      if (CDELTA) {
+        const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(kq + tt * NV * ROW + 2 * ROW + sub * SL);
+        f32x2 ks[2] = {0ull, 0ull};
+        ulonglong2 kv[RPT / 4];
+#pragma unroll
+        for (int r = 0; r < RPT / 4; ++r) {
+          kv[r] = k4[r];
+          const ulonglong2 qv = q4[r], av = a4[r];
+          S[0][2 * r] = mul2<true>(av.x, S[0][2 * r]);
+          S[0][2 * r + 1] = mul2<true>(av.y, S[0][2 * r + 1]);
+          ks[0] = fma2<true>(kv[r].x, S[0][2 * r], ks[0]);
+          ks[1] = fma2<true>(kv[r].y, S[0][2 * r + 1], ks[1]);
+          os[0][0] = fma2<true>(qv.x, S[0][2 * r], os[0][0]);
+          os[0][1] = fma2<true>(qv.y, S[0][2 * r + 1], os[0][1]);
+        }
+        float kt = (lo2(ks[0]) + hi2(ks[0])) + (lo2(ks[1]) + hi2(ks[1])), qt = (lo2(os[0][0]) + hi2(os[0][0])) + (lo2(os[0][1]) + hi2(os[0][1]));
+        kt += __shfl_xor_sync(0xffffffffu, kt, 1); qt += __shfl_xor_sync(0xffffffffu, qt, 1);
+        kt += __shfl_xor_sync(0xffffffffu, kt, 2); qt += __shfl_xor_sync(0xffffffffu, qt, 2);
+        kt += __shfl_xor_sync(0xffffffffu, kt, 4); qt += __shfl_xor_sync(0xffffffffu, qt, 4);
+        const float u = cf[tt * 4] * (v[0] - kt);
+        const f32x2 uu = pack2(u, u);
+#pragma unroll
+        for (int r = 0; r < RPT / 4; ++r) {
+          S[0][2 * r] = fma2<true>(kv[r].x, uu, S[0][2 * r]);
+          S[0][2 * r + 1] = fma2<true>(kv[r].y, uu, S[0][2 * r + 1]);
+        }
+        if (live[0] && sub == 0) orow[col[0]] = fmaf(u, cf[tt * 4 + 1], qt);
+        continue;
+      }
       if (NV == 3) {      // S <- diag(alpha) S + k v^T, o = f0 S^T q
         const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(kq + tt * NV * ROW + 2 * ROW + sub * SL);
         f32x2 vv[CPT];
@@ -2551,6 +2752,8 @@ __global__ void __launch_bounds__(1024) fq3s_sum_norm_kernel(const fq3c_op o) {
   const float* a = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda;
   const float* w = reinterpret_cast<const float*>(o.p0);
   float* c = reinterpret_cast<float*>(o.C) + (size_t)m * o.ldc;
+  const bool post = (o.flags & FQ3C_POST) != 0;
+  const float* nb = reinterpret_cast<const float*>(o.bias);
   float sm = 0.f;
   for (int i = threadIdx.x; i < o.N; i += blockDim.x) {
     float v = 0.f;
@@ -2562,12 +2765,12 @@ __global__ void __launch_bounds__(1024) fq3s_sum_norm_kernel(const fq3c_op o) {
       for (int q = 0; q < 4; ++q)
         if (j + q < o.i0) v = fmaf(wv[q], av[q], v);
     }
-    c[i] = v;
+    if (!post) c[i] = v;
     if (o.C2) reinterpret_cast<bf16*>(o.C2)[(size_t)m * o.ldc + i] = __float2bfloat16_rn(v);
     snm[i] = v;
     sm += v;
   }
-  if (!o.norm_out) return;
+  if (!o.norm_out && !post) return;
   if (!o.norm_w) {       // no norm: the finished row itself, in the product operands' type
     for (int i = threadIdx.x; i < o.N; i += blockDim.x) {
       if (o.flags & FQ3C_F32) reinterpret_cast<float*>(o.norm_out)[(size_t)m * o.norm_ld + i] = snm[i];
@@ -2582,7 +2785,10 @@ __global__ void __launch_bounds__(1024) fq3s_sum_norm_kernel(const fq3c_op o) {
   const float rs = 1.f / sqrtf(seq_block_sum(ss, red) / (float)o.N + o.norm_eps);
   const float* nw = reinterpret_cast<const float*>(o.norm_w);
   for (int i = threadIdx.x; i < o.N; i += blockDim.x) {
-    const float n = (snm[i] - mean) * rs * nw[i];
+    float n = (snm[i] - mean) * rs * nw[i];
+    if (nb) n += nb[i];
+    if (post) c[i] = n;
+    if (!o.norm_out) continue;
     if (o.flags & FQ3C_F32) reinterpret_cast<float*>(o.norm_out)[(size_t)m * o.norm_ld + i] = n;
     else reinterpret_cast<bf16*>(o.norm_out)[(size_t)m * o.norm_ld + i] = __float2bfloat16_rn(n);
   }
@@ -2596,6 +2802,7 @@ __global__ void __launch_bounds__(256) fq3s_sum_norm_vec_kernel(const fq3c_op o)
   const float* a = reinterpret_cast<const float*>(o.A) + (size_t)m * o.lda;
   const float* w = reinterpret_cast<const float*>(o.p0);
   float* c = reinterpret_cast<float*>(o.C) + (size_t)m * o.ldc;
+  const bool post = (o.flags & FQ3C_POST) != 0;
   float v[SN_VECS][4];
 #pragma unroll
   for (int q = 0; q < SN_VECS; ++q) { v[q][0] = 0.f; v[q][1] = 0.f; v[q][2] = 0.f; v[q][3] = 0.f; }
@@ -2623,10 +2830,10 @@ __global__ void __launch_bounds__(256) fq3s_sum_norm_vec_kernel(const fq3c_op o)
   for (int q = 0; q < SN_VECS; ++q) {
     const int i = (q * nth + tid) * 4;
     if (i >= o.N) continue;
-    st4(c + i, v[q]);
+    if (!post) st4(c + i, v[q]);
     sm += (v[q][0] + v[q][1]) + (v[q][2] + v[q][3]);
   }
-  if (!o.norm_out) return;
+  if (!o.norm_out && !post) return;
   float rs = 1.f, mean = 0.f;
   if (o.norm_w) {
     if (o.flags & FQ3C_CENTER) mean = seq_block_sum(sm, red) / (float)o.N;
@@ -2646,6 +2853,12 @@ __global__ void __launch_bounds__(256) fq3s_sum_norm_vec_kernel(const fq3c_op o)
     if (o.norm_w) {
       const float4 nw = ld4(reinterpret_cast<const float*>(o.norm_w) + i);
       v[q][0] = (v[q][0] - mean) * rs * nw.x; v[q][1] = (v[q][1] - mean) * rs * nw.y; v[q][2] = (v[q][2] - mean) * rs * nw.z; v[q][3] = (v[q][3] - mean) * rs * nw.w;
+      if (o.bias) {
+        const float4 nb = ld4(reinterpret_cast<const float*>(o.bias) + i);
+        v[q][0] += nb.x; v[q][1] += nb.y; v[q][2] += nb.z; v[q][3] += nb.w;
+      }
+      if (post) st4(c + i, v[q]);
+      if (!o.norm_out) continue;
     }
     if (o.flags & FQ3C_F32) st4(reinterpret_cast<float*>(o.norm_out) + (size_t)m * o.norm_ld + i, v[q]);
     else st4(reinterpret_cast<bf16*>(o.norm_out) + (size_t)m * o.norm_ld + i, v[q]);

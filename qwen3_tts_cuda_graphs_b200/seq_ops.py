@@ -17,7 +17,8 @@ with its constants as arguments, so another design composes them differently:
   weighted residual sum of sublayers that ran side by side, chained into the next layer norm or RMS norm), channel_decay_attention
   and retention (linear attentions on the matrix-state scan: a decay per key channel and token, one fixed decay per head),
   forget_gate_attention and matrix_memory (the same scan with gates that also decide what is written, and with exponential gates
-  under a running maximum), gelu_ff.
+  under a running maximum), gelu_ff, gelu_glu_ff (gated unit with the tanh form of gelu), channel_delta_rule (delta rule with a decay per
+  key channel), attention_beside_delta_rule (both on one stacked projection, one convolution and one output product).
 
 Precision: `f32=True` runs every product in true 32-bit.  Otherwise weights and product operands are bf16 with f32
 accumulation; the residual stream, norms, softmax, router, recurrence and everything entering it are f32 in both modes.
@@ -28,11 +29,11 @@ from typing import Dict, List, Optional
 
 import torch
 
-from .codec import (F_A_F32, F_BIAS, F_CENTER, F_SWIGLU, F_F32, F_GATE_POST, F_GATE_PRE, F_GELU, F_NOROUND, F_OUT_F32, F_RAW_WEIGHTS, F_RELU2, F_RESID,
+from .codec import (F_A_F32, F_BIAS, F_CENTER, F_SWIGLU, F_F32, F_GATE_ENTRY, F_GATE_POST, F_GATE_PRE, F_GELU, F_GELU_TANH, F_NOROUND, F_OUT_F32, F_POST, F_RAW_WEIGHTS, F_RELU2, F_RESID,
                     F_ROT_HALF, F_SIGMOID, F_SILU, F_UNIT,
                     K_BDGEMM, K_CACHE_ATTN, K_COMMIT, K_DEPTH_MIX, K_DYT, K_EMBED, K_GEMM, K_GGEMM, K_GLU, K_GNORM, K_HYPER, K_LATENT_ATTN,
                     K_LRU_SCAN, K_MOE_COMBINE, K_MOE_SORT, K_MSTATE_SCAN, K_POLYNORM, K_ROT_APPEND, K_ROUTER, K_SUM_NORM, K_TCONV, K_XIELU, Op, _Plan)
-from .config import (ChannelDecayAttentionConfig, DeltaRuleConfig, ForgetGateAttentionConfig, LatentAttentionConfig, MatrixMemoryConfig,
+from .config import (ChannelDecayAttentionConfig, ChannelDeltaRuleConfig, DeltaRuleConfig, ForgetGateAttentionConfig, LatentAttentionConfig, MatrixMemoryConfig,
                      MoEFFConfig, RetentionConfig, RglruConfig, SoftmaxAttentionConfig, StateSpaceConfig)
 from .seq_state import SlotState
 
@@ -111,12 +112,15 @@ class StepBuilder:
         return out
 
     def time_conv(self, x: torch.Tensor, w: torch.Tensor, state: str, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                  add_input: bool = False, col: int = 0, channels: Optional[int] = None, silu: bool = False):
-        """out = act((x if add_input) + bias + causal conv over time of x's columns [col, col + channels)); w f32 [channels, taps]."""
+                  add_input: bool = False, col: int = 0, channels: Optional[int] = None, silu: bool = False, silu_from: int = 0):
+        """out = act((x if add_input) + bias + causal conv over time of x's columns [col, col + channels)); w f32 [channels, taps].
+        silu_from: only channels from this one on pass silu."""
         taps = w.shape[1]
         n = channels or w.shape[0]
         flags = self._oflag(out) | (F_BIAS if bias is not None else 0) | (F_RESID if add_input else 0) | (F_SILU if silu else 0)
         kw = dict(M=self.M, N=n, taps=taps, A=_ptr(x, col), lda=x.shape[1], B=w, C=out, ldc=out.shape[1], flags=flags)
+        if silu:
+            kw["i0"] = silu_from
         if bias is not None:
             kw["bias"] = bias
         if taps > 1:
@@ -129,14 +133,19 @@ class StepBuilder:
                    col: int = 0, residual: Optional[torch.Tensor] = None, out_bf16: Optional[torch.Tensor] = None,
                    append_at_position: bool = False, gate: Optional[torch.Tensor] = None, gate_col: int = 0, gate_first: bool = False,
                    weight_period: int = 0, center: bool = False, rows: Optional[int] = None, gate_sigmoid: bool = False,
-                   divisor: Optional[torch.Tensor] = None):
+                   divisor: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, out_col: int = 0):
         """out = (residual +) rms_unit_per_group(x) * w.  `gate` (f32 rows, columns from gate_col): the row times silu(gate) before the
         statistics (gate_first) or after the weights.  weight_period > 0: w has that many entries and repeats (a per-head norm).
         w None: no weights (n required).  center: the statistics are mean and variance (a layer norm without bias).  gate_sigmoid: the
-        gate is a sigmoid instead of a silu.  divisor f32 [rows, groups]: a group is divided by its entry first."""
+        gate is a sigmoid instead of a silu.  divisor f32 [rows, groups]: a group is divided by its entry first.  bias f32 [N] is added to
+        the result (not together with a residual).  The result goes to out's columns from out_col on."""
         n = n or w.shape[0]
-        kw = dict(M=rows or self.M, N=n, i0=groups, f0=eps, A=_ptr(x, col), lda=x.shape[1], C=out, ldc=out.shape[1], i2=weight_period,
+        kw = dict(M=rows or self.M, N=n, i0=groups, f0=eps, A=_ptr(x, col), lda=x.shape[1], C=_ptr(out, out_col), ldc=out.shape[1], i2=weight_period,
                   flags=self._oflag(out) | (F_RESID if residual is not None else 0) | (F_CENTER if center else 0))
+        if bias is not None:      # one row added to every row
+            assert residual is None
+            kw["res"], kw["ldr"] = bias, 0
+            kw["flags"] |= F_RESID
         if w is not None:
             kw["scale"] = w
         if gate is not None:
@@ -151,15 +160,15 @@ class StepBuilder:
             kw["C2"] = out_bf16
         if append_at_position:
             kw["p0"] = self.slot.pos
-        self.plan.keep += [x]
+        self.plan.keep += [x, out]
         self._op(K_GNORM, **kw)
         return out
 
     def linear(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None, gelu: bool = False,
-               rows: Optional[int] = None, force_f32: bool = False, glu: bool = False, relu2: bool = False):
+               rows: Optional[int] = None, force_f32: bool = False, glu: bool = False, relu2: bool = False, glu_gelu: bool = False):
         """out = act(x W^T + bias), act = gelu, max(., 0)^2 (relu2) or none.  x and W share a type (bf16, or f32 for true 32-bit:
         `force_f32` for a router).  glu: W's rows
-        alternate (gate_n, up_n) and out [M, N / 2] = silu(gate) * up, formed in the product's epilogue."""
+        alternate (gate_n, up_n) and out [M, N / 2] = silu(gate) * up (glu_gelu: gelu_tanh(gate) * up), formed in the product's epilogue."""
         M = rows or self.M
         N, K = w.shape
         f32 = w.dtype == torch.float32
@@ -168,7 +177,7 @@ class StepBuilder:
         if out.dtype == torch.float32 or M <= 4 or glu or gelu:
             flags |= F_NOROUND      # f32 results and the activation's argument stay unrounded; with a few rows the flag also picks the weight-streaming product
         if glu:
-            flags |= F_SWIGLU
+            flags |= F_SWIGLU | (F_GELU_TANH if glu_gelu else 0)
         kw = dict(M=M, N=N, K=K, taps=1, cin=K, a_rows=x.shape[0], lda=x.shape[1], ldc=out.shape[1], col_mod=N, A=x, B=w, C=out, flags=flags)
         if bias is not None:
             kw["bias"] = bias
@@ -287,11 +296,13 @@ class StepBuilder:
         return out
 
     def sum_norm(self, parts: torch.Tensor, count: int, weights: torch.Tensor, norm_w: Optional[torch.Tensor] = None,
-                 norm_out: Optional[torch.Tensor] = None, eps: float = 0.0, center: bool = False, out: Optional[torch.Tensor] = None):
+                 norm_out: Optional[torch.Tensor] = None, eps: float = 0.0, center: bool = False, out: Optional[torch.Tensor] = None, norm_b: Optional[torch.Tensor] = None,
+                 post: bool = False):
         """parts f32 [slices, M, N]: out (default parts[0], the residual stream, in place) = sum_(j < count) weights[j] * parts[j],
         weights f32 [count] on the device.  With norm_out: also norm_out = norm(out) * norm_w — RMS, or with `center` mean / variance —
         in the same launch (the norm that reads the finished stream next); without norm_w norm_out gets the finished row itself (the
-        operand of a product that reads the stream)."""
+        operand of a product that reads the stream).  norm_b f32 [N]: the norm's bias.  post: out is the normed row itself (a norm behind
+        the sum) and norm_out, when given, a copy of it."""
         out = parts[0] if out is None else out
         kw = dict(M=self.M, N=parts.shape[2], i0=count, K=parts.shape[1] * parts.shape[2], A=parts, lda=parts.shape[2], p0=weights, C=out,
                   ldc=out.shape[1], flags=F_OUT_F32 | (F_CENTER if center else 0))
@@ -301,6 +312,11 @@ class StepBuilder:
                 kw["norm_w"] = norm_w
             if norm_out.dtype == torch.float32:
                 kw["flags"] |= F_F32
+        if post:
+            kw.update(norm_w=norm_w, norm_eps=float(eps))
+            kw["flags"] |= F_POST
+        if norm_b is not None:
+            kw["bias"] = norm_b
         self._op(K_SUM_NORM, **kw)
         return out
 
@@ -311,21 +327,37 @@ class StepBuilder:
         (unless the layer borrows a cache) keys and values, then the gate rows; bqkv f32 or None; freq f32 [rot_dims / 2] or None (freq_lo: what its
         entries lost to rounding, or None); sink f32 [H] or None; r12 f32 [2H] or None; o [width, H * vdim]; o_b f32 or None; q_norm / k_norm f32 [dim] with qk_norm
         (eps: their epsilon; qk_unit: no weights).  kcache / vcache name the slot's append states to write (own projections) and read;
-        with pooled blocks (c.pool) kcache + ".pool" and vcache + ".pool" hold one row per complete block."""
+        with pooled blocks (c.pool) kcache + ".pool" and vcache + ".pool" hold one row per complete block.  c.conv: conv f32 [query, key and
+        value channels, taps], its carried inputs under kcache + ".conv".  c.keys_as_values: no value rows in wqkv.  c.entry_gate: H * vdim gate rows."""
         M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
         own = c.kv_from is None
         kcol = H * d
-        vcol = kcol + (G * d if own else 0)
-        gcol = vcol + (G * dv if own else 0)
+        vcol = kcol + (G * d if own and not c.keys_as_values else 0)
+        gcol = kcol + (G * d + (0 if c.keys_as_values else G * dv) if own else 0)
         proj = self.linear(h, w["wqkv"], self.buf("sa.proj", M, w["wqkv"].shape[0]), bias=w.get("bqkv"))
+        rows = self.time_conv(proj, w["conv"], kcache + ".conv", self.buf("sa.cv", M, gcol), channels=gcol) if c.conv > 0 else proj
+        oa = self.buf("sa.o", M, H * dv, self.adt)
+        self._attend(c, w, rows, 0, kcol, vcol, (proj, gcol), kcache, vcache, eps, oa)
+        return self.linear(oa, w["o"], out, bias=w.get("o_b"))
+
+    def _attend(self, c: SoftmaxAttentionConfig, w: dict, rows: torch.Tensor, qcol: int, kcol: int, vcol: int, gate, kcache: str, vcache: str,
+                eps: float, oa: torch.Tensor, mult: float = 1.0):
+        """The part of softmax_attention between the projections and the output product: rows f32 hold queries / keys / values from columns
+        qcol / kcol / vcol on, gate = (rows, column) of the gate inputs; the heads' outputs (times mult) go to oa's first H * vdim columns."""
+        M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
+        own = c.kv_from is None
         kc, vc = self.slot.cur[kcache], self.slot.cur[vcache]
         cf32 = F_F32 if kc.dtype == torch.float32 else 0
         pool = c.pool if c.window > 0 else 0
-        if own or c.rot_dims > 0 or c.qk_norm or c.qk_unit:
-            kw = dict(M=M, i0=H, i1=G if own else 0, i2=d, cin=dv, taps=c.rot_dims, K=kcol, a_rows=vcol, A=proj, lda=proj.shape[1],
-                      p0=self.slot.pos, flags=cf32)
+        self.plan.keep += [rows, oa]
+        if own or c.rot_dims > 0 or c.qk_norm or c.qk_unit or c.q_temp is not None:
+            kw = dict(M=M, i0=H, i1=G if own else 0, i2=d, cin=dv, taps=c.rot_dims, K=kcol - qcol, a_rows=vcol - qcol, A=_ptr(rows, qcol),
+                      lda=rows.shape[1], p0=self.slot.pos, flags=cf32)
+            if c.q_temp is not None:
+                kw["f2"], kw["f3"] = c.q_temp
             if c.rot_dims > 0:
                 kw["B"] = w["freq"]
+                kw["f1"] = float(w.get("amp", 1.0))
                 if w.get("freq_lo") is not None:
                     kw["p1"] = w["freq_lo"]
             if c.qk_norm:   # per-head norms in the same launch, before the rotation
@@ -349,16 +381,17 @@ class StepBuilder:
         tiles = max(1, -(-span // 32))
         blocks = -(-M // QB) * G
         splits = min(64, tiles) if M <= 8 else (1 if blocks >= 74 else max(1, min(16, tiles, -(-296 // blocks))))
-        oa = self.buf("sa.o", M, H * dv, self.adt)
         kw = dict(M=M, N=H * dv, i0=H, i1=G, i2=d, cin=dv, f0=c.scale, f1=c.softcap, K=c.window, a_rows=c.keep_first if c.window > 0 else 0,
-                  A=proj, lda=proj.shape[1], B=kc, ldr=kc.shape[1], p1=vc, taps=vc.shape[1], p0=self.slot.pos, m_begin=splits,
+                  f2=float(mult), A=_ptr(rows, qcol), lda=rows.shape[1], B=kc, ldr=kc.shape[1], p1=vc, taps=vc.shape[1], p0=self.slot.pos, m_begin=splits,
                   C=oa, ldc=oa.shape[1], flags=cf32 | self._oflag(oa))
         if w.get("sink") is not None:
             kw["scale"] = w["sink"]
         if w.get("r12") is not None:
             kw["bias"] = w["r12"]
-        if c.gate:
-            kw["res"], kw["col_mod"] = _ptr(proj, gcol), proj.shape[1]
+        if c.gate or c.entry_gate:
+            kw["res"], kw["col_mod"] = _ptr(*gate), gate[0].shape[1]
+            kw["flags"] |= F_GATE_ENTRY if c.entry_gate else 0
+            self.plan.keep.append(gate[0])
         if pool > 0:
             kw["C2"], kw["norm_out"] = self.slot.cur[kcache + ".pool"], self.slot.cur[vcache + ".pool"]
         if splits > 1:
@@ -366,7 +399,7 @@ class StepBuilder:
             kw["ws"], kw["ws_bytes"] = ws, ws.numel() * 4
         op = self._op(K_CACHE_ATTN, **kw)
         op.tap_off[0], op.tap_off[1] = max(c.chunk, 0), pool
-        return self.linear(oa, w["o"], out, bias=w.get("o_b"))
+        return oa
 
     # ---- recurrences with a matrix state per head -----------------------------------------------------
     def _scan_ws(self, coef_cols: int, H: int, dk: int, dv: int, pieces: bool = True) -> torch.Tensor:
@@ -431,6 +464,50 @@ class StepBuilder:
         yn = self.group_norm(y, w["norm"], H, eps, self.buf("cd.yn", M, H * dv, self.adt), n=H * dv, gate=raw, gate_col=gcol, weight_period=dv)
         return self.linear(yn, w["o"], out)
 
+    def channel_delta_rule(self, h: torch.Tensor, c: ChannelDeltaRuleConfig, w: dict, state: str, eps: float, out: torch.Tensor):
+        """h [M, width] -> out f32 [M, width].  w: win [2 G dim + H vdim + H + decay rank + gate rank (+ padding), width] (q | k | v |
+        write-strength input | decay latent | gate latent), conv f32 [2 G dim + H vdim, taps], a2 [H dim, decay rank], dt_bias f32 [H dim],
+        A_log f32 [H], g2 [H vdim, gate rank], norm f32 [vdim], o [width, H vdim].  Per head S <- diag(g) S, g = exp(-exp(A_log) softplus(z));
+        u = beta (v - S^T k); S <- S + k u^T; o = S^T q, on unit queries (times dim^(-1/2)) and keys.  States: state + ".conv", state + ".s"."""
+        M, n = self.M, 2 * c.kv_heads * c.dim + c.heads * c.vdim
+        raw = self.linear(h, w["win"], self.buf("kd.raw", M, w["win"].shape[0]))
+        cv = self.time_conv(raw, w["conv"], state + ".conv", self.buf("kd.cv", M, n), channels=n, silu=True)
+        yn = self.buf("kd.yn", M, c.heads * c.vdim, self.adt)
+        self._channel_delta(c, w, cv, 0, raw, n, state + ".s", eps, yn, 0)
+        return self.linear(yn, w["o"], out)
+
+    def _channel_delta(self, c: ChannelDeltaRuleConfig, w: dict, cv: torch.Tensor, ccol: int, raw: torch.Tensor, rcol: int, state: str, eps: float,
+                       yn: torch.Tensor, ycol: int):
+        """channel_delta_rule between the convolution and the output product: q | k | v in cv's columns from ccol on, write-strength inputs |
+        decay latent | gate latent in raw's from rcol on; the gated read-out goes to yn's columns from ycol on."""
+        M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
+        ra, rg = w["a2"].shape[1], w["g2"].shape[1]
+        y, gate = self.buf("kd.y", M, H * dv), self.buf("kd.gate", M, H * dv)
+        ws = self._scan_ws(-(-((2 * G + H) * d + H + G) // 4) * 4, H, d, dv, pieces=False)
+        self.plan.keep += [cv, raw]
+        op = self._op(K_MSTATE_SCAN, M=M, N=H * dv, taps=6, i0=H, i1=G, i2=d, cin=dv, K=G * d, a_rows=2 * G * d, A=_ptr(cv, ccol), lda=cv.shape[1],
+                      res=raw, ldr=raw.shape[1], m_begin=rcol, col_mod=rcol + H, B=w["a2"], bias=w["dt_bias"], scale=w["A_log"], p1=w["g2"],
+                      norm_out=gate, norm_ld=H * dv, p0=self.slot.cur[state], C2=self.slot.next[state], C=y, ldc=y.shape[1], ws=ws,
+                      ws_bytes=ws.numel() * 4, flags=F_OUT_F32 | (F_F32 if w["a2"].dtype == torch.float32 else 0))
+        op.tap_off[0], op.tap_off[1], op.tap_off[2] = ra, rcol + H + ra, rg
+        return self.group_norm(y, w["norm"], H, eps, yn, n=H * dv, gate=gate, gate_sigmoid=True, weight_period=dv, out_col=ycol)
+
+    def attention_beside_delta_rule(self, h: torch.Tensor, left: SoftmaxAttentionConfig, right: ChannelDeltaRuleConfig, w: dict, kcache: str, vcache: str,
+                                    state: str, eps: float, out: torch.Tensor, left_scale: float = 1.0):
+        """left_scale * attention + delta rule, both reading h [M, width] -> out f32 [M, width], as one product each way: w["win"] stacks the
+        left's q | k | v, the right's q | k | v, the left's gate rows and the right's write-strength inputs | decay latent | gate latent;
+        w["conv"] f32 over the first six parts (state + ".conv"; the right's channels pass silu); w["o"] = [left's | right's] output projection
+        on the concatenated heads.  A scale of the right side belongs in w["right"]["norm"].  w["left"], w["right"]: what the parts between take."""
+        M, H, G, d, dv = self.M, left.heads, left.kv_heads, left.dim, left.vdim
+        nl = (H + G) * d + G * dv
+        n = nl + 2 * right.kv_heads * right.dim + right.heads * right.vdim
+        raw = self.linear(h, w["win"], self.buf("pd.raw", M, w["win"].shape[0]))
+        cv = self.time_conv(raw, w["conv"], state + ".conv", self.buf("pd.cv", M, n), channels=n, silu=True, silu_from=nl)
+        heads = self.buf("pd.heads", M, H * dv + right.heads * right.vdim, self.adt)
+        self._attend(left, w["left"], cv, 0, H * d, (H + G) * d, (raw, n), kcache, vcache, eps, heads, mult=left_scale)
+        self._channel_delta(right, w["right"], cv, nl, raw, n + H * dv, state + ".s", eps, heads, H * dv)
+        return self.linear(heads, w["o"], out)
+
     def retention(self, h: torch.Tensor, c: RetentionConfig, w: dict, state: str, eps: float, out: torch.Tensor):
         """h [M, width] -> out f32 [M, width].  w: win [2 H dim + 2 H vdim, width] (q | k | v | output gate), decay f32 [H],
         freq f32 [rot_dims / 2] or None, o [width, H vdim].  q and k turn in place (pairs i, i + rot_dims / 2); per head
@@ -486,6 +563,12 @@ class StepBuilder:
     def gelu_ff(self, x: torch.Tensor, w: dict, out: torch.Tensor):
         """out f32 = W_down gelu(W_up x) (erf form); w: up [ff, width], down [width, ff].  The activation rides in the first product."""
         za = self.linear(x, w["up"], self.buf("ff.za", self.M, w["up"].shape[0], self.adt), gelu=True)
+        return self.linear(za, w["down"], out)
+
+    def gelu_glu_ff(self, x: torch.Tensor, w: dict, out: torch.Tensor):
+        """out f32 = W_down (gelu_tanh(W_gate x) * (W_up x)); w: gate_up [2 ff, width] with alternating rows (gate_0, up_0, gate_1, ...),
+        down [width, ff].  The gated unit is formed in the first product's epilogue."""
+        za = self.linear(x, w["gate_up"], self.buf("ff.glu", self.M, w["gate_up"].shape[0] // 2, self.adt), glu=True, glu_gelu=True)
         return self.linear(za, w["down"], out)
 
     def xielu_ff(self, x: torch.Tensor, w: dict, out: torch.Tensor):
