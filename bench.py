@@ -271,7 +271,7 @@ def main():
                     help="instead of the default workload: prefill / decode throughput and per-kernel rooflines of the sequence "
                          "models (Sidalorn, Redodra, Ratizen, Zudusun, Sirodra) at real-size layers beside the talker (qwen3_tts_cuda_graphs_b200/seq_bench.py); one GPU")
     ap.add_argument("--seq-tokens", type=int, default=2048, dest="seq_tokens", help="--seq-model: prompt length / decode context")
-    ap.add_argument("--seq-sizes", default="w1024,w2048", dest="seq_sizes", help="--seq-model: comma list of sizes (w1024, w2048: Sidalorn; r1024, r2048: Redodra; z1024, z2048: Ratizen; u1024, u2048: Zudusun; s1024, s2048: Sirodra)")
+    ap.add_argument("--seq-sizes", default="w1024,w2048", dest="seq_sizes", help="--seq-model: comma list of sizes (w1024, w2048: Sidalorn; r1024, r2048: Redodra; z1024, z2048: Ratizen; u1024, u2048: Zudusun; s1024, s2048: Sirodra; m1024, m2048: Matidra)")
     args = ap.parse_args()
     if args.seq_model:
         from qwen3_tts_cuda_graphs_b200 import seq_bench

@@ -1,7 +1,7 @@
 """Throughput of a sequence model at layer sizes that resemble a real model's, beside the closest model of the framework.
 
 `bench.py --seq-model` (the default workload of bench.py is untouched).  Random weights, synthetic tokens.  Sizes w* are Sidalorn
-models, r* Redodra models, z* Ratizen models, u* Zudusun models, s* Sirodra models (`--seq-sizes s1024,u1024,z1024,r1024,w1024` puts the
+models, r* Redodra models, z* Ratizen models, u* Zudusun models, s* Sirodra models, m* Matidra models (`--seq-sizes m1024,s1024,u1024,z1024,r1024,w1024` puts the
 designs side by side at equal width).  For
 each size:
   * prefill: one step of T prompt tokens through `SequenceEngine.step` (tokens / s), and the same in portions;
@@ -23,8 +23,8 @@ from collections import defaultdict
 import torch
 
 from . import codec as K
-from .config import (ChannelDecayAttentionConfig, DeltaRuleConfig, DenseFFConfig, ForgetGateAttentionConfig, LatentAttentionConfig, LoopConfig,
-                     MatrixMemoryConfig, MoEFFConfig, ParallelMixerConfig, RatizenConfig, RedodraConfig, RetentionConfig, RglruConfig,
+from .config import (ChannelDecayAttentionConfig, ChannelDeltaRuleConfig, DeltaRuleConfig, DenseFFConfig, ForgetGateAttentionConfig, LatentAttentionConfig, LoopConfig,
+                     MatidraConfig, MatrixMemoryConfig, MoEFFConfig, ParallelMixerConfig, RatizenConfig, RedodraConfig, RetentionConfig, RglruConfig,
                      ScaledPairMixerConfig, SeqLayerConfig, SidalornConfig, SirodraConfig, SoftmaxAttentionConfig, StateSpaceConfig,
                      ZudusunConfig)
 
@@ -96,7 +96,17 @@ def sizes():
         mix = {"hgrn2": ForgetGateAttentionConfig(lin_heads, 128, 128), "mlstm": MatrixMemoryConfig(lin_heads, 128, 128, 12.0), "attention": att}
         return SirodraConfig(vocab, width, 1e-5, tuple(SeqLayerConfig(t, mix[t], DenseFFConfig(ff)) for t in order), LoopConfig(0, len(order), times))
 
-    return {"s1024": sirodra(1024, 16, 4, 8, 3072, ("mlstm", "hgrn2", "attention"), 2),
+    def matidra(width, heads, kv, lin_heads, ff, order, rank=64, vocab=3072):
+        att = SoftmaxAttentionConfig(heads, kv, 128, 128, 128 ** -0.5, rot_dims=64, rot_base=3e5, rot_scaling=(4.0, 8192.0, 24.0, 2.0), qk_norm=True,
+                                     keys_as_values=True)
+        left = SoftmaxAttentionConfig(heads // 2, max(1, kv // 2), 128, 128, 128 ** -0.5, qk_norm=True, conv=4, q_temp=(0.2, 1024.0), entry_gate=True)
+        pair = ScaledPairMixerConfig(left, ChannelDeltaRuleConfig(lin_heads, lin_heads, 128, 128, 4, rank, rank), 0.8, 0.6)
+        mix = {"parallel": pair, "attention": att}
+        return MatidraConfig(vocab, width, 1e-5, 1.5, tuple(SeqLayerConfig(t, mix[t], DenseFFConfig(ff)) for t in order))
+
+    return {"m1024": matidra(1024, 16, 4, 8, 3072, ("parallel", "attention", "parallel") * 2),
+            "m2048": matidra(2048, 32, 8, 16, 6144, ("parallel", "attention", "parallel")),
+            "s1024": sirodra(1024, 16, 4, 8, 3072, ("mlstm", "hgrn2", "attention"), 2),
             "s2048": sirodra(2048, 32, 8, 16, 6144, ("mlstm", "hgrn2", "attention"), 1),
             "u1024": zudusun(1024, 16, 4, 8, 16, 2, 768, 1536, ("parallel", "attention", "retention") * 2),
             "u2048": zudusun(2048, 32, 8, 16, 32, 4, 1024, 2048, ("parallel", "attention", "retention")),
@@ -124,6 +134,10 @@ def random_model(cfg, device, seed=0):
         from .sirodra import SirodraModel, init_synthetic
 
         return SirodraModel(cfg, init_synthetic(cfg, seed).get, device, f32=False)
+    if isinstance(cfg, MatidraConfig):
+        from .matidra import MatidraModel, init_synthetic
+
+        return MatidraModel(cfg, init_synthetic(cfg, seed).get, device, f32=False)
     from .sidalorn import SidalornModel, tensor_specs
 
     g = torch.Generator(device=device).manual_seed(seed)
@@ -170,6 +184,9 @@ def op_cost(o, ctx_keys: float):
             keys = min(keys, (o.tap_off[0] + 1) / 2.0)                      # chunked mask: half a chunk on average
         return 2.0 * M * o.i0 * (o.i2 + o.cin) * keys, min(ctx_keys + M / 2, keys + M) * o.i1 * (o.i2 + o.cin) * ws + M * o.i0 * (o.i2 * 4 + o.cin * outs)
     if k == K.K_MSTATE_SCAN:
+        if o.taps == 6:       # two up-projections; beside q, k, v and the output: decays, unit vectors (once per key head) and gate rows
+            low = 2.0 * M * (o.i0 * o.i2 * o.tap_off[0] + o.i0 * o.cin * o.tap_off[2])
+            return low + 8.0 * M * o.i0 * o.i2 * o.cin, M * (2 * o.i1 * o.i2 + 2 * o.i0 * o.cin + o.i0 * o.cin) * 4 + 2 * o.i0 * o.i2 * o.cin * 4
         per = 7.0 if o.taps == 0 else 5.0
         vecs = 4 if o.taps == 2 else 2        # channel decays: written by the first launch and read again by the walk, beside q and k
         return per * M * o.i0 * o.i2 * o.cin, M * (vecs * o.i1 * o.i2 + 2 * o.i0 * o.cin) * 4 + 2 * o.i0 * o.i2 * o.cin * 4
@@ -292,7 +309,7 @@ def bench_sequence_model(name, cfg, T, device):
     for i, (L, w) in enumerate(zip(cfg.layers, model.layers)):
         if isinstance(cfg, SirodraConfig):
             break
-        if isinstance(cfg, RedodraConfig):
+        if isinstance(cfg, (RedodraConfig, MatidraConfig)):
             wb += operand_bytes(w)
             continue
         if isinstance(cfg, (RatizenConfig, ZudusunConfig)):
