@@ -208,7 +208,10 @@ enum fq3c_kind {
    *       q, k <- unit vectors as for taps = 0;  g = exp(-exp(scale[h]) softplus(z)) per head and key channel;  beta = sigmoid(b);
    *       S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  C = S^T q.
    *     tap_off[2] = R > 0: a second up-projection in the same launch: norm_out (f32 [M, i0 * cin], pitch norm_ld) = p1 lat2 with p1
-   *     [i0 * cin, R] (B's type) and lat2 at column tap_off[1] of the rows res.  ws = f32 [M, round_up(2 * i1 * i2 + i0 * i2 + i0 + i1, 4)].  */
+   *     [i0 * cin, R] (B's type) and lat2 at column tap_off[1] of the rows res.  ws = f32 [M, round_up(2 * i1 * i2 + i0 * i2 + i0 + i1, 4)].
+   *     Both delta rules (taps 0 and 6), M >= 32 and i2 <= 256: when ws also has room for them (M * round_up(i0 * i2, 4) floats of decay
+   *     logarithms for taps = 6, then ceil(M / 16) * i0 records of 48 (D + 4) + D + 640 floats, D = i2 rounded up to 16), the rows are walked
+   *     in blocks of 16 tokens: same recurrence, other order of the sums.  */
 };
 
 enum fq3c_flags {

@@ -1431,6 +1431,9 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         const int cols = o.taps == 4 ? mstate_gate_cols(o.i0, o.i2) : mstate_max_cols(o.i0);
         if (o.M > MS_CH && (!o.ws || o.ws_bytes < (int64_t)o.M * cols * 4)) return fail("mstate_scan: workspace too small");
       }
+      // delta rules over many rows: blocks of tokens, when the workspace holds their records
+      const bool blocks = (o.taps == 0 || o.taps == 6) && o.M >= CD_MIN_ROWS && o.i2 <= CD_MAX_DK &&
+                          o.ws_bytes / 4 >= cd_ws_floats(o.M, o.i0, o.i2, o.taps == 6) && !(reinterpret_cast<uintptr_t>(o.ws) & 15);
       if (o.taps == 4 && o.M > MS_CH) {
         fq3s_mstate_gate_kernel<<<dim3(o.M, (o.i0 * o.i2 + 255) / 256), 256, 0, s>>>(o);
         count_launches(1);
@@ -1438,12 +1441,12 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         fq3s_mstate_max_kernel<<<o.i0, MM_THREADS, 0, s>>>(o);
         count_launches(1);
       } else if (o.taps == 6) {
-        const dim3 grid((o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS, (o.i0 * o.i2 + 255) / 256 + (o.tap_off[2] > 0 ? (o.i0 * o.cin + 255) / 256 : 0) + 1);
+        const dim3 grid((o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS, (o.i0 * o.i2 + 255) / 256 + (o.tap_off[2] > 0 ? (o.i0 * o.cin + 255) / 256 : 0) + (blocks ? 0 : 1));
         const size_t smem = sizeof(float) * MS_PREP_ROWS * (size_t)std::max(o.tap_off[0], o.tap_off[2]);
-        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, 256, smem, s>>>(o);
-        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, 256, smem, s>>>(o);
+        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, 256, smem, s>>>(o, false);
+        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, 256, smem, s>>>(o, blocks);
         count_launches(1);
-      } else if (o.taps < 3) {
+      } else if (o.taps < 3 && !blocks) {
         fq3s_mstate_prep_kernel<<<o.taps == 2 ? (o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS : o.M, 128, 0, s>>>(o);
         count_launches(1);
       }
@@ -1465,6 +1468,29 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<32, 3, false, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         cudaFuncSetAttribute(fq3s_mstate_scan_kernel<64, 3, false, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 216 * 1024);
         sattr[dev] = true;
+      }
+      if (blocks) {
+        static bool battr[64] = {};
+        if (dev >= 0 && dev < 64 && !battr[dev]) {
+          cudaFuncSetAttribute(fq3s_cdelta_record_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 4 * CD_C * cd_pitch(CD_MAX_DK) * 4);
+          cudaFuncSetAttribute(fq3s_cdelta_walk_kernel<8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, cd_walk_floats<8>(CD_MAX_DK) * 4);
+          cudaFuncSetAttribute(fq3s_cdelta_walk_kernel<8, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, cd_walk_floats<8>(CD_MAX_DK) * 4);
+          cudaFuncSetAttribute(fq3s_cdelta_walk_kernel<16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, cd_walk_floats<16>(CD_MAX_DK) * 4);
+          cudaFuncSetAttribute(fq3s_cdelta_walk_kernel<16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, cd_walk_floats<16>(CD_MAX_DK) * 4);
+          cudaFuncSetAttribute(fq3s_cdelta_walk_kernel<16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, cd_walk_floats<16>(CD_MAX_DK) * 4);
+          battr[dev] = true;
+        }
+        fq3s_cdelta_record_kernel<<<dim3((o.M + CD_C - 1) / CD_C, o.i0), CD_REC_THREADS, 4 * CD_C * cd_pitch(o.i2) * 4, s>>>(o);
+        count_launches(1);
+        // narrow state tiles while they do not outnumber the SMs, wide ones otherwise and for few state rows
+        const bool narrow = o.i2 > 64 && o.i0 * ((o.cin + 7) / 8) <= 148;
+        const dim3 grid((o.cin + (narrow ? 7 : 15)) / (narrow ? 8 : 16), o.i0);
+        if (narrow && o.i2 <= 128) fq3s_cdelta_walk_kernel<8, 1><<<grid, 128, cd_walk_floats<8>(o.i2) * 4, s>>>(o);
+        else if (narrow) fq3s_cdelta_walk_kernel<8, 2><<<grid, 128, cd_walk_floats<8>(o.i2) * 4, s>>>(o);
+        else if (o.i2 <= 64) fq3s_cdelta_walk_kernel<16, 1><<<grid, 128, cd_walk_floats<16>(o.i2) * 4, s>>>(o);
+        else if (o.i2 <= 128) fq3s_cdelta_walk_kernel<16, 2><<<grid, 128, cd_walk_floats<16>(o.i2) * 4, s>>>(o);
+        else fq3s_cdelta_walk_kernel<16, 4><<<grid, 128, cd_walk_floats<16>(o.i2) * 4, s>>>(o);
+        return 0;
       }
       // Long runs of a recurrence whose decays do not depend on the state: pieces walked twice (see the kernel), when the caller's
       // workspace has room behind the per-row coefficients for the pieces' states and decay products.

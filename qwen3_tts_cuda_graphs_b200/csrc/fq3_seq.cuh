@@ -2148,12 +2148,13 @@ __device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, co
     for (int r = 0; r < R; ++r) add(__bfloat162float(u[r]), r);
   }
 }
+// With `logs` the rows hold the base-2 logarithms of the decays alone (pitch round_up(H * dk, 4)), for the walk in blocks of tokens.
 template <int ROWS>
-__global__ void __launch_bounds__(256) fq3s_mstate_cdelta_prep_kernel(const fq3c_op o) {
+__global__ void __launch_bounds__(256) fq3s_mstate_cdelta_prep_kernel(const fq3c_op o, const bool logs) {
   extern __shared__ __align__(16) float cd_lat[];       // [inner size][8]
   const int H = o.i0, G = o.i1, dk = o.i2, m0 = blockIdx.x * MS_PREP_ROWS, nr = min(ROWS, o.M - m0), tid = threadIdx.x;
   const int nd = (H * dk + 255) / 256, ng = o.tap_off[2] > 0 ? (H * o.cin + 255) / 256 : 0, y = blockIdx.y;
-  const int cols = mstate_cdelta_cols(H, G, dk);
+  const int cols = logs ? (H * dk + 3) & ~3 : mstate_cdelta_cols(H, G, dk);
   const float* raw = reinterpret_cast<const float*>(o.res) + (size_t)m0 * o.ldr;
   float* w = reinterpret_cast<float*>(o.ws) + (size_t)m0 * cols;
   if (y < nd + ng) {
@@ -2171,7 +2172,11 @@ __global__ void __launch_bounds__(256) fq3s_mstate_cdelta_prep_kernel(const fq3c
       const float db = reinterpret_cast<const float*>(o.bias)[c], rate = expf(reinterpret_cast<const float*>(o.scale)[c / dk]);
 #pragma unroll
       for (int j = 0; j < ROWS; ++j)
-        if (j < nr) w[(size_t)j * cols + 2 * G * dk + c] = expf(-rate * softplus_f(z[j] + db));
+        if (j < nr) {
+          const float l = -rate * softplus_f(z[j] + db);
+          if (logs) w[(size_t)j * cols + c] = 1.4426950408889634f * l;
+          else w[(size_t)j * cols + 2 * G * dk + c] = expf(l);
+        }
     } else {
       if (c >= H * o.cin) return;
       cdelta_up<ROWS>(o, cd_lat, o.p1, c, R, z);
@@ -2664,6 +2669,299 @@ __global__ void __launch_bounds__(256) fq3s_mstate_carry_kernel(const fq3c_op o,
     R = fmaf(P[(size_t)z * o.i0 * o.i2 + hi], R, X[(size_t)(z + 1) * n + e]);
     X[(size_t)(z + 1) * n + e] = R;
   }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------
+// Both delta rules over many rows, in blocks of CD_C tokens, every sum in f32.  Inside a block that starts from the state S0, with b_t the sum of
+// the decays' logarithms from the block's first token to token t (per key channel; one number per head in mode 0) and G_t = e^(b_t),
+//   S_t = diag(G_t) S0 + sum_(s <= t) (k_s e^(b_t - b_s)) u_s^T
+//   u_t = beta_t (v_t - S0^T (G_t k_t) - sum_(s < t) A_ts u_s),   A_ts = sum_c k_t k_s e^(b_t - b_s)
+//   o_t = S0^T (G_t q_t) + sum_(s <= t) B_ts u_s,                 B_ts = sum_c q_t k_s e^(b_t - b_s)
+// so with the unit lower triangle I + diag(beta) A and T = (I + diag(beta) A)^-1 diag(beta):
+//   U = T (V - Kt S0),   O = Qt S0 + B U,   S <- diag(G_last) S0 + Kb^T U,   Kt = G_t k_t, Qt = G_t q_t, Kb = k_s e^(b_last - b_s).
+// Every exponent is a sum of decays between two tokens, hence never positive; the sums are kept as two floats, so that a difference of two large
+// ones is as good as the sum it stands for.  Three launches: the decays' logarithms row by row (fq3s_mstate_cdelta_prep_kernel; mode 0: none), the
+// records [Kt | Qt | Kb | G_last | T | B] of all (block, head) pairs at once, and one walk over the blocks per (head, DVT state columns): three
+// small dense products per block of tokens instead of a chain of dependent steps per token.  Tokens beyond the last row are empty (k = q = v = 0,
+// beta = 0, no decay).
+// ---------------------------------------------------------------------------------------------------------------------------
+constexpr int CD_C = 16;           // tokens per block
+constexpr int CD_TP = CD_C + 4;    // pitch of T and B
+constexpr int CD_PAIRS = CD_C * (CD_C + 1) / 2, CD_REC_THREADS = (CD_PAIRS + 31) / 32 * 32;
+constexpr int CD_MIN_ROWS = 32;    // fewer rows are walked token by token
+constexpr int CD_MAX_DK = 256;
+__host__ __device__ constexpr int cd_rows(int dk) { return (dk + 15) & ~15; }       // state rows, padded with zeros
+__host__ __device__ constexpr int cd_pitch(int dk) { return cd_rows(dk) + 4; }
+__host__ __device__ constexpr int cd_record(int dk) { return 3 * CD_C * cd_pitch(dk) + cd_rows(dk) + 2 * CD_C * CD_TP; }      // floats, a multiple of four
+__host__ __device__ inline long long cd_log_floats(int M, int H, int dk, bool channels) { return channels ? (long long)M * ((H * dk + 3) & ~3) : 0; }
+__host__ __device__ inline long long cd_ws_floats(int M, int H, int dk, bool channels) {
+  return cd_log_floats(M, H, dk, channels) + (long long)((M + CD_C - 1) / CD_C) * H * cd_record(dk);
+}
+constexpr float LOG2E_F = 1.4426950408889634f;
+// grid (blocks of tokens, H), CD_REC_THREADS threads; dynamic shared memory: sums (two floats), q and k, [CD_C][pitch] each
+__global__ void __launch_bounds__(CD_REC_THREADS) fq3s_cdelta_record_kernel(const fq3c_op o) {
+  extern __shared__ __align__(16) float cr[];
+  __shared__ float beta[CD_C], N[CD_C][CD_C], fq[CD_C], fk[CD_C];
+  const int H = o.i0, G = o.i1, dk = o.i2, h = blockIdx.y, g = h / (H / G), t0 = blockIdx.x * CD_C, tid = threadIdx.x;
+  const int D = cd_rows(dk), P = cd_pitch(dk), nt = min(CD_C, o.M - t0);
+  const bool channels = o.taps == 6;
+  float* bh = cr;
+  float* bl = bh + CD_C * P;
+  float* qs = bl + CD_C * P;
+  float* ks = qs + CD_C * P;
+  const float* raw = reinterpret_cast<const float*>(o.res) + (size_t)t0 * o.ldr;
+  const float* rows = reinterpret_cast<const float*>(o.A) + (size_t)t0 * o.lda;
+  const int lp = (H * dk + 3) & ~3;
+  if (tid < CD_C) beta[tid] = tid < nt ? sigmoid_f(raw[(size_t)tid * o.ldr + o.m_begin + h]) : 0.f;
+  const float rate = channels ? 0.f : LOG2E_F * expf(reinterpret_cast<const float*>(o.scale)[h]);
+  const float dtb = (!channels && o.bias) ? reinterpret_cast<const float*>(o.bias)[h] : 0.f;
+  for (int c = tid; c < D; c += CD_REC_THREADS) {
+    float hi = 0.f, lo = 0.f, l[CD_C];
+#pragma unroll
+    for (int t = 0; t < CD_C; ++t) {
+      const bool ok = t < nt && c < dk;
+      l[t] = !ok ? 0.f : channels ? reinterpret_cast<const float*>(o.ws)[(size_t)(t0 + t) * lp + h * dk + c]
+                                  : -rate * softplus_f(raw[(size_t)t * o.ldr + o.col_mod + h] + dtb);
+      qs[t * P + c] = ok ? rows[(size_t)t * o.lda + g * dk + c] : 0.f;
+      ks[t * P + c] = ok ? rows[(size_t)t * o.lda + o.K + g * dk + c] : 0.f;
+    }
+#pragma unroll
+    for (int t = 0; t < CD_C; ++t) {       // the exact sum of two floats is again two floats; the small part collects
+      const float x = fmaxf(l[t], -1000.f), s = hi + x, bb = s - hi;
+      lo += (hi - (s - bb)) + (x - bb);
+      hi = s;
+      bh[t * P + c] = hi;
+      bl[t * P + c] = lo;
+    }
+  }
+  __syncthreads();
+  const int warp = tid >> 5, lane = tid & 31;
+  for (int v = warp; v < 2 * CD_C; v += CD_REC_THREADS / 32) {
+    const float* x = (v < CD_C ? qs : ks) + (v & (CD_C - 1)) * P;
+    float ss = 0.f;
+    for (int c = lane; c < dk; c += 32) ss = fmaf(x[c], x[c], ss);
+    ss = warp_sum(ss);
+    if (lane == 0) (v < CD_C ? fq : fk)[v & (CD_C - 1)] = (v < CD_C ? 1.f / sqrtf((float)dk) : 1.f) / sqrtf(ss + 1e-6f);
+  }
+  __syncthreads();
+  float* rec = reinterpret_cast<float*>(o.ws) + cd_log_floats(o.M, H, dk, channels) + ((size_t)blockIdx.x * H + h) * cd_record(dk);
+  for (int i = tid; i < CD_C * (D >> 2); i += CD_REC_THREADS) {
+    const int t = i / (D >> 2), c = (i - t * (D >> 2)) * 4, at = t * P + c;
+    const float4 hi = ld4(bh + at), lo = ld4(bl + at), eh = ld4(bh + (CD_C - 1) * P + c), el = ld4(bl + (CD_C - 1) * P + c);
+    float4 q = ld4(qs + at), k = ld4(ks + at);
+    q.x *= fq[t]; q.y *= fq[t]; q.z *= fq[t]; q.w *= fq[t];
+    k.x *= fk[t]; k.y *= fk[t]; k.z *= fk[t]; k.w *= fk[t];
+    *reinterpret_cast<float4*>(qs + at) = q;
+    *reinterpret_cast<float4*>(ks + at) = k;
+    const float4 d = make_float4(exp2f(hi.x), exp2f(hi.y), exp2f(hi.z), exp2f(hi.w));
+    *reinterpret_cast<float4*>(rec + at) = make_float4(k.x * d.x, k.y * d.y, k.z * d.z, k.w * d.w);
+    *reinterpret_cast<float4*>(rec + CD_C * P + at) = make_float4(q.x * d.x, q.y * d.y, q.z * d.z, q.w * d.w);
+    *reinterpret_cast<float4*>(rec + 2 * CD_C * P + at) =
+        make_float4(k.x * exp2f((eh.x - hi.x) + (el.x - lo.x)), k.y * exp2f((eh.y - hi.y) + (el.y - lo.y)),
+                    k.z * exp2f((eh.z - hi.z) + (el.z - lo.z)), k.w * exp2f((eh.w - hi.w) + (el.w - lo.w)));
+    if (t == CD_C - 1) *reinterpret_cast<float4*>(rec + 3 * CD_C * P + c) = d;
+  }
+  __syncthreads();
+  float* Tm = rec + 3 * CD_C * P + D;
+  float* Bm = Tm + CD_C * CD_TP;
+  if (tid < CD_PAIRS) {
+    int t = (int)((sqrtf(8.f * (float)tid + 1.f) - 1.f) * 0.5f);
+    while ((t + 1) * (t + 2) / 2 <= tid) ++t;
+    while (t * (t + 1) / 2 > tid) --t;
+    const int s = tid - t * (t + 1) / 2;
+    float a = 0.f, b = 0.f;
+#pragma unroll 2
+    for (int c = 0; c < D; c += 4) {
+      const float4 ht = ld4(bh + t * P + c), lt = ld4(bl + t * P + c), hs = ld4(bh + s * P + c), ls = ld4(bl + s * P + c);
+      const float4 kt = ld4(ks + t * P + c), k = ld4(ks + s * P + c), q = ld4(qs + t * P + c);
+      const float e0 = k.x * exp2f((ht.x - hs.x) + (lt.x - ls.x)), e1 = k.y * exp2f((ht.y - hs.y) + (lt.y - ls.y));
+      const float e2 = k.z * exp2f((ht.z - hs.z) + (lt.z - ls.z)), e3 = k.w * exp2f((ht.w - hs.w) + (lt.w - ls.w));
+      a = fmaf(kt.x, e0, a); b = fmaf(q.x, e0, b);
+      a = fmaf(kt.y, e1, a); b = fmaf(q.y, e1, b);
+      a = fmaf(kt.z, e2, a); b = fmaf(q.z, e2, b);
+      a = fmaf(kt.w, e3, a); b = fmaf(q.w, e3, b);
+    }
+    N[t][s] = beta[t] * a;
+    Bm[t * CD_TP + s] = b;
+    if (s < t) { Bm[s * CD_TP + t] = 0.f; Tm[s * CD_TP + t] = 0.f; }
+  }
+  __syncthreads();
+  if (tid < CD_C) {       // column tid of T by forward substitution
+    float x[CD_C];
+#pragma unroll
+    for (int t = 0; t < CD_C; ++t) {
+      float v = t == tid ? beta[t] : 0.f;
+#pragma unroll
+      for (int s = 0; s < t; ++s) v = fmaf(-N[t][s], x[s], v);
+      x[t] = v;
+      if (t >= tid) Tm[t * CD_TP + tid] = v;
+    }
+  }
+}
+
+// grid (ceil(dv / DVT), H), 128 threads.  The state tile [D rows, DVT columns] lives in registers (four rows x two columns x RQ per thread) and, as
+// the operand of the next block's products, transposed in shared memory.  [Kt; Qt] S0: a warp takes a quarter of the state rows for all 2 CD_C x DVT
+// sums (a lane: rows r, r + 8, r + 16, r + 24 and every fourth column), the quarters are added where the sums are used.  U and O: a lane per
+// (token, column).  Records arrive by cp.async, one block of tokens ahead.
+template <int DVT>
+__host__ __device__ constexpr int cd_walk_floats(int dk) {
+  return 2 * cd_record(dk) + DVT * cd_pitch(dk) + 4 * 2 * CD_C * (DVT + 1) + DVT * CD_TP + 2 * CD_C * DVT + 4;
+}
+template <int DVT, int RQ>
+__global__ void __launch_bounds__(128) fq3s_cdelta_walk_kernel(const fq3c_op o) {
+  extern __shared__ __align__(16) float cw[];
+  constexpr int NCP = DVT / 2, QS = 128 / NCP, NC = DVT / 4, PP = DVT + 1, JW = DVT / 4;
+  const int H = o.i0, dk = o.i2, dv = o.cin, h = blockIdx.y, j0 = blockIdx.x * DVT, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int D = cd_rows(dk), P = cd_pitch(dk), REC = cd_record(dk), nblk = (o.M + CD_C - 1) / CD_C;
+  float* St = cw + 2 * REC;                          // [DVT][P]
+  float* Ud = St + DVT * P;                          // [CD_C][DVT] pairs (u, u)
+  float* Xs = Ud + 2 * CD_C * DVT;                   // [DVT][CD_TP]
+  float* Pp = Xs + DVT * CD_TP;                      // [4][2 CD_C][PP]
+  const float* recs = reinterpret_cast<const float*>(o.ws) + cd_log_floats(o.M, H, dk, o.taps == 6) + (size_t)h * REC;
+  auto fetch = [&](const int n) {
+    const float* src = recs + (size_t)n * H * REC;
+    float* dst = cw + (n & 1) * REC;
+    for (int i = tid * 4; i < REC; i += 512) cp_async16(dst + i, src + i, true);
+    cp_async_commit();
+  };
+  fetch(0);
+  // this thread's part of the state: rows rq + q QS (quads), columns 2 cp, 2 cp + 1
+  const int cp = tid % NCP, rq = tid / NCP;
+  f32x2 S[RQ][2][2];          // [quad][column][row pair]
+  const float* st = reinterpret_cast<const float*>(o.p0) + (size_t)h * dk * dv;
+#pragma unroll
+  for (int q = 0; q < RQ; ++q)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int r = (rq + q * QS) * 4, c = j0 + 2 * cp + j;
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = (r + e < dk && c < dv) ? st[(size_t)(r + e) * dv + c] : 0.f;
+      S[q][j][0] = pack2(v[0], v[1]);
+      S[q][j][1] = pack2(v[2], v[3]);
+      if (r < D) *reinterpret_cast<float4*>(St + (2 * cp + j) * P + r) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+  // this thread's (token, column) pairs of U and O: token lane % 16, columns warp JW + lane / 16 (+ 2)
+  const int t = lane & (CD_C - 1), jb = warp * JW + (lane >> 4);
+  const float* vrow = reinterpret_cast<const float*>(o.A) + o.a_rows + (size_t)h * dv + j0;
+  float vn[JW / 2];
+  auto load_v = [&](const int n) {
+#pragma unroll
+    for (int e = 0; e < JW / 2; ++e) {
+      const int m = n * CD_C + t, j = jb + 2 * e;
+      vn[e] = (m < o.M && j0 + j < dv) ? __ldg(vrow + (size_t)m * o.lda + j) : 0.f;
+    }
+  };
+  load_v(0);
+  const int rl = lane & 7, cl = lane >> 3, KW = D >> 2;      // products: rows rl + 8 i of [Kt; Qt], columns cl + 4 i
+  for (int n = 0; n < nblk; ++n) {
+    cp_async_wait<0>();
+    __syncthreads();           // the record is there, the transposed state too; everyone is done with the other buffer
+    if (n + 1 < nblk) fetch(n + 1);
+    const float* rec = cw + (n & 1) * REC;
+    {
+      f32x2 acc[4][NC];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < NC; ++j) acc[i][j] = 0ull;
+      const float* kr = rec + rl * P + warp * KW;
+      const float* sr = St + cl * P + warp * KW;
+#pragma unroll 2
+      for (int k = 0; k < KW; k += 4) {
+        ulonglong2 a[4], b[NC];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const ulonglong2*>(kr + 8 * i * P + k);
+#pragma unroll
+        for (int j = 0; j < NC; ++j) b[j] = *reinterpret_cast<const ulonglong2*>(sr + 4 * j * P + k);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < NC; ++j) {
+            acc[i][j] = fma2<true>(a[i].x, b[j].x, acc[i][j]);
+            acc[i][j] = fma2<true>(a[i].y, b[j].y, acc[i][j]);
+          }
+      }
+      float* pw = Pp + warp * 2 * CD_C * PP;
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < NC; ++j) pw[(rl + 8 * i) * PP + cl + 4 * j] = lo2(acc[i][j]) + hi2(acc[i][j]);
+    }
+    __syncthreads();
+    const float* Tm = rec + 3 * CD_C * P + D;
+    const float* Bm = Tm + CD_C * CD_TP;
+    auto quarters = [&](const int r, const int j) {
+      const float* p = Pp + r * PP + j;
+      return (p[0] + p[2 * CD_C * PP]) + (p[4 * CD_C * PP] + p[6 * CD_C * PP]);
+    };
+    auto row_times = [&](const float* m, const int j) {       // sum_s m[t][s] Xs[j][s]
+      const float* x = Xs + j * CD_TP;
+      float a = 0.f, b = 0.f;
+#pragma unroll
+      for (int s = 0; s < CD_C; s += 4) {
+        const float4 mv = ld4(m + t * CD_TP + s), xv = ld4(x + s);
+        a = fmaf(mv.x, xv.x, a); b = fmaf(mv.y, xv.y, b);
+        a = fmaf(mv.z, xv.z, a); b = fmaf(mv.w, xv.w, b);
+      }
+      return a + b;
+    };
+    float u[JW / 2];
+#pragma unroll
+    for (int e = 0; e < JW / 2; ++e) Xs[(jb + 2 * e) * CD_TP + t] = vn[e] - quarters(t, jb + 2 * e);
+    __syncwarp();
+#pragma unroll
+    for (int e = 0; e < JW / 2; ++e) u[e] = row_times(Tm, jb + 2 * e);
+    __syncwarp();
+#pragma unroll
+    for (int e = 0; e < JW / 2; ++e) {
+      Xs[(jb + 2 * e) * CD_TP + t] = u[e];
+      *reinterpret_cast<float2*>(Ud + 2 * (t * DVT + jb + 2 * e)) = make_float2(u[e], u[e]);
+    }
+    if (n + 1 < nblk) load_v(n + 1);
+    __syncthreads();
+    {   // S <- diag(G_last) S + Kb^T U
+      const float* Kb = rec + 2 * CD_C * P;
+      const float* Gl = rec + 3 * CD_C * P;
+#pragma unroll
+      for (int q = 0; q < RQ; ++q) {
+        const int r = (rq + q * QS) * 4;
+        if (r >= D) continue;
+        const ulonglong2 gl = *reinterpret_cast<const ulonglong2*>(Gl + r);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) { S[q][j][0] = mul2<true>(gl.x, S[q][j][0]); S[q][j][1] = mul2<true>(gl.y, S[q][j][1]); }
+#pragma unroll
+        for (int s = 0; s < CD_C; ++s) {
+          const ulonglong2 kb = *reinterpret_cast<const ulonglong2*>(Kb + s * P + r);
+          const ulonglong2 uu = *reinterpret_cast<const ulonglong2*>(Ud + 2 * (s * DVT + 2 * cp));
+          S[q][0][0] = fma2<true>(kb.x, uu.x, S[q][0][0]);
+          S[q][0][1] = fma2<true>(kb.y, uu.x, S[q][0][1]);
+          S[q][1][0] = fma2<true>(kb.x, uu.y, S[q][1][0]);
+          S[q][1][1] = fma2<true>(kb.y, uu.y, S[q][1][1]);
+        }
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+          *reinterpret_cast<ulonglong2*>(St + (2 * cp + j) * P + r) = make_ulonglong2(S[q][j][0], S[q][j][1]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < JW / 2; ++e) {       // O = Qt S0 + B U
+      const int j = jb + 2 * e, m = n * CD_C + t;
+      const float ov = quarters(CD_C + t, j) + row_times(Bm, j);
+      if (m < o.M && j0 + j < dv) reinterpret_cast<float*>(o.C)[(size_t)m * o.ldc + (size_t)h * dv + j0 + j] = ov;
+    }
+  }
+  float* nst = reinterpret_cast<float*>(o.C2) + (size_t)h * dk * dv;
+#pragma unroll
+  for (int q = 0; q < RQ; ++q)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int r = (rq + q * QS) * 4, c = j0 + 2 * cp + j;
+      const float v[4] = {lo2(S[q][j][0]), hi2(S[q][j][0]), lo2(S[q][j][1]), hi2(S[q][j][1])};
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (r + e < dk && c < dv) nst[(size_t)(r + e) * dv + c] = v[e];
+    }
 }
 
 // ===========================================================================================================================

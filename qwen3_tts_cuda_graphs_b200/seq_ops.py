@@ -402,18 +402,25 @@ class StepBuilder:
         return oa
 
     # ---- recurrences with a matrix state per head -----------------------------------------------------
-    def _scan_ws(self, coef_cols: int, H: int, dk: int, dv: int, pieces: bool = True) -> torch.Tensor:
+    def _scan_ws(self, coef_cols: int, H: int, dk: int, dv: int) -> torch.Tensor:
         """Workspace of a matrix-state scan: per-row coefficients [M, coef_cols], and for a long run of rows (state-independent
         decays only) room for up to 16 pieces' start states and decay products, which lets the library walk the pieces side by side."""
         n = -(-(self.M * coef_cols) // 4) * 4
-        if pieces and self.M >= 512:
+        if self.M >= 512:
             n += 16 * H * dk * (dv + 1)
         return self.buf("ms.ws", 1, max(n, 4))
+
+    def _delta_ws(self, coef_cols: int, H: int, dk: int, log_cols: int) -> torch.Tensor:
+        """Workspace of a delta rule: the rows of the walk token by token, or, for many rows, room for the records of the walk in blocks of
+        16 tokens (cd_record of csrc/fq3_seq.cuh: three operands of 16 rows, the last decays, two 16 x 16 matrices) behind the decay rows."""
+        d16 = -(-dk // 16) * 16
+        blocks = -(-self.M // 16) * H * (48 * (d16 + 4) + d16 + 640) + self.M * log_cols if self.M >= 32 else 0
+        return self.buf("ms.ws", 1, max(self.M * coef_cols, blocks, 4))
 
     def _mstate(self, mode: int, rows: torch.Tensor, raw: torch.Tensor, H: int, G: int, dk: int, dv: int, kcol: int, vcol: int,
                 decay_col: int, write_col: int, w: dict, state: str, y: torch.Tensor):
         wcols = -(-(2 * H + (2 * G * dk + G if mode == 0 else 0)) // 4) * 4      # rows padded to 16 bytes
-        ws = self._scan_ws(wcols, H, dk, dv, pieces=mode != 0)
+        ws = self._scan_ws(wcols, H, dk, dv) if mode != 0 else self._delta_ws(wcols, H, dk, 0)
         kw = dict(M=self.M, N=H * dv, taps=mode, i0=H, i1=G, i2=dk, cin=dv, K=kcol, a_rows=vcol, A=rows, lda=rows.shape[1], res=raw,
                   ldr=raw.shape[1], col_mod=decay_col, m_begin=write_col, scale=w["A_log"], bias=w["dt_bias"],
                   p0=self.slot.cur[state], C2=self.slot.next[state], C=y, ldc=y.shape[1], ws=ws, ws_bytes=ws.numel() * 4, flags=F_OUT_F32)
@@ -483,7 +490,7 @@ class StepBuilder:
         M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
         ra, rg = w["a2"].shape[1], w["g2"].shape[1]
         y, gate = self.buf("kd.y", M, H * dv), self.buf("kd.gate", M, H * dv)
-        ws = self._scan_ws(-(-((2 * G + H) * d + H + G) // 4) * 4, H, d, dv, pieces=False)
+        ws = self._delta_ws(-(-((2 * G + H) * d + H + G) // 4) * 4, H, d, -(-(H * d) // 4) * 4)
         self.plan.keep += [cv, raw]
         op = self._op(K_MSTATE_SCAN, M=M, N=H * dv, taps=6, i0=H, i1=G, i2=d, cin=dv, K=G * d, a_rows=2 * G * d, A=_ptr(cv, ccol), lda=cv.shape[1],
                       res=raw, ldr=raw.shape[1], m_begin=rcol, col_mod=rcol + H, B=w["a2"], bias=w["dt_bias"], scale=w["A_log"], p1=w["g2"],
