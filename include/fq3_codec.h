@@ -157,7 +157,11 @@ enum fq3c_kind {
                          one buffer; C may be slice 0), p0 = f32 [i0] on the device.  With norm_out: norm_out[m, :] (bf16; f32 with
                          FQ3C_F32; pitch norm_ld) = n(C[m, :]) * norm_w (f32 [N]), n = v / sqrt(mean(v^2) + norm_eps), or, with
                          FQ3C_CENTER, (v - mean) / sqrt(mean((v - mean)^2) + norm_eps).  One block per row; the statistics are taken
-                         in two passes over the row kept in shared memory                                                          */
+                         in two passes over the row kept in shared memory                                                          */,
+  /* ---- ABI 11 */
+  FQ3C_BRANCH = 33    /* two independent parts of a list side by side: i0 = 0 opens a side stream behind everything launched so far, the
+                         following ops go there; i0 = 1: the following ops go to the main stream again; i0 = 2: the main stream waits for
+                         the side stream (at the end of a list this happens by itself).  A captured list keeps both as graph branches.  M = 1 */
   /* ABI 9 also adds to existing kinds:
    *   FQ3C_GNORM: FQ3C_CENTER (the statistics are mean and variance: a layer norm without bias); scale may be NULL (no weights).
    *   FQ3C_ROT_APPEND: FQ3C_ROT_HALF pairs entry i with entry i + taps / 2 instead of 2i with 2i + 1.
@@ -204,13 +208,13 @@ enum fq3c_kind {
    *     the output.
    *   FQ3C_MSTATE_SCAN: taps = 6 (delta rule with a decay per key channel): rows A = queries of group g at column g * i2, keys at
    *     K + g * i2, values of head h at a_rows + h * cin; raw rows res (f32, pitch ldr): decay latent (tap_off[0] entries) at column col_mod,
-   *     write-strength input of head h at m_begin + h;  z = B lat + bias with B [i0 * i2, tap_off[0]] (bf16; FQ3C_F32: f32), bias f32 [i0 * i2];
+   *     write-strength input of head h at m_begin + h;  z = B^T lat + bias with B [tap_off[0], i0 * i2] (bf16; FQ3C_F32: f32), bias f32 [i0 * i2];
    *       q, k <- unit vectors as for taps = 0;  g = exp(-exp(scale[h]) softplus(z)) per head and key channel;  beta = sigmoid(b);
    *       S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  C = S^T q.
-   *     tap_off[2] = R > 0: a second up-projection in the same launch: norm_out (f32 [M, i0 * cin], pitch norm_ld) = p1 lat2 with p1
-   *     [i0 * cin, R] (B's type) and lat2 at column tap_off[1] of the rows res.  ws = f32 [M, round_up(2 * i1 * i2 + i0 * i2 + i0 + i1, 4)].
+   *     tap_off[2] = R > 0: a second up-projection in the same launch: norm_out (f32 [M, i0 * cin], pitch norm_ld) = p1^T lat2 with p1
+   *     [R, i0 * cin] (B's type) and lat2 at column tap_off[1] of the rows res.  ws = f32 [M, round_up(2 * i1 * i2 + i0 * i2 + i0 + i1, 4)].
    *     Both delta rules (taps 0 and 6), M >= 32 and i2 <= 256: when ws also has room for them (M * round_up(i0 * i2, 4) floats of decay
-   *     logarithms for taps = 6, then ceil(M / 16) * i0 records of 48 (D + 4) + D + 640 floats, D = i2 rounded up to 16), the rows are walked
+   *     logarithms for taps = 6, then ceil(M / 16) * i0 records of 48 (D + 4) + D + 640 floats, D = i2 rounded up to 32), the rows are walked
    *     in blocks of 16 tokens: same recurrence, other order of the sums.  */
 };
 
@@ -280,6 +284,8 @@ const char* fq3c_last_error(void);
 int fq3c_run(const fq3c_op* ops, int n_ops, void* stream);
 /* number of kernel launches issued so far by this process through fq3c_run / fq3c_graph_launch */
 int64_t fq3c_launch_count(void);
+/* ABI 11: nonzero when a kernel's bounded wait for its own copy ran out on the current device (its outputs are NaN); synchronises */
+int fq3c_wait_errors(void);
 /* A decode plan is static for a given frame count: capture its launches once (stream capture of fq3c_run) and replay
  * them as one CUDA graph.  The ops' buffers must stay alive and at the same addresses for the life of the graph. */
 int fq3c_graph_create(const fq3c_op* ops, int n_ops, void** out_graph);

@@ -36,6 +36,7 @@ K_COPY, K_ADVANCE, K_ROLL = 9, 10, 11
 K_DYT, K_DEPTH_MIX, K_XIELU, K_ROT_APPEND, K_CACHE_ATTN, K_MSTATE_SCAN = range(24, 30)
 K_HYPER, K_GLU = 30, 31
 K_SUM_NORM = 32
+K_BRANCH = 33
 F_BIAS, F_GELU, F_RESID, F_SCALE, F_SWIGLU, F_CLAMP, F_OUT_F32, F_SNAKE2, F_SILU = 1, 2, 4, 8, 16, 32, 64, 128, 256
 F_F32, F_NOROUND, F_GELU_TANH, F_SIGMOID, F_A_F32 = 512, 1024, 2048, 4096, 8192
 F_GATE_PRE, F_GATE_POST = 16384, 32768
@@ -146,6 +147,7 @@ def load_lib():
     lib.fq3c_run.restype = C.c_int
     lib.fq3c_run.argtypes = [C.POINTER(Op), C.c_int, C.c_void_p]
     lib.fq3c_launch_count.restype = C.c_int64
+    lib.fq3c_wait_errors.restype = C.c_int
     lib.fq3c_graph_create.restype = C.c_int
     lib.fq3c_graph_create.argtypes = [C.POINTER(Op), C.c_int, C.POINTER(C.c_void_p)]
     lib.fq3c_graph_launch.restype = C.c_int

@@ -1300,15 +1300,16 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
       if (!o.A || !o.p0 || !o.C) return fail("xielu: missing operand");
       fq3s_xielu_kernel<<<dim3((o.N + 255) / 256, o.M), 256, 0, s>>>(o);
       return 0;
-    case FQ3C_ROT_APPEND:
+    case FQ3C_ROT_APPEND: {
       if (!o.A || o.i0 < 0 || o.i1 < 0 || o.i2 < 1 || o.taps < 0 || (o.taps & 1) || o.taps > o.i2 || (o.taps > 0 && !o.B) ||
           (o.i1 > 0 && (!o.C || (o.cin > 0 && !o.C2))))
         return fail("rot_append: bad configuration");
       if (o.m_begin > 0 && (o.i1 < 1 || o.cin < 1 || !o.norm_out || !o.ws || !o.p0)) return fail("rot_append: pooled blocks need both caches, their pooled rows and a position");
-      if (o.m_begin > 0 && o.M == 1 && (o.flags & FQ3C_F32)) fq3s_rot_append_kernel<float, true><<<1, 256, 0, s>>>(o);
-      else if (o.m_begin > 0 && o.M == 1) fq3s_rot_append_kernel<bf16, true><<<1, 256, 0, s>>>(o);
-      else if (o.flags & FQ3C_F32) fq3s_rot_append_kernel<float><<<o.M, 256, 0, s>>>(o);
-      else fq3s_rot_append_kernel<bf16><<<o.M, 256, 0, s>>>(o);
+      const int rth = o.M <= 8 ? std::max(256, std::min(1024, 32 * (o.i0 + o.i1))) : 256;      // few rows: a warp per head
+      if (o.m_begin > 0 && o.M == 1 && (o.flags & FQ3C_F32)) fq3s_rot_append_kernel<float, true><<<1, rth, 0, s>>>(o);
+      else if (o.m_begin > 0 && o.M == 1) fq3s_rot_append_kernel<bf16, true><<<1, rth, 0, s>>>(o);
+      else if (o.flags & FQ3C_F32) fq3s_rot_append_kernel<float><<<o.M, rth, 0, s>>>(o);
+      else fq3s_rot_append_kernel<bf16><<<o.M, rth, 0, s>>>(o);
       if (o.m_begin > 0 && o.M > 1) {
         const dim3 grid(o.M / o.m_begin + 1, (o.i1 * std::max(o.i2, o.cin) + 255) / 256, 2);
         if (o.flags & FQ3C_F32) fq3s_pool_append_kernel<float><<<grid, 256, 0, s>>>(o);
@@ -1316,6 +1317,7 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         count_launches(1);
       }
       return 0;
+    }
     case FQ3C_CACHE_ATTN: {
       if (o.i0 < 1 || o.i1 < 1 || o.i0 % o.i1 || o.i2 < 1 || o.cin < 1 || !o.A || !o.B || !o.p1 || !o.C) return fail("cache_attn: bad configuration");
       const int splits = std::max(1, o.m_begin), HG = o.i0 / o.i1;
@@ -1441,10 +1443,11 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         fq3s_mstate_max_kernel<<<o.i0, MM_THREADS, 0, s>>>(o);
         count_launches(1);
       } else if (o.taps == 6) {
-        const dim3 grid((o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS, (o.i0 * o.i2 + 255) / 256 + (o.tap_off[2] > 0 ? (o.i0 * o.cin + 255) / 256 : 0) + (blocks ? 0 : 1));
+        const int nth = o.M <= 8 ? 64 : 256, per = 2 * nth;      // few rows: more, smaller blocks
+        const dim3 grid((o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS, (o.i0 * o.i2 + per - 1) / per + (o.tap_off[2] > 0 ? (o.i0 * o.cin + per - 1) / per : 0) + (blocks ? 0 : 1));
         const size_t smem = sizeof(float) * MS_PREP_ROWS * (size_t)std::max(o.tap_off[0], o.tap_off[2]);
-        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, 256, smem, s>>>(o, false);
-        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, 256, smem, s>>>(o, blocks);
+        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, nth, smem, s>>>(o, false);
+        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, nth, smem, s>>>(o, blocks);
         count_launches(1);
       } else if (o.taps < 3 && !blocks) {
         fq3s_mstate_prep_kernel<<<o.taps == 2 ? (o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS : o.M, 128, 0, s>>>(o);
@@ -1485,11 +1488,12 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         // narrow state tiles while they do not outnumber the SMs, wide ones otherwise and for few state rows
         const bool narrow = o.i2 > 64 && o.i0 * ((o.cin + 7) / 8) <= 148;
         const dim3 grid((o.cin + (narrow ? 7 : 15)) / (narrow ? 8 : 16), o.i0);
-        if (narrow && o.i2 <= 128) fq3s_cdelta_walk_kernel<8, 1><<<grid, 128, cd_walk_floats<8>(o.i2) * 4, s>>>(o);
-        else if (narrow) fq3s_cdelta_walk_kernel<8, 2><<<grid, 128, cd_walk_floats<8>(o.i2) * 4, s>>>(o);
-        else if (o.i2 <= 64) fq3s_cdelta_walk_kernel<16, 1><<<grid, 128, cd_walk_floats<16>(o.i2) * 4, s>>>(o);
-        else if (o.i2 <= 128) fq3s_cdelta_walk_kernel<16, 2><<<grid, 128, cd_walk_floats<16>(o.i2) * 4, s>>>(o);
-        else fq3s_cdelta_walk_kernel<16, 4><<<grid, 128, cd_walk_floats<16>(o.i2) * 4, s>>>(o);
+        const size_t wsm = (narrow ? cd_walk_floats<8>(o.i2) : cd_walk_floats<16>(o.i2)) * 4;
+        if (narrow && o.i2 <= 128) fq3s_cdelta_walk_kernel<8, 1><<<grid, CD_WALK_THREADS, wsm, s>>>(o);
+        else if (narrow) fq3s_cdelta_walk_kernel<8, 2><<<grid, CD_WALK_THREADS, wsm, s>>>(o);
+        else if (o.i2 <= 64) fq3s_cdelta_walk_kernel<16, 1><<<grid, CD_WALK_THREADS, wsm, s>>>(o);
+        else if (o.i2 <= 128) fq3s_cdelta_walk_kernel<16, 2><<<grid, CD_WALK_THREADS, wsm, s>>>(o);
+        else fq3s_cdelta_walk_kernel<16, 4><<<grid, CD_WALK_THREADS, wsm, s>>>(o);
         return 0;
       }
       // Long runs of a recurrence whose decays do not depend on the state: pieces walked twice (see the kernel), when the caller's
@@ -1584,6 +1588,10 @@ extern "C" {
 int fq3c_abi_version(void) { return 11; }
 const char* fq3c_last_error(void) { return g_err.c_str(); }
 int64_t fq3c_launch_count(void) { return g_launches.load(); }
+int fq3c_wait_errors(void) {
+  int v = 0;
+  return cudaMemcpyFromSymbol(&v, seq_wait_error, sizeof v) == cudaSuccess ? v : -1;
+}
 
 // Opt-in shared-memory sizes are a per-DEVICE function attribute: a process that serves several GPUs (server.py --gpus N: one scheduler
 // thread per device) must set them on each device it launches on, not once per process.
@@ -1602,12 +1610,58 @@ static bool device_attrs_ready() {
   return true;
 }
 
+// The side stream of FQ3C_BRANCH and its two events, per host thread and device: lists that run in several threads never share one.
+struct SideStream { cudaStream_t stream = nullptr; cudaEvent_t begun = nullptr, done = nullptr; };
+static SideStream* side_stream() {
+  static thread_local SideStream sides[64];
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return nullptr;
+  SideStream& e = sides[dev];
+  if (e.done) return &e;
+  if ((!e.stream && cudaStreamCreateWithFlags(&e.stream, cudaStreamNonBlocking) != cudaSuccess) ||
+      (!e.begun && cudaEventCreateWithFlags(&e.begun, cudaEventDisableTiming) != cudaSuccess) ||
+      cudaEventCreateWithFlags(&e.done, cudaEventDisableTiming) != cudaSuccess) {
+    e.done = nullptr;
+    cudaGetLastError();
+    return nullptr;
+  }
+  return &e;
+}
+static int run_ops(const fq3c_op* ops, int n_ops, cudaStream_t main_stream, SideStream*& open);
 int fq3c_run(const fq3c_op* ops, int n_ops, void* stream) {
-  cudaStream_t s = (cudaStream_t)stream;
+  SideStream* open = nullptr;
+  const int rc = run_ops(ops, n_ops, (cudaStream_t)stream, open);
+  if (open && (cudaEventRecord(open->done, open->stream) != cudaSuccess || cudaStreamWaitEvent((cudaStream_t)stream, open->done, 0) != cudaSuccess))
+    return rc != 0 ? rc : fail("branch: join failed");      // a list (or an error) that left the side stream open
+  return rc;
+}
+static int run_ops(const fq3c_op* ops, int n_ops, cudaStream_t main_stream, SideStream*& open) {
+  cudaStream_t s = main_stream;
   for (int i = 0; i < n_ops; ++i) {
     const fq3c_op& o = ops[i];
     if (o.M <= 0) continue;
     switch (o.kind) {
+      case FQ3C_BRANCH: {
+        if (o.i0 == 0) {
+          if (open) return fail("branch: one side stream at a time");
+          SideStream* side = side_stream();
+          if (!side || cudaEventRecord(side->begun, main_stream) != cudaSuccess || cudaStreamWaitEvent(side->stream, side->begun, 0) != cudaSuccess)
+            return fail("branch: cannot open the side stream");
+          open = side;
+          s = side->stream;
+        } else if (o.i0 == 1) {
+          s = main_stream;
+        } else {
+          s = main_stream;
+          if (open) {
+            SideStream* side = open;
+            open = nullptr;
+            if (cudaEventRecord(side->done, side->stream) != cudaSuccess || cudaStreamWaitEvent(main_stream, side->done, 0) != cudaSuccess)
+              return fail("branch: join failed");
+          }
+        }
+        continue;
+      }
       case FQ3C_GEMM: {
         // True 32-bit operands, few rows (decode: weight streaming, one warp per output column) and shapes the tensor-core
         // kernels do not take (K not a multiple of 8, unaligned rows) go to the sequence-model product.
@@ -1788,6 +1842,7 @@ int fq3c_graph_create(const fq3c_op* ops, int n_ops, void** out) {
   cudaStream_t cs;
   if (cudaStreamCreateWithFlags(&cs, cudaStreamNonBlocking) != cudaSuccess) return fail("graph: stream create failed");
   const int64_t before = t_launches;
+  side_stream();      // made before the capture begins
   cudaGraph_t g = nullptr;
   cudaError_t e = cudaStreamBeginCapture(cs, cudaStreamCaptureModeThreadLocal);
   int rc = 0;

@@ -1464,7 +1464,7 @@ __global__ void __launch_bounds__(256) fq3s_pool_append_kernel(const fq3c_op o) 
   else pool_run<TC>(reinterpret_cast<const TC*>(o.C2), o.ldr, reinterpret_cast<TC*>(o.ws), b, P, c, min(n, c + 1), 1);
 }
 
-// grid (M), 256 threads, a warp per query / key head.  Angles in f32: position (exact as a float below 2^24) times the frequency,
+// grid (M), 256 threads (up to 1024 for a few rows), a warp per query / key head.  Angles in f32: position (exact as a float below 2^24) times the frequency,
 // full-range sincosf; cos and sin times the amplitude f1 when that is set.  With norm weights a head is first divided by its root
 // mean square (eps f0) and multiplied by them; with FQ3C_UNIT it is divided only (a rotation keeps the root mean square, so it does
 // not matter which comes first).  Queries in place, keys (read from `res` rows when given) into the cache.
@@ -1472,7 +1472,7 @@ __global__ void __launch_bounds__(256) fq3s_pool_append_kernel(const fq3c_op o) 
 // row b of norm_out / ws.  A single row does it here (POOL; its block has just written the run's last row); more rows take
 // fq3s_pool_append_kernel behind this launch.
 template <typename TC, bool POOL = false>
-__global__ void __launch_bounds__(256) fq3s_rot_append_kernel(const fq3c_op o) {
+__global__ void __launch_bounds__(1024) fq3s_rot_append_kernel(const fq3c_op o) {
   const int m = blockIdx.x, H = o.i0, G = o.i1, d = o.i2, dv = o.cin, half = o.taps >> 1;
   const int pos = (o.p0 ? *reinterpret_cast<const int*>(o.p0) : 0) + m;
   float* row = const_cast<float*>(reinterpret_cast<const float*>(o.A)) + (size_t)m * o.lda;
@@ -2110,91 +2110,94 @@ __global__ void __launch_bounds__(128) fq3s_mstate_prep_kernel(const fq3c_op o) 
 }
 
 // mode 6: ws row m = unit q [G * dk] | unit k [G * dk] | decays [H * dk] | write strengths [H] | q.k [G].  A block takes MS_PREP_ROWS rows (ROWS:
-// how many of them it computes, 1 in decoding) and one share of the columns (grid.y): 256 channels of the decays' up-projection, 256 channels of
-// the gate's, or, the last one, the unit vectors with their products and the write strengths.  A row of an up-projection is loaded once for all
-// rows of the block, whose latents lie transposed in shared memory (sixteen-byte broadcasts).  Dynamic shared memory: 8 x the larger inner size.
+// how many of them it computes, 1 in decoding) and one share of the columns (grid.y): two channels per thread of the decays' up-projection, or
+// of the gate's, or, the last one, the unit vectors with their products and the write strengths.  The up-projections lie transposed [inner size,
+// channels]: neighbouring threads load neighbouring entries, each once for all rows of the block, whose latents lie transposed in shared memory
+// (sixteen-byte broadcasts).  Dynamic shared memory: 8 x the larger inner size.
 __host__ __device__ inline int mstate_cdelta_cols(int H, int G, int dk) { return ((2 * G + H) * dk + H + G + 3) & ~3; }
 template <int ROWS>
-__device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, const void* U, const int c, const int R, float (&z)[ROWS]) {
+__device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, const void* U, const int c, const int n, const int R, float (&z)[2][ROWS]) {
 #pragma unroll
-  for (int j = 0; j < ROWS; ++j) z[j] = 0.f;
-  auto add = [&](const float uv, const int r) {
+  for (int j = 0; j < ROWS; ++j) { z[0][j] = 0.f; z[1][j] = 0.f; }
+  const bool two = c + 1 < n;
+  auto add = [&](const float u0, const float u1, const int r) {
+    float l[ROWS];
     if (ROWS == 8) {
       const float4 a = *reinterpret_cast<const float4*>(lat + r * 8), b = *reinterpret_cast<const float4*>(lat + r * 8 + 4);
-      const float l[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+      l[0] = a.x; l[1 % ROWS] = a.y; l[2 % ROWS] = a.z; l[3 % ROWS] = a.w; l[4 % ROWS] = b.x; l[5 % ROWS] = b.y; l[6 % ROWS] = b.z; l[7 % ROWS] = b.w;
+    } else l[0] = lat[r * 8];
 #pragma unroll
-      for (int j = 0; j < ROWS; ++j) z[j] = fmaf(l[j], uv, z[j]);
-    } else {
-#pragma unroll
-      for (int j = 0; j < ROWS; ++j) z[j] = fmaf(lat[r * 8 + j], uv, z[j]);
-    }
+    for (int j = 0; j < ROWS; ++j) { z[0][j] = fmaf(l[j], u0, z[0][j]); z[1][j] = fmaf(l[j], u1, z[1][j]); }
   };
   if (o.flags & FQ3C_F32) {
-    const float* u = reinterpret_cast<const float*>(U) + (size_t)c * R;
-#pragma unroll 4
-    for (int r = 0; r < R; ++r) add(u[r], r);
+    const float* u = reinterpret_cast<const float*>(U) + c;
+#pragma unroll 8
+    for (int r = 0; r < R; ++r) add(u[(size_t)r * n], two ? u[(size_t)r * n + 1] : 0.f, r);
     return;
   }
-  const bf16* u = reinterpret_cast<const bf16*>(U) + (size_t)c * R;
-  if (R % 8 == 0 && !(reinterpret_cast<uintptr_t>(U) & 15)) {
-#pragma unroll 2
-    for (int r = 0; r < R; r += 8) {
-      const uint4 p = __ldg(reinterpret_cast<const uint4*>(u + r));
-      const uint32_t w[4] = {p.x, p.y, p.z, p.w};
-#pragma unroll
-      for (int q = 0; q < 4; ++q) { add(__uint_as_float(w[q] << 16), r + 2 * q); add(__uint_as_float(w[q] & 0xffff0000u), r + 2 * q + 1); }
+  const bf16* u = reinterpret_cast<const bf16*>(U) + c;
+  if (n % 2 == 0 && !(reinterpret_cast<uintptr_t>(U) & 3)) {
+#pragma unroll 16
+    for (int r = 0; r < R; ++r) {
+      const uint32_t w = __ldg(reinterpret_cast<const uint32_t*>(u + (size_t)r * n));
+      add(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u), r);
     }
   } else {
-    for (int r = 0; r < R; ++r) add(__bfloat162float(u[r]), r);
+    for (int r = 0; r < R; ++r) add(__bfloat162float(u[(size_t)r * n]), two ? __bfloat162float(u[(size_t)r * n + 1]) : 0.f, r);
   }
 }
 // With `logs` the rows hold the base-2 logarithms of the decays alone (pitch round_up(H * dk, 4)), for the walk in blocks of tokens.
 template <int ROWS>
 __global__ void __launch_bounds__(256) fq3s_mstate_cdelta_prep_kernel(const fq3c_op o, const bool logs) {
   extern __shared__ __align__(16) float cd_lat[];       // [inner size][8]
-  const int H = o.i0, G = o.i1, dk = o.i2, m0 = blockIdx.x * MS_PREP_ROWS, nr = min(ROWS, o.M - m0), tid = threadIdx.x;
-  const int nd = (H * dk + 255) / 256, ng = o.tap_off[2] > 0 ? (H * o.cin + 255) / 256 : 0, y = blockIdx.y;
+  const int H = o.i0, G = o.i1, dk = o.i2, m0 = blockIdx.x * MS_PREP_ROWS, nr = min(ROWS, o.M - m0), tid = threadIdx.x, nth = blockDim.x;
+  const int nd = (H * dk + 2 * nth - 1) / (2 * nth), ng = o.tap_off[2] > 0 ? (H * o.cin + 2 * nth - 1) / (2 * nth) : 0, y = blockIdx.y;
   const int cols = logs ? (H * dk + 3) & ~3 : mstate_cdelta_cols(H, G, dk);
   const float* raw = reinterpret_cast<const float*>(o.res) + (size_t)m0 * o.ldr;
   float* w = reinterpret_cast<float*>(o.ws) + (size_t)m0 * cols;
   if (y < nd + ng) {
     const bool decay = y < nd;
-    const int R = o.tap_off[decay ? 0 : 2], lcol = decay ? o.col_mod : o.tap_off[1], c = (decay ? y : y - nd) * 256 + tid;
-    for (int i = tid; i < ROWS * R; i += 256) {
+    const int R = o.tap_off[decay ? 0 : 2], lcol = decay ? o.col_mod : o.tap_off[1], c = ((decay ? y : y - nd) * nth + tid) * 2;
+    const int n = H * (decay ? dk : o.cin);
+    for (int i = tid; i < ROWS * R; i += nth) {
       const int j = i / R, r = i - j * R;
       cd_lat[r * 8 + j] = j < nr ? raw[(size_t)j * o.ldr + lcol + r] : 0.f;
     }
     __syncthreads();
-    float z[ROWS];
-    if (decay) {
-      if (c >= H * dk) return;
-      cdelta_up<ROWS>(o, cd_lat, o.B, c, R, z);
-      const float db = reinterpret_cast<const float*>(o.bias)[c], rate = expf(reinterpret_cast<const float*>(o.scale)[c / dk]);
+    if (c >= n) return;
+    float z[2][ROWS];
+    cdelta_up<ROWS>(o, cd_lat, decay ? o.B : o.p1, c, n, R, z);
 #pragma unroll
-      for (int j = 0; j < ROWS; ++j)
-        if (j < nr) {
-          const float l = -rate * softplus_f(z[j] + db);
-          if (logs) w[(size_t)j * cols + c] = 1.4426950408889634f * l;
-          else w[(size_t)j * cols + 2 * G * dk + c] = expf(l);
-        }
-    } else {
-      if (c >= H * o.cin) return;
-      cdelta_up<ROWS>(o, cd_lat, o.p1, c, R, z);
-      float* gr = reinterpret_cast<float*>(o.norm_out) + (size_t)m0 * o.norm_ld + c;
+    for (int e = 0; e < 2; ++e) {
+      const int ce = c + e;
+      if (ce >= n) break;
+      if (decay) {
+        const float db = reinterpret_cast<const float*>(o.bias)[ce], rate = expf(reinterpret_cast<const float*>(o.scale)[ce / dk]);
 #pragma unroll
-      for (int j = 0; j < ROWS; ++j)
-        if (j < nr) gr[(size_t)j * o.norm_ld] = z[j];
+        for (int j = 0; j < ROWS; ++j) z[e][j] = -rate * softplus_f(z[e][j] + db);
+#pragma unroll
+        for (int j = 0; j < ROWS; ++j) z[e][j] = logs ? 1.4426950408889634f * z[e][j] : expf(z[e][j]);
+      }
+    }
+    float* d = decay ? w + (logs ? 0 : 2 * G * dk) + c : reinterpret_cast<float*>(o.norm_out) + (size_t)m0 * o.norm_ld + c;
+    const int ld = decay ? cols : o.norm_ld;
+    const bool pairs = c + 1 < n && ld % 2 == 0 && !(reinterpret_cast<uintptr_t>(d) & 7);
+#pragma unroll
+    for (int j = 0; j < ROWS; ++j) {
+      if (j >= nr) break;
+      if (pairs) *reinterpret_cast<float2*>(d + (size_t)j * ld) = make_float2(z[0][j], z[1][j]);
+      else { d[(size_t)j * ld] = z[0][j]; if (c + 1 < n) d[(size_t)j * ld + 1] = z[1][j]; }
     }
     return;
   }
   float* cf = w + (2 * G + H) * dk;
-  for (int i = tid; i < nr * H; i += 256) {
+  for (int i = tid; i < nr * H; i += nth) {
     const int j = i / H, h = i - j * H;
     cf[(size_t)j * cols + h] = sigmoid_f(raw[(size_t)j * o.ldr + o.m_begin + h]);
   }
   const int warp = tid >> 5, lane = tid & 31;
   const float qs = 1.f / sqrtf((float)dk);
-  for (int i = warp; i < nr * G; i += 8) {          // a warp per (row, group): both unit vectors and their product
+  for (int i = warp; i < nr * G; i += nth >> 5) {          // a warp per (row, group): both unit vectors and their product
     const int j = i / G, g = i - j * G;
     const float* q = reinterpret_cast<const float*>(o.A) + (size_t)(m0 + j) * o.lda + (size_t)g * dk;
     const float* k = q + o.K;
@@ -2687,10 +2690,10 @@ __global__ void __launch_bounds__(256) fq3s_mstate_carry_kernel(const fq3c_op o,
 // ---------------------------------------------------------------------------------------------------------------------------
 constexpr int CD_C = 16;           // tokens per block
 constexpr int CD_TP = CD_C + 4;    // pitch of T and B
-constexpr int CD_PAIRS = CD_C * (CD_C + 1) / 2, CD_REC_THREADS = (CD_PAIRS + 31) / 32 * 32;
+constexpr int CD_TILES = CD_C / 2 * (CD_C / 2 + 1) / 2, CD_REC_THREADS = (CD_TILES * 4 + 31) / 32 * 32;      // 2 x 2 tiles of (t, s) pairs, four threads each
 constexpr int CD_MIN_ROWS = 32;    // fewer rows are walked token by token
 constexpr int CD_MAX_DK = 256;
-__host__ __device__ constexpr int cd_rows(int dk) { return (dk + 15) & ~15; }       // state rows, padded with zeros
+__host__ __device__ constexpr int cd_rows(int dk) { return (dk + 31) & ~31; }       // state rows, padded with zeros
 __host__ __device__ constexpr int cd_pitch(int dk) { return cd_rows(dk) + 4; }
 __host__ __device__ constexpr int cd_record(int dk) { return 3 * CD_C * cd_pitch(dk) + cd_rows(dk) + 2 * CD_C * CD_TP; }      // floats, a multiple of four
 __host__ __device__ inline long long cd_log_floats(int M, int H, int dk, bool channels) { return channels ? (long long)M * ((H * dk + 3) & ~3) : 0; }
@@ -2698,6 +2701,7 @@ __host__ __device__ inline long long cd_ws_floats(int M, int H, int dk, bool cha
   return cd_log_floats(M, H, dk, channels) + (long long)((M + CD_C - 1) / CD_C) * H * cd_record(dk);
 }
 constexpr float LOG2E_F = 1.4426950408889634f;
+__device__ __forceinline__ float pow2_f(const float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 // grid (blocks of tokens, H), CD_REC_THREADS threads; dynamic shared memory: sums (two floats), q and k, [CD_C][pitch] each
 __global__ void __launch_bounds__(CD_REC_THREADS) fq3s_cdelta_record_kernel(const fq3c_op o) {
   extern __shared__ __align__(16) float cr[];
@@ -2753,37 +2757,62 @@ __global__ void __launch_bounds__(CD_REC_THREADS) fq3s_cdelta_record_kernel(cons
     k.x *= fk[t]; k.y *= fk[t]; k.z *= fk[t]; k.w *= fk[t];
     *reinterpret_cast<float4*>(qs + at) = q;
     *reinterpret_cast<float4*>(ks + at) = k;
-    const float4 d = make_float4(exp2f(hi.x), exp2f(hi.y), exp2f(hi.z), exp2f(hi.w));
+    const float4 d = make_float4(pow2_f(hi.x), pow2_f(hi.y), pow2_f(hi.z), pow2_f(hi.w));
     *reinterpret_cast<float4*>(rec + at) = make_float4(k.x * d.x, k.y * d.y, k.z * d.z, k.w * d.w);
     *reinterpret_cast<float4*>(rec + CD_C * P + at) = make_float4(q.x * d.x, q.y * d.y, q.z * d.z, q.w * d.w);
     *reinterpret_cast<float4*>(rec + 2 * CD_C * P + at) =
-        make_float4(k.x * exp2f((eh.x - hi.x) + (el.x - lo.x)), k.y * exp2f((eh.y - hi.y) + (el.y - lo.y)),
-                    k.z * exp2f((eh.z - hi.z) + (el.z - lo.z)), k.w * exp2f((eh.w - hi.w) + (el.w - lo.w)));
+        make_float4(k.x * pow2_f((eh.x - hi.x) + (el.x - lo.x)), k.y * pow2_f((eh.y - hi.y) + (el.y - lo.y)),
+                    k.z * pow2_f((eh.z - hi.z) + (el.z - lo.z)), k.w * pow2_f((eh.w - hi.w) + (el.w - lo.w)));
     if (t == CD_C - 1) *reinterpret_cast<float4*>(rec + 3 * CD_C * P + c) = d;
   }
   __syncthreads();
   float* Tm = rec + 3 * CD_C * P + D;
   float* Bm = Tm + CD_C * CD_TP;
-  if (tid < CD_PAIRS) {
-    int t = (int)((sqrtf(8.f * (float)tid + 1.f) - 1.f) * 0.5f);
-    while ((t + 1) * (t + 2) / 2 <= tid) ++t;
-    while (t * (t + 1) / 2 > tid) --t;
-    const int s = tid - t * (t + 1) / 2;
-    float a = 0.f, b = 0.f;
-#pragma unroll 2
-    for (int c = 0; c < D; c += 4) {
-      const float4 ht = ld4(bh + t * P + c), lt = ld4(bl + t * P + c), hs = ld4(bh + s * P + c), ls = ld4(bl + s * P + c);
-      const float4 kt = ld4(ks + t * P + c), k = ld4(ks + s * P + c), q = ld4(qs + t * P + c);
-      const float e0 = k.x * exp2f((ht.x - hs.x) + (lt.x - ls.x)), e1 = k.y * exp2f((ht.y - hs.y) + (lt.y - ls.y));
-      const float e2 = k.z * exp2f((ht.z - hs.z) + (lt.z - ls.z)), e3 = k.w * exp2f((ht.w - hs.w) + (lt.w - ls.w));
-      a = fmaf(kt.x, e0, a); b = fmaf(q.x, e0, b);
-      a = fmaf(kt.y, e1, a); b = fmaf(q.y, e1, b);
-      a = fmaf(kt.z, e2, a); b = fmaf(q.z, e2, b);
-      a = fmaf(kt.w, e3, a); b = fmaf(q.w, e3, b);
+  if (tid < CD_TILES * 4) {       // 2 x 2 pairs (t, s): rows 2 ti and next, columns 2 si and next; a quarter of the channels per thread
+    const int tile = tid >> 2;
+    int ti = (int)((sqrtf(8.f * (float)tile + 1.f) - 1.f) * 0.5f);
+    while ((ti + 1) * (ti + 2) / 2 <= tile) ++ti;
+    while (ti * (ti + 1) / 2 > tile) --ti;
+    const int si = tile - ti * (ti + 1) / 2;
+    const unsigned lanes = (warp + 1) * 32 <= CD_TILES * 4 ? 0xffffffffu : (1u << (CD_TILES * 4 % 32)) - 1u;      // the last warp has fewer
+    float a[2][2] = {{0.f, 0.f}, {0.f, 0.f}}, b[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+    for (int c = (tid & 3) * 4; c < D; c += 16) {
+      float4 ht[2], lt[2], kt[2], qt[2];
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int at = (2 * ti + x) * P + c;
+        ht[x] = ld4(bh + at); lt[x] = ld4(bl + at); kt[x] = ld4(ks + at); qt[x] = ld4(qs + at);
+      }
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const int at = (2 * si + y) * P + c;
+        const float4 hs = ld4(bh + at), ls = ld4(bl + at), k = ld4(ks + at);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {      // (above the diagonal the exponent is positive and may overflow: not stored)
+          const float e0 = k.x * pow2_f((ht[x].x - hs.x) + (lt[x].x - ls.x)), e1 = k.y * pow2_f((ht[x].y - hs.y) + (lt[x].y - ls.y));
+          const float e2 = k.z * pow2_f((ht[x].z - hs.z) + (lt[x].z - ls.z)), e3 = k.w * pow2_f((ht[x].w - hs.w) + (lt[x].w - ls.w));
+          a[x][y] = fmaf(kt[x].x, e0, a[x][y]); b[x][y] = fmaf(qt[x].x, e0, b[x][y]);
+          a[x][y] = fmaf(kt[x].y, e1, a[x][y]); b[x][y] = fmaf(qt[x].y, e1, b[x][y]);
+          a[x][y] = fmaf(kt[x].z, e2, a[x][y]); b[x][y] = fmaf(qt[x].z, e2, b[x][y]);
+          a[x][y] = fmaf(kt[x].w, e3, a[x][y]); b[x][y] = fmaf(qt[x].w, e3, b[x][y]);
+        }
+      }
     }
-    N[t][s] = beta[t] * a;
-    Bm[t * CD_TP + s] = b;
-    if (s < t) { Bm[s * CD_TP + t] = 0.f; Tm[s * CD_TP + t] = 0.f; }
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        a[x][y] += __shfl_xor_sync(lanes, a[x][y], 1); b[x][y] += __shfl_xor_sync(lanes, b[x][y], 1);
+        a[x][y] += __shfl_xor_sync(lanes, a[x][y], 2); b[x][y] += __shfl_xor_sync(lanes, b[x][y], 2);
+        const int t = 2 * ti + x, s = 2 * si + y;
+        if ((tid & 3) == 2 * x + y) {        // one of the tile's four threads keeps it
+          if (s <= t) {
+            N[t][s] = beta[t] * a[x][y];
+            Bm[t * CD_TP + s] = b[x][y];
+          }
+          if (s != t) Tm[(s < t ? s : t) * CD_TP + (s < t ? t : s)] = 0.f, Bm[(s < t ? s : t) * CD_TP + (s < t ? t : s)] = 0.f;
+        }
+      }
   }
   __syncthreads();
   if (tid < CD_C) {       // column tid of T by forward substitution
@@ -2799,32 +2828,60 @@ __global__ void __launch_bounds__(CD_REC_THREADS) fq3s_cdelta_record_kernel(cons
   }
 }
 
-// grid (ceil(dv / DVT), H), 128 threads.  The state tile [D rows, DVT columns] lives in registers (four rows x two columns x RQ per thread) and, as
-// the operand of the next block's products, transposed in shared memory.  [Kt; Qt] S0: a warp takes a quarter of the state rows for all 2 CD_C x DVT
-// sums (a lane: rows r, r + 8, r + 16, r + 24 and every fourth column), the quarters are added where the sums are used.  U and O: a lane per
-// (token, column).  Records arrive by cp.async, one block of tokens ahead.
+// set by a kernel whose bounded wait for its own copy ran out; its outputs are then NaN
+__device__ int seq_wait_error;
+// true when the barrier's phase completed, false when the limit ran out (about a second)
+__device__ __forceinline__ bool mbar_wait_bounded(const uint32_t bar, const uint32_t parity) {
+  for (int i = 0; i < (1 << 20); ++i) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if (i > 64) __nanosleep(256);
+  }
+  return false;
+}
+// grid (ceil(dv / DVT), H), 160 threads: four warps compute, the fifth asks for the records, one bulk copy per block of tokens, one block ahead.
+// The state tile [D rows, DVT columns] lives in registers (four rows x two columns x RQ per thread) and, as the operand of the next block's
+// products, transposed in shared memory.  [Kt; Qt] S0: a warp takes a quarter of the state rows for all 2 CD_C x DVT sums (a lane: rows r, r + 8,
+// r + 16, r + 24 and four columns; with eight columns the half-warps split the quarter once more and exchange halves of their sums), the quarters
+// are added where the sums are used.  U and O: a lane per (token, column).
+constexpr int CD_WALK_THREADS = 160;
 template <int DVT>
 __host__ __device__ constexpr int cd_walk_floats(int dk) {
-  return 2 * cd_record(dk) + DVT * cd_pitch(dk) + 4 * 2 * CD_C * (DVT + 1) + DVT * CD_TP + 2 * CD_C * DVT + 4;
+  return 2 * cd_record(dk) + DVT * cd_pitch(dk) + 4 * 2 * CD_C * (DVT + 1) + DVT * CD_TP + 4;
 }
 template <int DVT, int RQ>
-__global__ void __launch_bounds__(128) fq3s_cdelta_walk_kernel(const fq3c_op o) {
-  extern __shared__ __align__(16) float cw[];
-  constexpr int NCP = DVT / 2, QS = 128 / NCP, NC = DVT / 4, PP = DVT + 1, JW = DVT / 4;
+__global__ void __launch_bounds__(CD_WALK_THREADS) fq3s_cdelta_walk_kernel(const fq3c_op o) {
+  extern __shared__ __align__(128) float cw[];
+  __shared__ __align__(8) unsigned long long full[2];
+  constexpr int NCP = DVT / 2, QS = 128 / NCP, CG = DVT / 4, KH = 4 / CG, PP = DVT + 1, JW = DVT / 4;
   const int H = o.i0, dk = o.i2, dv = o.cin, h = blockIdx.y, j0 = blockIdx.x * DVT, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int D = cd_rows(dk), P = cd_pitch(dk), REC = cd_record(dk), nblk = (o.M + CD_C - 1) / CD_C;
   float* St = cw + 2 * REC;                          // [DVT][P]
-  float* Ud = St + DVT * P;                          // [CD_C][DVT] pairs (u, u)
-  float* Xs = Ud + 2 * CD_C * DVT;                   // [DVT][CD_TP]
+  float* Xs = St + DVT * P;                          // [DVT][CD_TP]: V - Kt S0, then U
   float* Pp = Xs + DVT * CD_TP;                      // [4][2 CD_C][PP]
   const float* recs = reinterpret_cast<const float*>(o.ws) + cd_log_floats(o.M, H, dk, o.taps == 6) + (size_t)h * REC;
-  auto fetch = [&](const int n) {
-    const float* src = recs + (size_t)n * H * REC;
-    float* dst = cw + (n & 1) * REC;
-    for (int i = tid * 4; i < REC; i += 512) cp_async16(dst + i, src + i, true);
-    cp_async_commit();
+  auto fetch = [&](const int n) {       // one thread
+    const uint32_t bar = smem_u32(&full[n & 1]);
+    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"((uint32_t)REC * 4u) : "memory");
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(cw + (n & 1) * REC)),
+                 "l"(recs + (size_t)n * H * REC), "r"((uint32_t)REC * 4u), "r"(bar)
+                 : "memory");
   };
-  fetch(0);
+  if (tid == 128) {
+    mbar_init(smem_u32(&full[0]), 1);
+    mbar_init(smem_u32(&full[1]), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    fetch(0);
+  }
+  __syncthreads();             // the barriers are initialised
+  if (warp == 4) {
+    for (int n = 0; n < nblk; ++n) {
+      if (__syncthreads_or(0)) return;       // the four warps gave up
+      if (lane == 0 && n + 1 < nblk) fetch(n + 1);
+      __syncthreads();
+      __syncthreads();
+    }
+    return;
+  }
   // this thread's part of the state: rows rq + q QS (quads), columns 2 cp, 2 cp + 1
   const int cp = tid % NCP, rq = tid / NCP;
   f32x2 S[RQ][2][2];          // [quad][column][row pair]
@@ -2853,40 +2910,52 @@ __global__ void __launch_bounds__(128) fq3s_cdelta_walk_kernel(const fq3c_op o) 
     }
   };
   load_v(0);
-  const int rl = lane & 7, cl = lane >> 3, KW = D >> 2;      // products: rows rl + 8 i of [Kt; Qt], columns cl + 4 i
+  const int rl = lane & 7, cl = (lane >> 3) % CG, kh = (lane >> 3) / CG, KW = (D >> 2) / KH;      // products: rows rl + 8 i of [Kt; Qt], columns cl + CG i
   for (int n = 0; n < nblk; ++n) {
-    cp_async_wait<0>();
-    __syncthreads();           // the record is there, the transposed state too; everyone is done with the other buffer
-    if (n + 1 < nblk) fetch(n + 1);
+    const bool there = mbar_wait_bounded(smem_u32(&full[n & 1]), (uint32_t)((n >> 1) & 1));
+    // the record is there, the transposed state too; everyone is done with the other buffer
+    if (__syncthreads_or(!there)) {
+      if (tid == 0) { seq_wait_error = 1; mbar_wait_bounded(smem_u32(&full[n & 1]), (uint32_t)((n >> 1) & 1)); }
+      for (int i = tid; i < o.M * DVT; i += 128)
+        if (j0 + i % DVT < dv) reinterpret_cast<float*>(o.C)[(size_t)(i / DVT) * o.ldc + (size_t)h * dv + j0 + i % DVT] = __int_as_float(0x7fc00000);
+      return;
+    }
     const float* rec = cw + (n & 1) * REC;
     {
-      f32x2 acc[4][NC];
+      f32x2 acc[4][4];
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < NC; ++j) acc[i][j] = 0ull;
-      const float* kr = rec + rl * P + warp * KW;
-      const float* sr = St + cl * P + warp * KW;
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0ull;
+      const float* kr = rec + rl * P + (warp * KH + kh) * KW;
+      const float* sr = St + cl * P + (warp * KH + kh) * KW;
 #pragma unroll 2
       for (int k = 0; k < KW; k += 4) {
-        ulonglong2 a[4], b[NC];
+        ulonglong2 a[4], b[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const ulonglong2*>(kr + 8 * i * P + k);
 #pragma unroll
-        for (int j = 0; j < NC; ++j) b[j] = *reinterpret_cast<const ulonglong2*>(sr + 4 * j * P + k);
+        for (int j = 0; j < 4; ++j) b[j] = *reinterpret_cast<const ulonglong2*>(sr + CG * j * P + k);
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-          for (int j = 0; j < NC; ++j) {
+          for (int j = 0; j < 4; ++j) {
             acc[i][j] = fma2<true>(a[i].x, b[j].x, acc[i][j]);
             acc[i][j] = fma2<true>(a[i].y, b[j].y, acc[i][j]);
           }
       }
       float* pw = Pp + warp * 2 * CD_C * PP;
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+      for (int i = 0; i < 4; i += KH)
 #pragma unroll
-        for (int j = 0; j < NC; ++j) pw[(rl + 8 * i) * PP + cl + 4 * j] = lo2(acc[i][j]) + hi2(acc[i][j]);
+        for (int j = 0; j < 4; ++j) {
+          float v = lo2(acc[i][j]) + hi2(acc[i][j]);
+          if (KH == 2) {       // a half-warp keeps every other row of its four
+            const float w = lo2(acc[i + KH - 1][j]) + hi2(acc[i + KH - 1][j]);
+            v = (kh ? w : v) + __shfl_xor_sync(0xffffffffu, kh ? v : w, 16);
+          }
+          pw[(rl + 8 * (i + (KH == 2 ? kh : 0))) * PP + cl + CG * j] = v;
+        }
     }
     __syncthreads();
     const float* Tm = rec + 3 * CD_C * P + D;
@@ -2914,15 +2983,13 @@ __global__ void __launch_bounds__(128) fq3s_cdelta_walk_kernel(const fq3c_op o) 
     for (int e = 0; e < JW / 2; ++e) u[e] = row_times(Tm, jb + 2 * e);
     __syncwarp();
 #pragma unroll
-    for (int e = 0; e < JW / 2; ++e) {
-      Xs[(jb + 2 * e) * CD_TP + t] = u[e];
-      *reinterpret_cast<float2*>(Ud + 2 * (t * DVT + jb + 2 * e)) = make_float2(u[e], u[e]);
-    }
+    for (int e = 0; e < JW / 2; ++e) Xs[(jb + 2 * e) * CD_TP + t] = u[e];
     if (n + 1 < nblk) load_v(n + 1);
     __syncthreads();
     {   // S <- diag(G_last) S + Kb^T U
       const float* Kb = rec + 2 * CD_C * P;
       const float* Gl = rec + 3 * CD_C * P;
+      const float* u0 = Xs + 2 * cp * CD_TP;
 #pragma unroll
       for (int q = 0; q < RQ; ++q) {
         const int r = (rq + q * QS) * 4;
@@ -2931,13 +2998,20 @@ __global__ void __launch_bounds__(128) fq3s_cdelta_walk_kernel(const fq3c_op o) 
 #pragma unroll
         for (int j = 0; j < 2; ++j) { S[q][j][0] = mul2<true>(gl.x, S[q][j][0]); S[q][j][1] = mul2<true>(gl.y, S[q][j][1]); }
 #pragma unroll
-        for (int s = 0; s < CD_C; ++s) {
-          const ulonglong2 kb = *reinterpret_cast<const ulonglong2*>(Kb + s * P + r);
-          const ulonglong2 uu = *reinterpret_cast<const ulonglong2*>(Ud + 2 * (s * DVT + 2 * cp));
-          S[q][0][0] = fma2<true>(kb.x, uu.x, S[q][0][0]);
-          S[q][0][1] = fma2<true>(kb.y, uu.x, S[q][0][1]);
-          S[q][1][0] = fma2<true>(kb.x, uu.y, S[q][1][0]);
-          S[q][1][1] = fma2<true>(kb.y, uu.y, S[q][1][1]);
+        for (int s = 0; s < CD_C; s += 4) {
+          ulonglong2 kb[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) kb[e] = *reinterpret_cast<const ulonglong2*>(Kb + (s + e) * P + r);
+          const float4 ua = ld4(u0 + s), ub = ld4(u0 + CD_TP + s);
+          const float uv[2][4] = {{ua.x, ua.y, ua.z, ua.w}, {ub.x, ub.y, ub.z, ub.w}};
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+              const f32x2 uu = pack2(uv[j][e], uv[j][e]);
+              S[q][j][0] = fma2<true>(kb[e].x, uu, S[q][j][0]);
+              S[q][j][1] = fma2<true>(kb[e].y, uu, S[q][j][1]);
+            }
         }
 #pragma unroll
         for (int j = 0; j < 2; ++j)

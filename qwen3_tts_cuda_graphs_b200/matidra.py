@@ -126,7 +126,7 @@ class Packer:
         a1, a2, g1, g2 = (self.raw(p + n) for n in ("a1", "a2", "g1", "g2"))
         if a1.shape[0] != a2.shape[1] or g1.shape[0] != g2.shape[1]:
             raise ValueError(f"{p}: the two factors of a low-rank projection disagree on their inner size")
-        return {"a2": self.W(a2), "g2": self.W(g2), "dt_bias": self.F(self.raw(p + "dt_bias")), "A_log": self.F(self.raw(p + "A_log")),
+        return {"a2": self.W(a2.T), "g2": self.W(g2.T), "dt_bias": self.F(self.raw(p + "dt_bias")), "A_log": self.F(self.raw(p + "A_log")),
                 "norm": self.F(self.raw(p + "norm").to(torch.float64) * scale)}
 
     def channel_delta(self, p: str) -> dict:

@@ -218,6 +218,8 @@ def time_ops(lib, arr, n_ops, ctx_of, skip_last=False, reps=5, top=None):
     single = []
     n = n_ops - (1 if skip_last else 0)
     for i in range(n):
+        if arr[i].kind == K.K_BRANCH:
+            continue
         one = (K.Op * 1)(arr[i])
         ts = []
         for r in range(reps + 1):

@@ -157,9 +157,15 @@ class SequenceEngine:
                     break
                 if i + 1 < max_new_tokens:
                     logits = self.step(request, [t], [0])
+            self.check_waits()
             return out
         finally:
             self.close(request)
+
+    def check_waits(self) -> None:
+        """Raises when a kernel gave up a bounded wait (its outputs are NaN then).  Synchronises the device."""
+        if self.lib.fq3c_wait_errors() != 0:
+            raise RuntimeError("a kernel's wait for its own copy ran out: the outputs since then are not valid")
 
     def close_all(self):
         for e in list(self._steps.values()) + list(self._heads.values()):

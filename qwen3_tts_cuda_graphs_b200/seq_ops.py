@@ -31,7 +31,7 @@ import torch
 
 from .codec import (F_A_F32, F_BIAS, F_CENTER, F_SWIGLU, F_F32, F_GATE_ENTRY, F_GATE_POST, F_GATE_PRE, F_GELU, F_GELU_TANH, F_NOROUND, F_OUT_F32, F_POST, F_RAW_WEIGHTS, F_RELU2, F_RESID,
                     F_ROT_HALF, F_SIGMOID, F_SILU, F_UNIT,
-                    K_BDGEMM, K_CACHE_ATTN, K_COMMIT, K_DEPTH_MIX, K_DYT, K_EMBED, K_GEMM, K_GGEMM, K_GLU, K_GNORM, K_HYPER, K_LATENT_ATTN,
+                    K_BDGEMM, K_BRANCH, K_CACHE_ATTN, K_COMMIT, K_DEPTH_MIX, K_DYT, K_EMBED, K_GEMM, K_GGEMM, K_GLU, K_GNORM, K_HYPER, K_LATENT_ATTN,
                     K_LRU_SCAN, K_MOE_COMBINE, K_MOE_SORT, K_MSTATE_SCAN, K_POLYNORM, K_ROT_APPEND, K_ROUTER, K_SUM_NORM, K_TCONV, K_XIELU, Op, _Plan)
 from .config import (ChannelDecayAttentionConfig, ChannelDeltaRuleConfig, DeltaRuleConfig, ForgetGateAttentionConfig, LatentAttentionConfig, MatrixMemoryConfig,
                      MoEFFConfig, RetentionConfig, RglruConfig, SoftmaxAttentionConfig, StateSpaceConfig)
@@ -413,8 +413,8 @@ class StepBuilder:
     def _delta_ws(self, coef_cols: int, H: int, dk: int, log_cols: int) -> torch.Tensor:
         """Workspace of a delta rule: the rows of the walk token by token, or, for many rows, room for the records of the walk in blocks of
         16 tokens (cd_record of csrc/fq3_seq.cuh: three operands of 16 rows, the last decays, two 16 x 16 matrices) behind the decay rows."""
-        d16 = -(-dk // 16) * 16
-        blocks = -(-self.M // 16) * H * (48 * (d16 + 4) + d16 + 640) + self.M * log_cols if self.M >= 32 else 0
+        D = -(-dk // 32) * 32
+        blocks = -(-self.M // 16) * H * (48 * (D + 4) + D + 640) + self.M * log_cols if self.M >= 32 else 0
         return self.buf("ms.ws", 1, max(self.M * coef_cols, blocks, 4))
 
     def _mstate(self, mode: int, rows: torch.Tensor, raw: torch.Tensor, H: int, G: int, dk: int, dv: int, kcol: int, vcol: int,
@@ -473,8 +473,8 @@ class StepBuilder:
 
     def channel_delta_rule(self, h: torch.Tensor, c: ChannelDeltaRuleConfig, w: dict, state: str, eps: float, out: torch.Tensor):
         """h [M, width] -> out f32 [M, width].  w: win [2 G dim + H vdim + H + decay rank + gate rank (+ padding), width] (q | k | v |
-        write-strength input | decay latent | gate latent), conv f32 [2 G dim + H vdim, taps], a2 [H dim, decay rank], dt_bias f32 [H dim],
-        A_log f32 [H], g2 [H vdim, gate rank], norm f32 [vdim], o [width, H vdim].  Per head S <- diag(g) S, g = exp(-exp(A_log) softplus(z));
+        write-strength input | decay latent | gate latent), conv f32 [2 G dim + H vdim, taps], a2 [decay rank, H dim] (transposed), dt_bias f32
+        [H dim], A_log f32 [H], g2 [gate rank, H vdim] (transposed), norm f32 [vdim], o [width, H vdim].  Per head S <- diag(g) S, g = exp(-exp(A_log) softplus(z));
         u = beta (v - S^T k); S <- S + k u^T; o = S^T q, on unit queries (times dim^(-1/2)) and keys.  States: state + ".conv", state + ".s"."""
         M, n = self.M, 2 * c.kv_heads * c.dim + c.heads * c.vdim
         raw = self.linear(h, w["win"], self.buf("kd.raw", M, w["win"].shape[0]))
@@ -488,7 +488,7 @@ class StepBuilder:
         """channel_delta_rule between the convolution and the output product: q | k | v in cv's columns from ccol on, write-strength inputs |
         decay latent | gate latent in raw's from rcol on; the gated read-out goes to yn's columns from ycol on."""
         M, H, G, d, dv = self.M, c.heads, c.kv_heads, c.dim, c.vdim
-        ra, rg = w["a2"].shape[1], w["g2"].shape[1]
+        ra, rg = w["a2"].shape[0], w["g2"].shape[0]
         y, gate = self.buf("kd.y", M, H * dv), self.buf("kd.gate", M, H * dv)
         ws = self._delta_ws(-(-((2 * G + H) * d + H + G) // 4) * 4, H, d, -(-(H * d) // 4) * 4)
         self.plan.keep += [cv, raw]
@@ -511,8 +511,11 @@ class StepBuilder:
         raw = self.linear(h, w["win"], self.buf("pd.raw", M, w["win"].shape[0]))
         cv = self.time_conv(raw, w["conv"], state + ".conv", self.buf("pd.cv", M, n), channels=n, silu=True, silu_from=nl)
         heads = self.buf("pd.heads", M, H * dv + right.heads * right.vdim, self.adt)
+        self.branch(0)         # the two mixers run side by side
         self._attend(left, w["left"], cv, 0, H * d, (H + G) * d, (raw, n), kcache, vcache, eps, heads, mult=left_scale)
+        self.branch(1)
         self._channel_delta(right, w["right"], cv, nl, raw, n + H * dv, state + ".s", eps, heads, H * dv)
+        self.branch(2)
         return self.linear(heads, w["o"], out)
 
     def retention(self, h: torch.Tensor, c: RetentionConfig, w: dict, state: str, eps: float, out: torch.Tensor):
@@ -669,6 +672,11 @@ class StepBuilder:
             kw["p1"] = weight
         self._op(K_GLU, **kw)
         return out
+
+    def branch(self, what: int):
+        """0: the following ops go to a side stream; 1: to the main stream again, beside it; 2: the main stream waits for the side stream.
+        The two parts must not share scratch buffers."""
+        self._op(K_BRANCH, M=1, i0=what)
 
     def commit(self):
         """Close the step: install every carry's next value and advance the slot's position counter by M."""

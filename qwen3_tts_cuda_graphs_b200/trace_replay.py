@@ -58,6 +58,7 @@ def main(argv=None) -> int:
             torch.cuda.synchronize()
         out.write("done %d\n" % st["step"])
         out.flush()
+    eng.check_waits()
     eng.close_all()
     return 0
 

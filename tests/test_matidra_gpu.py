@@ -482,6 +482,43 @@ def test_both_mixers_on_one_projection(taps, f32):
         assert close_enough(got, want, f32), (sizes, float(row_errors(got, want).max()))
 
 
+def test_two_parts_of_a_list_side_by_side():
+    """A side stream sees what was launched before it, the main stream sees its results behind the join; a list may end with the side
+    stream open; the same list captured as a graph gives the same."""
+    from qwen3_tts_cuda_graphs_b200.seq_ops import StepBuilder
+
+    torch.manual_seed(1)
+    M, N = 700, 256
+    bench = Bench([], True)
+    x, one = cuda(torch.randn(1, M, N)), cuda(torch.ones(2))
+    for ending in (True, False):
+        b = StepBuilder(torch.device(DEV), M, bench.slot, True)
+        a, parts, out = torch.zeros(M, N, device=DEV), torch.zeros(2, M, N, device=DEV), torch.zeros(M, N, device=DEV)
+        b.sum_norm(x, 1, cuda(torch.tensor([2.0])), out=a)                     # before both: a = 2 x
+        b.branch(0)
+        for _ in range(6):
+            b.sum_norm(a[None], 1, cuda(torch.tensor([3.0])), out=parts[0])     # side: 6 x
+        b.branch(1)
+        b.sum_norm(a[None], 1, cuda(torch.tensor([5.0])), out=parts[1])         # main: 10 x
+        if ending:
+            b.branch(2)
+            b.sum_norm(parts, 2, one, out=out)
+        plan = b.finish()
+        for _ in range(4):          # launched, then captured and replayed
+            parts.zero_()
+            out.zero_()
+            bench.codec.run_op_plan(bench.lib, plan, True)
+            total = out if ending else parts[0] + parts[1]
+            assert torch.allclose(total, 16.0 * x[0], rtol=1e-5)
+        assert getattr(plan, "graph", None) is not None
+        bench.lib.fq3c_graph_destroy(plan.graph)
+    b = StepBuilder(torch.device(DEV), M, bench.slot, True)       # a second side stream inside the first is refused
+    b.branch(0)
+    b.branch(0)
+    with pytest.raises(Exception, match="one side stream"):
+        bench.codec.run_op_plan(bench.lib, b.finish(), False)
+
+
 # ---------------------------------------------------------------------------------------------------------------------------
 # whole models
 # ---------------------------------------------------------------------------------------------------------------------------
