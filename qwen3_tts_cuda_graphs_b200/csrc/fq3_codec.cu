@@ -1443,11 +1443,11 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         fq3s_mstate_max_kernel<<<o.i0, MM_THREADS, 0, s>>>(o);
         count_launches(1);
       } else if (o.taps == 6) {
-        const int nth = o.M <= 8 ? 64 : 256, per = 2 * nth;      // few rows: more, smaller blocks
+        const int per = cdelta_prep_channels(o.M == 1 ? 1 : MS_PREP_ROWS);
         const dim3 grid((o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS, (o.i0 * o.i2 + per - 1) / per + (o.tap_off[2] > 0 ? (o.i0 * o.cin + per - 1) / per : 0) + (blocks ? 0 : 1));
         const size_t smem = sizeof(float) * MS_PREP_ROWS * (size_t)std::max(o.tap_off[0], o.tap_off[2]);
-        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, nth, smem, s>>>(o, false);
-        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, nth, smem, s>>>(o, blocks);
+        if (o.M == 1) fq3s_mstate_cdelta_prep_kernel<1><<<grid, 256, smem, s>>>(o, false);
+        else fq3s_mstate_cdelta_prep_kernel<MS_PREP_ROWS><<<grid, 256, smem, s>>>(o, blocks);
         count_launches(1);
       } else if (o.taps < 3 && !blocks) {
         fq3s_mstate_prep_kernel<<<o.taps == 2 ? (o.M + MS_PREP_ROWS - 1) / MS_PREP_ROWS : o.M, 128, 0, s>>>(o);

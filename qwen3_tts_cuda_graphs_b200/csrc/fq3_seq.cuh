@@ -1739,7 +1739,7 @@ __global__ void __launch_bounds__(128) fq3s_cache_attn_merge_kernel(const fq3c_o
   const float sc = gate * (o.f2 != 0.f ? o.f2 : 1.f) / den;
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
     float acc = 0.f;
-#pragma unroll 8
+#pragma unroll 16
     for (int s = 0; s < splits; ++s) acc = fmaf(wsm[s], src[(size_t)s * (dv + 2) + 2 + c], acc);
     float v = acc * sc;
     if (entry) v *= sigmoid_f(gr[(size_t)h * dv + c]);
@@ -2116,7 +2116,7 @@ __global__ void __launch_bounds__(128) fq3s_mstate_prep_kernel(const fq3c_op o) 
 // (sixteen-byte broadcasts).  Dynamic shared memory: 8 x the larger inner size.
 __host__ __device__ inline int mstate_cdelta_cols(int H, int G, int dk) { return ((2 * G + H) * dk + H + G + 3) & ~3; }
 template <int ROWS>
-__device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, const void* U, const int c, const int n, const int R, float (&z)[2][ROWS]) {
+__device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, const void* U, const int c, const int n, const int r0, const int R, float (&z)[2][ROWS]) {
 #pragma unroll
   for (int j = 0; j < ROWS; ++j) { z[0][j] = 0.f; z[1][j] = 0.f; }
   const bool two = c + 1 < n;
@@ -2132,41 +2132,56 @@ __device__ __forceinline__ void cdelta_up(const fq3c_op& o, const float* lat, co
   if (o.flags & FQ3C_F32) {
     const float* u = reinterpret_cast<const float*>(U) + c;
 #pragma unroll 8
-    for (int r = 0; r < R; ++r) add(u[(size_t)r * n], two ? u[(size_t)r * n + 1] : 0.f, r);
+    for (int r = r0; r < R; ++r) add(u[(size_t)r * n], two ? u[(size_t)r * n + 1] : 0.f, r);
     return;
   }
   const bf16* u = reinterpret_cast<const bf16*>(U) + c;
   if (n % 2 == 0 && !(reinterpret_cast<uintptr_t>(U) & 3)) {
 #pragma unroll 16
-    for (int r = 0; r < R; ++r) {
+    for (int r = r0; r < R; ++r) {
       const uint32_t w = __ldg(reinterpret_cast<const uint32_t*>(u + (size_t)r * n));
       add(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u), r);
     }
   } else {
-    for (int r = 0; r < R; ++r) add(__bfloat162float(u[(size_t)r * n]), two ? __bfloat162float(u[(size_t)r * n + 1]) : 0.f, r);
+    for (int r = r0; r < R; ++r) add(__bfloat162float(u[(size_t)r * n]), two ? __bfloat162float(u[(size_t)r * n + 1]) : 0.f, r);
   }
 }
 // With `logs` the rows hold the base-2 logarithms of the decays alone (pitch round_up(H * dk, 4)), for the walk in blocks of tokens.
+// channels per block: two per thread; with one row four threads share a pair
+__host__ __device__ constexpr int cdelta_prep_channels(int rows) { return rows == 1 ? 128 : 512; }
 template <int ROWS>
 __global__ void __launch_bounds__(256) fq3s_mstate_cdelta_prep_kernel(const fq3c_op o, const bool logs) {
   extern __shared__ __align__(16) float cd_lat[];       // [inner size][8]
-  const int H = o.i0, G = o.i1, dk = o.i2, m0 = blockIdx.x * MS_PREP_ROWS, nr = min(ROWS, o.M - m0), tid = threadIdx.x, nth = blockDim.x;
-  const int nd = (H * dk + 2 * nth - 1) / (2 * nth), ng = o.tap_off[2] > 0 ? (H * o.cin + 2 * nth - 1) / (2 * nth) : 0, y = blockIdx.y;
+  const int H = o.i0, G = o.i1, dk = o.i2, m0 = blockIdx.x * MS_PREP_ROWS, nr = min(ROWS, o.M - m0), tid = threadIdx.x;
+  constexpr int nth = 256, per = cdelta_prep_channels(ROWS);
+  const int nd = (H * dk + per - 1) / per, ng = o.tap_off[2] > 0 ? (H * o.cin + per - 1) / per : 0, y = blockIdx.y;
   const int cols = logs ? (H * dk + 3) & ~3 : mstate_cdelta_cols(H, G, dk);
   const float* raw = reinterpret_cast<const float*>(o.res) + (size_t)m0 * o.ldr;
   float* w = reinterpret_cast<float*>(o.ws) + (size_t)m0 * cols;
   if (y < nd + ng) {
     const bool decay = y < nd;
-    const int R = o.tap_off[decay ? 0 : 2], lcol = decay ? o.col_mod : o.tap_off[1], c = ((decay ? y : y - nd) * nth + tid) * 2;
+    const int R = o.tap_off[decay ? 0 : 2], lcol = decay ? o.col_mod : o.tap_off[1], c = (decay ? y : y - nd) * per + (tid % (per / 2)) * 2;
     const int n = H * (decay ? dk : o.cin);
     for (int i = tid; i < ROWS * R; i += nth) {
       const int j = i / R, r = i - j * R;
       cd_lat[r * 8 + j] = j < nr ? raw[(size_t)j * o.ldr + lcol + r] : 0.f;
     }
     __syncthreads();
-    if (c >= n) return;
     float z[2][ROWS];
-    cdelta_up<ROWS>(o, cd_lat, decay ? o.B : o.p1, c, n, R, z);
+    if (ROWS == 1) {         // one row: quarters of the inner size side by side, added through shared memory
+      const int q = tid / (per / 2), len = (R + 3) / 4;
+      if (c < n) cdelta_up<ROWS>(o, cd_lat, decay ? o.B : o.p1, c, n, min(R, q * len), min(R, (q + 1) * len), z);
+      else z[0][0] = z[1][0] = 0.f;
+      __shared__ float2 part[256];
+      part[tid] = make_float2(z[0][0], z[1][0]);
+      __syncthreads();
+      if (q > 0 || c >= n) return;
+#pragma unroll
+      for (int e = 1; e < 4; ++e) { const float2 p = part[e * (per / 2) + tid]; z[0][0] += p.x; z[1][0] += p.y; }
+    } else {
+      if (c >= n) return;
+      cdelta_up<ROWS>(o, cd_lat, decay ? o.B : o.p1, c, n, 0, R, z);
+    }
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int ce = c + e;
