@@ -1306,10 +1306,12 @@ int seq_run(const fq3c_op& o, cudaStream_t s) {
         return fail("rot_append: bad configuration");
       if (o.m_begin > 0 && (o.i1 < 1 || o.cin < 1 || !o.norm_out || !o.ws || !o.p0)) return fail("rot_append: pooled blocks need both caches, their pooled rows and a position");
       const int rth = o.M <= 8 ? std::max(256, std::min(1024, 32 * (o.i0 + o.i1))) : 256;      // few rows: a warp per head
-      if (o.m_begin > 0 && o.M == 1 && (o.flags & FQ3C_F32)) fq3s_rot_append_kernel<float, true><<<1, rth, 0, s>>>(o);
-      else if (o.m_begin > 0 && o.M == 1) fq3s_rot_append_kernel<bf16, true><<<1, rth, 0, s>>>(o);
-      else if (o.flags & FQ3C_F32) fq3s_rot_append_kernel<float><<<o.M, rth, 0, s>>>(o);
-      else fq3s_rot_append_kernel<bf16><<<o.M, rth, 0, s>>>(o);
+      if (o.m_begin > 0 && o.M == 1 && (o.flags & FQ3C_F32)) fq3s_rot_append_kernel<float, true, 1024><<<1, rth, 0, s>>>(o);
+      else if (o.m_begin > 0 && o.M == 1) fq3s_rot_append_kernel<bf16, true, 1024><<<1, rth, 0, s>>>(o);
+      else if (rth > 256 && (o.flags & FQ3C_F32)) fq3s_rot_append_kernel<float, false, 1024><<<o.M, rth, 0, s>>>(o);
+      else if (rth > 256) fq3s_rot_append_kernel<bf16, false, 1024><<<o.M, rth, 0, s>>>(o);
+      else if (o.flags & FQ3C_F32) fq3s_rot_append_kernel<float><<<o.M, 256, 0, s>>>(o);
+      else fq3s_rot_append_kernel<bf16><<<o.M, 256, 0, s>>>(o);
       if (o.m_begin > 0 && o.M > 1) {
         const dim3 grid(o.M / o.m_begin + 1, (o.i1 * std::max(o.i2, o.cin) + 255) / 256, 2);
         if (o.flags & FQ3C_F32) fq3s_pool_append_kernel<float><<<grid, 256, 0, s>>>(o);

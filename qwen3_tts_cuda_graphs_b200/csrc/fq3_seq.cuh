@@ -1464,15 +1464,15 @@ __global__ void __launch_bounds__(256) fq3s_pool_append_kernel(const fq3c_op o) 
   else pool_run<TC>(reinterpret_cast<const TC*>(o.C2), o.ldr, reinterpret_cast<TC*>(o.ws), b, P, c, min(n, c + 1), 1);
 }
 
-// grid (M), 256 threads (up to 1024 for a few rows), a warp per query / key head.  Angles in f32: position (exact as a float below 2^24) times the frequency,
+// grid (M), up to THREADS threads (256, or 1024 for a few rows), a warp per query / key head.  Angles in f32: position (exact as a float below 2^24) times the frequency,
 // full-range sincosf; cos and sin times the amplitude f1 when that is set.  With norm weights a head is first divided by its root
 // mean square (eps f0) and multiplied by them; with FQ3C_UNIT it is divided only (a rotation keeps the root mean square, so it does
 // not matter which comes first).  Queries in place, keys (read from `res` rows when given) into the cache.
 // m_begin = P > 0: every run of P positions bP .. bP + P - 1 that the step completes leaves the mean of its P cached keys and values as
 // row b of norm_out / ws.  A single row does it here (POOL; its block has just written the run's last row); more rows take
 // fq3s_pool_append_kernel behind this launch.
-template <typename TC, bool POOL = false>
-__global__ void __launch_bounds__(1024) fq3s_rot_append_kernel(const fq3c_op o) {
+template <typename TC, bool POOL = false, int THREADS = 256>
+__global__ void __launch_bounds__(THREADS) fq3s_rot_append_kernel(const fq3c_op o) {
   const int m = blockIdx.x, H = o.i0, G = o.i1, d = o.i2, dv = o.cin, half = o.taps >> 1;
   const int pos = (o.p0 ? *reinterpret_cast<const int*>(o.p0) : 0) + m;
   float* row = const_cast<float*>(reinterpret_cast<const float*>(o.A)) + (size_t)m * o.lda;
@@ -2864,7 +2864,7 @@ __host__ __device__ constexpr int cd_walk_floats(int dk) {
   return 2 * cd_record(dk) + DVT * cd_pitch(dk) + 4 * 2 * CD_C * (DVT + 1) + DVT * CD_TP + 4;
 }
 template <int DVT, int RQ>
-__global__ void __launch_bounds__(CD_WALK_THREADS) fq3s_cdelta_walk_kernel(const fq3c_op o) {
+__global__ void __launch_bounds__(CD_WALK_THREADS, 1) fq3s_cdelta_walk_kernel(const fq3c_op o) {
   extern __shared__ __align__(128) float cw[];
   __shared__ __align__(8) unsigned long long full[2];
   constexpr int NCP = DVT / 2, QS = 128 / NCP, CG = DVT / 4, KH = 4 / CG, PP = DVT + 1, JW = DVT / 4;
